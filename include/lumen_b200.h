@@ -51,6 +51,7 @@ typedef struct lumen_kv_cache lumen_kv_cache;             /* KVCacheInner */
 typedef struct lumen_llama_kv_cache lumen_llama_kv_cache; /* LlamaKVCache */
 typedef struct lumen_self_attention lumen_self_attention;
 typedef struct lumen_llama lumen_llama;
+typedef struct lumen_model lumen_model; /* any language model */
 
 /* ---- context ------------------------------------------------------------------------------
  * No counterpart in the reference (it has no device or process boundary).  tp_size > 1 makes
@@ -256,6 +257,73 @@ size_t lumen_llama_weight_bytes(const lumen_llama *m);
  * end, followed by one stamp per phase taken when the producer issued the phase's first weight tile.
  * Copies up to `capacity` stamps of the last step to the host. */
 int lumen_llama_decode_trace(lumen_llama *m, uint64_t *out, size_t capacity, size_t *n_out);
+
+/* ---- models given as a list of layers ---------------------------------------------------------
+ * A second kind of language model beside LlamaModel (no counterpart in the reference): every layer is described
+ * by its own entry, so that layers of one model may differ.  Available mixers and feed-forwards:
+ *   latent attention   queries of `heads` x (dim + rot_dim); keys and values come from one latent of kv_rank numbers
+ *                      per token (RMS-normed) plus one rotated key part of rot_dim numbers that all heads share; the
+ *                      cache holds these kv_rank + rot_dim numbers per token.  The first rot_dims of the rotated part
+ *                      turn in interleaved pairs (2i, 2i+1) with frequency rot_base^(-2i/rot_dims).  A sigmoid gate per head
+ *                      scales the head's output.
+ *   dense              down(gelu_tanh(up(x)))
+ *   moe                `top` of `experts` clamped-SwiGLU experts by sigmoid scores (the score scales the expert's input),
+ *                      plus a shared expert (shared_ff == 0: none)
+ * Sublayers read the residual itself; their outputs are RMS-normed with gain 1 + w and added.  Options of the model:
+ * a bigram embedding (bigram_buckets == 0: none), and a per-layer token input after the feed-forward (side_dim == 0: none). */
+#define LUMEN_MLP_NONE 0
+#define LUMEN_MLP_DENSE 1
+#define LUMEN_MLP_MOE 2
+typedef struct {
+    size_t heads;
+    size_t dim;
+    size_t rot_dim;
+    size_t vdim;
+    size_t kv_rank;
+    size_t rot_dims;
+    double rot_base;
+    float scale;
+    int mlp_kind;
+    size_t ff;
+    size_t experts;
+    size_t top;
+    size_t expert_ff;
+    float expert_limit;
+    size_t shared_ff;
+    float shared_limit;
+} lumen_decoder_layer;
+typedef struct {
+    size_t vocab_size;
+    size_t width;
+    size_t num_layers;
+    const lumen_decoder_layer *layers;
+    float norm_eps;
+    size_t max_seq_len;
+    size_t bigram_buckets;
+    size_t bigram_mul_prev;
+    size_t bigram_mul_cur;
+    size_t side_dim;
+    lumen_dtype weight_dtype;
+} lumen_decoder_config;
+/* Parameters are named as in the checkpoint (embed, bigram, side.embed, l<i>.mix.q, l<i>.mlp.e<j>.gate, final.norm, head, ...).
+ * weight_dtype f32: every product in 32-bit arithmetic.  weight_dtype bf16: bf16 products with 32-bit accumulation and
+ * a bf16 latent cache; positions, scores, norms, routers and the residual in 32-bit. */
+int lumen_decoder_new(lumen_ctx *ctx, const lumen_decoder_config *cfg, lumen_model **out);
+
+/* The interface every model shares; the lumen_llama_* entry points above are these under the reference's names. */
+int lumen_model_set_param(lumen_model *m, const char *name, const void *host_data, const size_t *shape, int ndim, lumen_dtype dtype);
+int lumen_model_init_kv_caches(lumen_model *m, size_t batch, lumen_kv_cache **caches_out);
+int lumen_model_reset_kv_caches(lumen_model *m, lumen_kv_cache **caches, size_t n_caches);
+int lumen_model_forward(lumen_model *m, const float *ids_host, size_t b, size_t s, lumen_kv_cache **caches,
+                        size_t n_caches, float *logits_host);
+int lumen_model_forward_last(lumen_model *m, const float *ids_host, size_t b, size_t s, lumen_kv_cache **caches,
+                             size_t n_caches, float *logits_host);
+int lumen_model_forward_device(lumen_model *m, const float *ids_dev, size_t b, size_t s, lumen_kv_cache **caches,
+                               size_t n_caches, float *logits_dev);
+int lumen_model_forward_sample(lumen_model *m, const float *ids_host, size_t s, lumen_kv_cache **caches, size_t n_caches,
+                               const lumen_sample_params *params, int32_t *token_out);
+size_t lumen_model_weight_bytes(const lumen_model *m);
+int lumen_model_free(lumen_model *m);
 
 /* ---- measurement helpers (no counterpart in the reference) ----------------------------------
  * A kernel timed as a kernel: `iters` calls of lumen_gemv (src/ops/matmul.rs:42-69) / lumen_attention_decode

@@ -35,6 +35,29 @@ class LlamaConfigC(C.Structure):
     ]
 
 
+class DecoderLayerC(C.Structure):
+    """`lumen_decoder_layer`: one layer of a model given as a list of layers."""
+
+    _fields_ = [
+        ("heads", C.c_size_t), ("dim", C.c_size_t), ("rot_dim", C.c_size_t), ("vdim", C.c_size_t), ("kv_rank", C.c_size_t),
+        ("rot_dims", C.c_size_t), ("rot_base", C.c_double), ("scale", C.c_float), ("mlp_kind", C.c_int), ("ff", C.c_size_t),
+        ("experts", C.c_size_t), ("top", C.c_size_t), ("expert_ff", C.c_size_t), ("expert_limit", C.c_float),
+        ("shared_ff", C.c_size_t), ("shared_limit", C.c_float),
+    ]
+
+
+class DecoderConfigC(C.Structure):
+    """`lumen_decoder_config`."""
+
+    _fields_ = [
+        ("vocab_size", C.c_size_t), ("width", C.c_size_t), ("num_layers", C.c_size_t), ("layers", C.POINTER(DecoderLayerC)),
+        ("norm_eps", C.c_float), ("max_seq_len", C.c_size_t), ("bigram_buckets", C.c_size_t), ("bigram_mul_prev", C.c_size_t),
+        ("bigram_mul_cur", C.c_size_t), ("side_dim", C.c_size_t), ("weight_dtype", C.c_int),
+    ]
+
+
+MLP_NONE, MLP_DENSE, MLP_MOE = 0, 1, 2
+
 _P = C.c_void_p
 _PP = C.POINTER(C.c_void_p)
 _SZ = C.c_size_t
@@ -107,6 +130,16 @@ PROTOTYPES = {
     "lumen_sample_top_p": (_I, [_P, _FP, _SZ, C.POINTER(SampleParamsC), C.POINTER(C.c_int32)]),
     "lumen_llama_forward_sample": (_I, [_P, _FP, _SZ, _PP, _SZ, C.POINTER(SampleParamsC), C.POINTER(C.c_int32)]),
     "lumen_llama_free": (_I, [_P]),
+    "lumen_decoder_new": (_I, [_P, C.POINTER(DecoderConfigC), _PP]),
+    "lumen_model_set_param": (_I, [_P, C.c_char_p, _P, _SZP, _I, _I]),
+    "lumen_model_init_kv_caches": (_I, [_P, _SZ, _PP]),
+    "lumen_model_reset_kv_caches": (_I, [_P, _PP, _SZ]),
+    "lumen_model_forward": (_I, [_P, _FP, _SZ, _SZ, _PP, _SZ, _FP]),
+    "lumen_model_forward_last": (_I, [_P, _FP, _SZ, _SZ, _PP, _SZ, _FP]),
+    "lumen_model_forward_device": (_I, [_P, _FP, _SZ, _SZ, _PP, _SZ, _FP]),
+    "lumen_model_forward_sample": (_I, [_P, _FP, _SZ, _PP, _SZ, C.POINTER(SampleParamsC), C.POINTER(C.c_int32)]),
+    "lumen_model_weight_bytes": (_SZ, [_P]),
+    "lumen_model_free": (_I, [_P]),
     "lumen_llama_weight_bytes": (_SZ, [_P]),
     "lumen_llama_decode_trace": (_I, [_P, C.POINTER(C.c_uint64), _SZ, _SZP]),
 }

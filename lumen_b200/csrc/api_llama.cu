@@ -16,6 +16,7 @@
 
 #include "common.cuh"
 #include "decode_mega.cuh"
+#include "model_base.cuh"
 #include "tp_plan.cuh"
 
 using namespace lumen;
@@ -47,23 +48,11 @@ struct Workspace {
 
 constexpr int kMaxSplits = 64;
 
-__global__ void f32_to_bf16_kernel(const float *in, __nv_bfloat16 *out, size_t n) {
-    size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < n) out[i] = __float2bfloat16_rn(in[i]);
-}
-__global__ void bf16_to_f32_kernel2(const __nv_bfloat16 *in, float *out, size_t n) {
-    size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < n) out[i] = __bfloat162float(in[i]);
-}
-
-size_t align_up(size_t v, size_t a) { return (v + a - 1) / a * a; }
-
 }  // namespace
 
-struct lumen_llama {
-    lumen_ctx *ctx = nullptr;
+struct lumen_llama : lumen_model {
     lumen_llama_config cfg{};
-    size_t D = 0, H = 0, V = 0, I = 0, L = 0;
+    size_t D = 0, H = 0, I = 0;
     size_t hq_l = 0, hkv_l = 0, qd_l = 0, kvd_l = 0, inter_l = 0, vocab_l = 0, qkv_rows = 0;
     size_t kv_head0 = 0, q_head0 = 0;  // first global head owned by this rank
     size_t esz = 4;
@@ -78,14 +67,7 @@ struct lumen_llama {
     char *embed = nullptr, *lm_head = nullptr;
     float *final_norm = nullptr;
     float *cos_t = nullptr, *sin_t = nullptr;
-    std::map<std::string, bool> is_set;
-    size_t n_expected = 0;
     Workspace ws;
-    // decode graphs keyed by (batch, splits, first cache's k pointer)
-    std::map<std::tuple<size_t, int, const void *>, cudaGraphExec_t> graphs;
-    std::map<std::tuple<size_t, int, const void *>, int> eager_runs;
-    std::map<std::tuple<size_t, int, const void *>, unsigned long long> graph_nodes;
-    bool use_graph = true;
     // persistent whole-step decode kernel (batch 1)
     bool use_mega = true;
     MegaLayer *d_mega_layers = nullptr;
@@ -97,15 +79,17 @@ struct lumen_llama {
     size_t tmaps_capacity = 0;
     const void *mega_key = nullptr;  // first cache's k pointer the layer table was built for
     unsigned long long *d_trace = nullptr;  // phase timestamps of the last persistent step (LUMEN_DECODE_TRACE=1)
+
+    ~lumen_llama() override;
+    int set_param(const char *name, const void *host_data, const size_t *shape, int ndim, lumen_dtype dtype) override;
+    int init_kv_caches(size_t batch, lumen_kv_cache **out) override;
+    int check_caches(size_t b, size_t s, lumen_kv_cache **caches, size_t n_caches) override;
+    int ensure_workspace(size_t rows) override;
+    int run_forward(size_t b, size_t s, lumen_kv_cache **caches, bool last_only) override;
+    size_t weight_bytes() const override { return stream_bytes; }
 };
 
 namespace {
-
-void drop_graphs(lumen_llama *m) {
-    for (auto &kv : m->graphs) cudaGraphExecDestroy(kv.second);
-    m->graphs.clear();
-    m->eager_runs.clear();
-}
 
 int ensure_workspace(lumen_llama *m, size_t M) {
     Workspace &w = m->ws;
@@ -113,7 +97,7 @@ int ensure_workspace(lumen_llama *m, size_t M) {
     LUMEN_TRY(ensure_tp_sum(ctx));  // (every rank passes here at the same points; no-op after the first time)
     if (M <= w.M) return LUMEN_OK;
     LUMEN_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
-    drop_graphs(m);
+    m->drop_graphs();
     if (w.base) cudaFree(w.base);
     if (w.h_ids) cudaFreeHost(w.h_ids);
     if (w.h_logits) cudaFreeHost(w.h_logits);
@@ -145,43 +129,8 @@ int ensure_workspace(lumen_llama *m, size_t M) {
     w.h_logits_elems = std::min<size_t>(M * m->V, (size_t)16 << 20);  // pinned staging up to 64 MB
     LUMEN_CUDA(ctx, cudaMallocHost(&w.h_logits, std::max<size_t>(w.h_logits_elems, 1) * sizeof(float)));
     w.M = M;
+    m->io = StepIo{w.ids, w.logits, w.h_ids, w.h_logits, w.h_logits_elems};
     return LUMEN_OK;
-}
-
-// Copies the [rows x ncols] block starting at column col0 of a row-major host matrix with `cols_total`
-// columns into a dense device matrix of dtype dst_dt, converting between f32 and bf16 when needed.
-int upload_block(lumen_ctx *ctx, void *dst, lumen_dtype dst_dt, const void *src_host, lumen_dtype src_dt, size_t rows,
-                 size_t cols_total, size_t col0, size_t ncols) {
-    if (rows == 0 || ncols == 0) return LUMEN_OK;
-    const size_t se = src_dt == LUMEN_F32 ? 4 : 2;
-    const char *src = static_cast<const char *>(src_host) + col0 * se;
-    cudaStream_t s = ctx->stream;
-    if (src_dt == dst_dt) {
-        LUMEN_CUDA(ctx, cudaMemcpy2DAsync(dst, ncols * se, src, cols_total * se, ncols * se, rows, cudaMemcpyHostToDevice, s));
-        LUMEN_CUDA(ctx, cudaStreamSynchronize(s));
-        return LUMEN_OK;
-    }
-    // Convert in row chunks to bound the staging buffer.
-    const size_t chunk_rows = std::max<size_t>(1, ((size_t)64 << 20) / (ncols * se));
-    void *tmp = nullptr;
-    LUMEN_CUDA(ctx, cudaMalloc(&tmp, std::min(rows, chunk_rows) * ncols * se));
-    const size_t de = dst_dt == LUMEN_F32 ? 4 : 2;
-    int rc = LUMEN_OK;
-    for (size_t r0 = 0; r0 < rows && rc == LUMEN_OK; r0 += chunk_rows) {
-        const size_t nr = std::min(chunk_rows, rows - r0), n = nr * ncols;
-        cudaError_t e = cudaMemcpy2DAsync(tmp, ncols * se, src + r0 * cols_total * se, cols_total * se, ncols * se, nr,
-                                          cudaMemcpyHostToDevice, s);
-        if (e != cudaSuccess) { rc = cuda_fail(ctx, e, "cudaMemcpy2DAsync"); break; }
-        char *d = static_cast<char *>(dst) + r0 * ncols * de;
-        if (dst_dt == LUMEN_BF16)
-            f32_to_bf16_kernel<<<(unsigned)((n + 255) / 256), 256, 0, s>>>((const float *)tmp, (__nv_bfloat16 *)d, n);
-        else
-            bf16_to_f32_kernel2<<<(unsigned)((n + 255) / 256), 256, 0, s>>>((const __nv_bfloat16 *)tmp, (float *)d, n);
-        e = cudaStreamSynchronize(s);
-        if (e != cudaSuccess) rc = cuda_fail(ctx, e, "convert upload");
-    }
-    cudaFree(tmp);
-    return rc;
 }
 
 int ensure_weight_split(lumen_llama *m) {
@@ -402,7 +351,7 @@ int check_caches(lumen_llama *m, size_t b, size_t s, lumen_kv_cache **caches, si
         lumen_kv_cache *c = caches[l];
         if (!c) return set_error(ctx, LUMEN_ERR_INVALID, "null KV cache for layer %zu", l);
         LUMEN_TRY(kv_resync_len(c));
-        if (c->b != b || c->h_kv != m->hkv_l || c->d != m->D)
+        if (c->b != b || c->h_kv != m->hkv_l || c->d != m->D || !c->v)
             return set_error(ctx, LUMEN_ERR_SHAPE, "KV cache %zu geometry [%zu,%zu,%zu,%zu] does not match batch %zu / model", l, c->b, c->h_kv, c->max_seq, c->d, b);
         if (c->len != caches[0]->len) return set_error(ctx, LUMEN_ERR_INVALID, "KV caches have different lengths");
         if (s == 1) {  // decode asserts overflow before touching RoPE (self_attention.rs:144-149)
@@ -557,77 +506,107 @@ int run_forward(lumen_llama *m, size_t b, size_t s, lumen_kv_cache **caches, boo
     StepPlan p{b, s, b * s, s == 1, 1};
     if (p.M > 8) LUMEN_TRY(ensure_weight_split(m));  // (outside any stream capture; the streaming kernels of <= 8 rows read f32)
     if (p.decode) p.nsplit = pick_decode_splits(m, b, caches[0]->len + 1);
-    int rc = LUMEN_OK;
-    if (p.decode && m->use_graph) {
-        auto key = std::make_tuple(b, p.nsplit, (const void *)caches[0]->k);
-        auto it = m->graphs.find(key);
-        if (it == m->graphs.end() && m->eager_runs[key]++ >= 1) {
-            cudaGraph_t graph = nullptr;
-            const unsigned long long before = ctx->launches;
-            LUMEN_CUDA(ctx, cudaStreamBeginCapture(ctx->stream, cudaStreamCaptureModeThreadLocal));
-            rc = enqueue_forward(m, p, caches, last_only);
-            cudaError_t e = cudaStreamEndCapture(ctx->stream, &graph);
-            m->graph_nodes[key] = ctx->launches - before;  // captured, not run
-            ctx->launches = before;
-            if (rc != LUMEN_OK) {
-                if (graph) cudaGraphDestroy(graph);
-                return rc;
-            }
-            if (e != cudaSuccess) return cuda_fail(ctx, e, "cudaStreamEndCapture");
-            cudaGraphExec_t exec = nullptr;
-            e = cudaGraphInstantiate(&exec, graph, 0);
-            cudaGraphDestroy(graph);
-            if (e != cudaSuccess) return cuda_fail(ctx, e, "cudaGraphInstantiate");
-            it = m->graphs.emplace(key, exec).first;
-        }
-        if (it != m->graphs.end()) {
-            LUMEN_CUDA(ctx, cudaGraphLaunch(it->second, ctx->stream));
-            ctx->launches += m->graph_nodes[key];
-        } else {
-            rc = enqueue_forward(m, p, caches, last_only);
-        }
-    } else {
-        rc = enqueue_forward(m, p, caches, last_only);
-    }
+    const int rc = p.decode ? m->run_graphed(std::make_tuple(b, p.nsplit, (const void *)caches[0]->k),
+                                             [&] { return enqueue_forward(m, p, caches, last_only); })
+                            : enqueue_forward(m, p, caches, last_only);
     if (rc == LUMEN_OK)
         for (size_t l = 0; l < m->L; ++l) caches[l]->len += s;
     return rc;
 }
 
-int forward_host(lumen_llama *m, const float *ids_host, size_t b, size_t s, lumen_kv_cache **caches, size_t n_caches,
-                 float *logits_host, bool last_only) {
-    if (!m || !ids_host || !logits_host) return LUMEN_ERR_INVALID;
-    lumen_ctx *ctx = m->ctx;
-    if (m->is_set.size() < m->n_expected) return set_error(ctx, LUMEN_ERR_MISSING_PARAM, "%zu of %zu parameters set", m->is_set.size(), m->n_expected);
-    const size_t M = b * s;
-    if (M == 0) return LUMEN_OK;
-    LUMEN_TRY(check_caches(m, b, s, caches, n_caches));
-    // Embedding range check on the host (src/layers/basic/embedding.rs:50-56) before anything is launched.
-    for (size_t i = 0; i < M; ++i) {
-        const float f = ids_host[i];
-        if (f >= (float)m->V && f == f) return set_error(ctx, LUMEN_ERR_EMBED_RANGE, "Embedding index out of bounds: %.0f >= %zu", (double)f, m->V);
-    }
-    LUMEN_TRY(ensure_workspace(m, M));
-    Workspace &w = m->ws;
-    // The pinned staging buffers are reused every step: wait for the previous step's copies first.
-    LUMEN_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
-    memcpy(w.h_ids, ids_host, M * sizeof(float));
-    LUMEN_CUDA(ctx, cudaMemcpyAsync(w.ids, w.h_ids, M * sizeof(float), cudaMemcpyHostToDevice, ctx->stream));
-    LUMEN_TRY(run_forward(m, b, s, caches, last_only));
-    const size_t rows = (last_only && s > 1) ? b : M;
-    const size_t n = rows * m->V;
-    if (n <= w.h_logits_elems) {
-        LUMEN_CUDA(ctx, cudaMemcpyAsync(w.h_logits, w.logits, n * 4, cudaMemcpyDeviceToHost, ctx->stream));
-        LUMEN_TRY(check_device_status(ctx));
-        memcpy(logits_host, w.h_logits, n * 4);
-    } else {
-        LUMEN_CUDA(ctx, cudaMemcpyAsync(logits_host, w.logits, n * 4, cudaMemcpyDeviceToHost, ctx->stream));
-        LUMEN_TRY(check_device_status(ctx));
-    }
-    return LUMEN_OK;
+}  // namespace
+
+int lumen_llama::check_caches(size_t b, size_t s, lumen_kv_cache **caches, size_t n_caches) { return ::check_caches(this, b, s, caches, n_caches); }
+int lumen_llama::ensure_workspace(size_t rows) { return ::ensure_workspace(this, rows); }
+int lumen_llama::run_forward(size_t b, size_t s, lumen_kv_cache **caches, bool last_only) { return ::run_forward(this, b, s, caches, last_only); }
+
+lumen_llama::~lumen_llama() {
+    if (d_mega_layers) cudaFree(d_mega_layers);
+    if (d_sched) cudaFree(d_sched);
+    if (d_sched_count) cudaFree(d_sched_count);
+    if (d_tmaps) cudaFree(d_tmaps);
+    if (d_trace) cudaFree(d_trace);
+    if (ws.base) cudaFree(ws.base);
+    if (ws.h_ids) cudaFreeHost(ws.h_ids);
+    if (ws.h_logits) cudaFreeHost(ws.h_logits);
+    if (wslab) cudaFree(wslab);
+    if (wsplit) cudaFree(wsplit);
 }
 
-}  // namespace
+int lumen_llama::set_param(const char *name, const void *host_data, const size_t *shape, int ndim, lumen_dtype dtype) {
+    lumen_llama *m = this;
+    const lumen_dtype wdt = m->cfg.weight_dtype;
+    const size_t se = dtype == LUMEN_F32 ? 4 : 2, e = m->esz, H = m->H;
+    m->wsplit_valid = false;  // (the kept bf16 split of the f32 weights is rebuilt before its next use)
+    // Which part of the tensor this rank keeps comes from the shard plan; what is left here is where it goes.
+    TpSlice sl;
+    long li = -1;
+    const char *leaf = name;
+    int rc = tp_param_slice(m->cfg, ctx->tp_size, ctx->tp_rank, name, sl, &li, &leaf);
+    if (rc != LUMEN_OK) return set_error(ctx, rc, "unknown parameter '%s'", name);
+    if (sl.cols == 0) {
+        if (ndim != 1 || shape[0] != sl.rows) return set_error(ctx, LUMEN_ERR_SHAPE, "%s: expected [%zu]", name, sl.rows);
+    } else if (ndim != 2 || shape[0] != sl.rows || shape[1] != sl.cols) {
+        return set_error(ctx, LUMEN_ERR_SHAPE, "%s: expected [%zu,%zu]", name, sl.rows, sl.cols);
+    }
+    char *dst = nullptr;
+    lumen_dtype ddt = wdt;
+    if (li < 0) {
+        if (!strcmp(leaf, "model.embed_tokens.weight")) dst = m->embed;
+        else if (!strcmp(leaf, "lm_head.weight")) dst = m->lm_head;
+        else { dst = reinterpret_cast<char *>(m->final_norm); ddt = LUMEN_F32; }
+    } else {
+        LayerW &w = m->layers[li];
+        if (!strcmp(leaf, "self_attn.q_proj.weight")) dst = w.wqkv;
+        else if (!strcmp(leaf, "self_attn.k_proj.weight")) dst = w.wqkv + m->qd_l * H * e;
+        else if (!strcmp(leaf, "self_attn.v_proj.weight")) dst = w.wqkv + (m->qd_l + m->kvd_l) * H * e;
+        else if (!strcmp(leaf, "self_attn.o_proj.weight")) dst = w.wo;
+        else if (!strcmp(leaf, "mlp.gate_proj.weight")) dst = w.wgate;
+        else if (!strcmp(leaf, "mlp.up_proj.weight")) dst = w.wup;
+        else if (!strcmp(leaf, "mlp.down_proj.weight")) dst = w.wdown;
+        else {
+            ddt = LUMEN_F32;
+            if (!strcmp(leaf, "input_layernorm.weight")) dst = reinterpret_cast<char *>(w.norm1);
+            else if (!strcmp(leaf, "post_attention_layernorm.weight")) dst = reinterpret_cast<char *>(w.norm2);
+            else if (!strcmp(leaf, "self_attn.q_norm.weight")) dst = reinterpret_cast<char *>(w.qn);
+            else dst = reinterpret_cast<char *>(w.kn);
+        }
+    }
+    if (sl.cols == 0) {
+        rc = upload_block(ctx, dst, ddt, host_data, dtype, 1, sl.rows, 0, sl.rows);
+    } else {
+        const char *src = static_cast<const char *>(host_data) + sl.row0 * sl.cols * se;
+        rc = upload_block(ctx, dst, ddt, src, dtype, sl.nrows, sl.cols, sl.col0, sl.ncols);
+    }
+    if (rc == LUMEN_ERR_PARAM_NAME) return set_error(ctx, rc, "unknown parameter '%s'", name);
+    if (rc == LUMEN_OK) m->is_set[name] = true;
+    return rc;
+}
+
+int lumen_llama::init_kv_caches(size_t batch, lumen_kv_cache **caches_out) {
+    lumen_llama *m = this;
+    const size_t per = batch * m->hkv_l * m->cfg.max_seq_len * m->D;  // floats per k (or v) slab of a layer
+    const size_t bytes = m->L * 2 * per * sizeof(float) + align_up(m->L * sizeof(int), 256);
+    int rc = LUMEN_OK;
+    lumen_storage *slab = new_cache_slab(ctx, bytes, &rc);
+    if (!slab) return rc;
+    float *base = static_cast<float *>(slab->ptr);
+    int *lens = reinterpret_cast<int *>(base + m->L * 2 * per);
+    for (size_t l = 0; l < m->L; ++l) {
+        auto *c = new lumen_kv_cache();
+        c->ctx = ctx; c->b = batch; c->h_kv = m->hkv_l; c->max_seq = m->cfg.max_seq_len; c->d = m->D;
+        c->k = base + (2 * l) * per;
+        c->v = base + (2 * l + 1) * per;
+        c->d_len = lens + l;
+        c->seen_abort = ctx->abort_gen;
+        c->owns_slab = false;
+        c->slab = slab;
+        slab->refs += 1;
+        caches_out[l] = c;
+    }
+    if (m->L == 0) { cudaFree(slab->ptr); delete slab; }
+    return LUMEN_OK;
+}
 
 extern "C" {
 
@@ -718,144 +697,33 @@ int lumen_llama_new(lumen_ctx *ctx, const lumen_llama_config *cfg, lumen_llama *
 }
 
 int lumen_llama_set_param(lumen_llama *m, const char *name, const void *host_data, const size_t *shape, int ndim, lumen_dtype dtype) {
-    if (!m || !name || !host_data || !shape) return LUMEN_ERR_INVALID;
-    lumen_ctx *ctx = m->ctx;
-    if (dtype != LUMEN_F32 && dtype != LUMEN_BF16) return set_error(ctx, LUMEN_ERR_DTYPE, "set_param: dtype %d", (int)dtype);
-    const lumen_dtype wdt = m->cfg.weight_dtype;
-    const size_t se = dtype == LUMEN_F32 ? 4 : 2, e = m->esz, H = m->H;
-    m->wsplit_valid = false;  // (the kept bf16 split of the f32 weights is rebuilt before its next use)
-    // Which part of the tensor this rank keeps comes from the shard plan; what is left here is where it goes.
-    TpSlice sl;
-    long li = -1;
-    const char *leaf = name;
-    int rc = tp_param_slice(m->cfg, ctx->tp_size, ctx->tp_rank, name, sl, &li, &leaf);
-    if (rc != LUMEN_OK) return set_error(ctx, rc, "unknown parameter '%s'", name);
-    if (sl.cols == 0) {
-        if (ndim != 1 || shape[0] != sl.rows) return set_error(ctx, LUMEN_ERR_SHAPE, "%s: expected [%zu]", name, sl.rows);
-    } else if (ndim != 2 || shape[0] != sl.rows || shape[1] != sl.cols) {
-        return set_error(ctx, LUMEN_ERR_SHAPE, "%s: expected [%zu,%zu]", name, sl.rows, sl.cols);
-    }
-    char *dst = nullptr;
-    lumen_dtype ddt = wdt;
-    if (li < 0) {
-        if (!strcmp(leaf, "model.embed_tokens.weight")) dst = m->embed;
-        else if (!strcmp(leaf, "lm_head.weight")) dst = m->lm_head;
-        else { dst = reinterpret_cast<char *>(m->final_norm); ddt = LUMEN_F32; }
-    } else {
-        LayerW &w = m->layers[li];
-        if (!strcmp(leaf, "self_attn.q_proj.weight")) dst = w.wqkv;
-        else if (!strcmp(leaf, "self_attn.k_proj.weight")) dst = w.wqkv + m->qd_l * H * e;
-        else if (!strcmp(leaf, "self_attn.v_proj.weight")) dst = w.wqkv + (m->qd_l + m->kvd_l) * H * e;
-        else if (!strcmp(leaf, "self_attn.o_proj.weight")) dst = w.wo;
-        else if (!strcmp(leaf, "mlp.gate_proj.weight")) dst = w.wgate;
-        else if (!strcmp(leaf, "mlp.up_proj.weight")) dst = w.wup;
-        else if (!strcmp(leaf, "mlp.down_proj.weight")) dst = w.wdown;
-        else {
-            ddt = LUMEN_F32;
-            if (!strcmp(leaf, "input_layernorm.weight")) dst = reinterpret_cast<char *>(w.norm1);
-            else if (!strcmp(leaf, "post_attention_layernorm.weight")) dst = reinterpret_cast<char *>(w.norm2);
-            else if (!strcmp(leaf, "self_attn.q_norm.weight")) dst = reinterpret_cast<char *>(w.qn);
-            else dst = reinterpret_cast<char *>(w.kn);
-        }
-    }
-    if (sl.cols == 0) {
-        rc = upload_block(ctx, dst, ddt, host_data, dtype, 1, sl.rows, 0, sl.rows);
-    } else {
-        const char *src = static_cast<const char *>(host_data) + sl.row0 * sl.cols * se;
-        rc = upload_block(ctx, dst, ddt, src, dtype, sl.nrows, sl.cols, sl.col0, sl.ncols);
-    }
-    if (rc == LUMEN_ERR_PARAM_NAME) return set_error(ctx, rc, "unknown parameter '%s'", name);
-    if (rc == LUMEN_OK) m->is_set[name] = true;
-    return rc;
+    return lumen_model_set_param(m, name, host_data, shape, ndim, dtype);
 }
 
-int lumen_llama_init_kv_caches(lumen_llama *m, size_t batch, lumen_kv_cache **caches_out) {
-    if (!m || !caches_out) return LUMEN_ERR_INVALID;
-    lumen_ctx *ctx = m->ctx;
-    const size_t per = batch * m->hkv_l * m->cfg.max_seq_len * m->D;  // floats per k (or v) slab of a layer
-    const size_t bytes = m->L * 2 * per * sizeof(float) + align_up(m->L * sizeof(int), 256);
-    auto *slab = new lumen_storage();
-    slab->ctx = ctx;
-    slab->bytes = bytes;
-    slab->refs = 0;
-    cudaError_t e = cudaMalloc(&slab->ptr, std::max<size_t>(bytes, 256));
-    if (e != cudaSuccess) { delete slab; return cuda_fail(ctx, e, "cudaMalloc(kv slab)"); }
-    LUMEN_CUDA(ctx, cudaMemsetAsync(slab->ptr, 0, bytes, ctx->stream));  // Array4::zeros, self_attention.rs:35-36
-    float *base = static_cast<float *>(slab->ptr);
-    int *lens = reinterpret_cast<int *>(base + m->L * 2 * per);
-    for (size_t l = 0; l < m->L; ++l) {
-        auto *c = new lumen_kv_cache();
-        c->ctx = ctx; c->b = batch; c->h_kv = m->hkv_l; c->max_seq = m->cfg.max_seq_len; c->d = m->D;
-        c->k = base + (2 * l) * per;
-        c->v = base + (2 * l + 1) * per;
-        c->d_len = lens + l;
-        c->seen_abort = ctx->abort_gen;
-        c->owns_slab = false;
-        c->slab = slab;
-        slab->refs += 1;
-        caches_out[l] = c;
-    }
-    if (m->L == 0) { cudaFree(slab->ptr); delete slab; }
-    return LUMEN_OK;
-}
+int lumen_llama_init_kv_caches(lumen_llama *m, size_t batch, lumen_kv_cache **caches_out) { return lumen_model_init_kv_caches(m, batch, caches_out); }
 
-int lumen_llama_reset_kv_caches(lumen_llama *m, lumen_kv_cache **caches, size_t n_caches) {
-    if (!m || (!caches && n_caches)) return LUMEN_ERR_INVALID;
-    for (size_t i = 0; i < n_caches; ++i) LUMEN_TRY(lumen_kv_reset(caches[i]));
-    return LUMEN_OK;
-}
+int lumen_llama_reset_kv_caches(lumen_llama *m, lumen_kv_cache **caches, size_t n_caches) { return lumen_model_reset_kv_caches(m, caches, n_caches); }
 
 int lumen_llama_forward(lumen_llama *m, const float *ids_host, size_t b, size_t s, lumen_kv_cache **caches, size_t n_caches,
                         size_t pos, float *logits_host) {
     (void)pos;  // `_pos` is ignored by the reference too (llama.rs:180-181)
-    return forward_host(m, ids_host, b, s, caches, n_caches, logits_host, false);
+    return lumen_model_forward(m, ids_host, b, s, caches, n_caches, logits_host);
 }
 
 int lumen_llama_forward_last(lumen_llama *m, const float *ids_host, size_t b, size_t s, lumen_kv_cache **caches, size_t n_caches,
                              size_t pos, float *logits_host) {
     (void)pos;
-    return forward_host(m, ids_host, b, s, caches, n_caches, logits_host, true);
+    return lumen_model_forward_last(m, ids_host, b, s, caches, n_caches, logits_host);
 }
 
 int lumen_llama_forward_sample(lumen_llama *m, const float *ids_host, size_t s, lumen_kv_cache **caches, size_t n_caches,
                                const lumen_sample_params *sp, int32_t *token_out) {
-    if (!m || !ids_host || !sp || !token_out || (sp->n_recent && !sp->recent_tokens)) return LUMEN_ERR_INVALID;
-    lumen_ctx *ctx = m->ctx;
-    if (m->is_set.size() < m->n_expected) return set_error(ctx, LUMEN_ERR_MISSING_PARAM, "%zu of %zu parameters set", m->is_set.size(), m->n_expected);
-    if (s == 0) return set_error(ctx, LUMEN_ERR_SHAPE, "forward_sample: empty input");
-    LUMEN_TRY(check_caches(m, 1, s, caches, n_caches));
-    for (size_t i = 0; i < s; ++i) {
-        const float f = ids_host[i];
-        if (f >= (float)m->V && f == f) return set_error(ctx, LUMEN_ERR_EMBED_RANGE, "Embedding index out of bounds: %.0f >= %zu", (double)f, m->V);
-    }
-    LUMEN_TRY(ensure_workspace(m, s));
-    Workspace &w = m->ws;
-    LUMEN_CUDA(ctx, cudaStreamSynchronize(ctx->stream));  // the pinned staging buffer is reused every step
-    memcpy(w.h_ids, ids_host, s * sizeof(float));
-    LUMEN_CUDA(ctx, cudaMemcpyAsync(w.ids, w.h_ids, s * sizeof(float), cudaMemcpyHostToDevice, ctx->stream));
-    LUMEN_TRY(run_forward(m, 1, s, caches, true));  // last position's logits in w.logits[V]
-    int *token_dev = reinterpret_cast<int *>(w.ids);  // the id buffer is free again once the forward is enqueued behind it
-    LUMEN_TRY(launch_sample_top_p(ctx, w.logits, m->V, sp->temperature, sp->top_p, sp->repetition_penalty, sp->recent_tokens,
-                                  sp->n_recent, sp->uniform, token_dev, ctx->stream));
-    LUMEN_CUDA(ctx, cudaMemcpyAsync(w.h_ids, token_dev, sizeof(int), cudaMemcpyDeviceToHost, ctx->stream));
-    LUMEN_TRY(check_device_status(ctx));
-    memcpy(token_out, w.h_ids, sizeof(int));
-    return LUMEN_OK;
+    return lumen_model_forward_sample(m, ids_host, s, caches, n_caches, sp, token_out);
 }
 
 int lumen_llama_forward_device(lumen_llama *m, const float *ids_dev, size_t b, size_t s, lumen_kv_cache **caches, size_t n_caches,
                                float *logits_dev) {
-    if (!m || !ids_dev || !logits_dev) return LUMEN_ERR_INVALID;
-    lumen_ctx *ctx = m->ctx;
-    if (m->is_set.size() < m->n_expected) return set_error(ctx, LUMEN_ERR_MISSING_PARAM, "%zu of %zu parameters set", m->is_set.size(), m->n_expected);
-    const size_t M = b * s;
-    if (M == 0) return LUMEN_OK;
-    LUMEN_TRY(check_caches(m, b, s, caches, n_caches));
-    LUMEN_TRY(ensure_workspace(m, M));
-    LUMEN_CUDA(ctx, cudaMemcpyAsync(m->ws.ids, ids_dev, M * sizeof(float), cudaMemcpyDeviceToDevice, ctx->stream));
-    LUMEN_TRY(run_forward(m, b, s, caches, false));
-    LUMEN_CUDA(ctx, cudaMemcpyAsync(logits_dev, m->ws.logits, M * m->V * sizeof(float), cudaMemcpyDeviceToDevice, ctx->stream));
-    return LUMEN_OK;
+    return lumen_model_forward_device(m, ids_dev, b, s, caches, n_caches, logits_dev);
 }
 
 size_t lumen_llama_weight_bytes(const lumen_llama *m) { return m ? m->stream_bytes : 0; }
@@ -871,22 +739,6 @@ int lumen_llama_decode_trace(lumen_llama *m, uint64_t *out, size_t capacity, siz
     return LUMEN_OK;
 }
 
-int lumen_llama_free(lumen_llama *m) {
-    if (!m) return LUMEN_ERR_INVALID;
-    cudaStreamSynchronize(m->ctx->stream);
-    drop_graphs(m);
-    if (m->d_mega_layers) cudaFree(m->d_mega_layers);
-    if (m->d_sched) cudaFree(m->d_sched);
-    if (m->d_sched_count) cudaFree(m->d_sched_count);
-    if (m->d_tmaps) cudaFree(m->d_tmaps);
-    if (m->d_trace) cudaFree(m->d_trace);
-    if (m->ws.base) cudaFree(m->ws.base);
-    if (m->ws.h_ids) cudaFreeHost(m->ws.h_ids);
-    if (m->ws.h_logits) cudaFreeHost(m->ws.h_logits);
-    if (m->wslab) cudaFree(m->wslab);
-    if (m->wsplit) cudaFree(m->wsplit);
-    delete m;
-    return LUMEN_OK;
-}
+int lumen_llama_free(lumen_llama *m) { return lumen_model_free(m); }
 
 }  // extern "C"

@@ -16,8 +16,16 @@
 // the f32 reference to ~1e-5.  Q, K and V^T are split (and V transposed) by small kernels beforehand; rows
 // beyond the context are zero so that masked weights (exactly 0) meet finite values.
 //
+// The same kernel serves latent attention over expanded keys and values (launch_latent_prefill): Q, K and V are single bf16
+// matrices (PAIR false), a key is a block of the head's expanded part followed by the rotated part that all heads
+// share (read from the cache itself), keys and values have sizes of their own, and the head's output gate is applied
+// to the result.  The softmax weights stay a hi/lo pair there too.
+//
 // Every wait is bounded; a wait that gives up records LUMEN_ERR_TIMEOUT, the CTA leaves its loop at the next
 // block-wide barrier, lets the copies in flight land, frees its tensor memory and returns.
+#include <algorithm>
+
+#include "decoder_kernels.cuh"
 #include "tc_common.cuh"
 
 namespace lumen {
@@ -30,30 +38,39 @@ constexpr int kBKV = 64;   // cached rows per tile
 constexpr int kFaWorkers = 256;             // 8 warps: two threads per query row
 constexpr int kFaThreads = kFaWorkers + 64;  // + a warp whose first lane issues the MMAs + a warp whose first lane issues the copies
 
-template <int D>
+// KB: 64-element blocks of a query / key; DV: values of a head (padded to 64); PAIR: operands as hi/lo pairs.
+template <int KB, int DV, bool PAIR>
 struct FaGeom {
-    static constexpr int kKB = D / kBK;                      // 64-element blocks along the head dimension
+    static constexpr int kKB = KB, kParts = PAIR ? 2 : 1;
     static constexpr uint32_t kQTile = kBQ * kBK * 2;        // one (hi | lo, block) tile of Q: 128 rows of 128 bytes
-    static constexpr uint32_t kQBytes = 2 * kKB * kQTile;    // hi blocks, then lo blocks
+    static constexpr uint32_t kQBytes = kParts * kKB * kQTile;  // hi blocks, then lo blocks
     static constexpr uint32_t kKTile = kBKV * kBK * 2;       // 64 rows of 128 bytes
-    static constexpr uint32_t kKBytes = 2 * kKB * kKTile;    // hi blocks, then lo blocks
-    static constexpr uint32_t kVTile = D * kBK * 2;          // V^T: D rows of 64 cached rows
-    static constexpr uint32_t kVBytes = 2 * kVTile;          // hi, lo
+    static constexpr uint32_t kKBytes = kParts * kKB * kKTile;  // hi blocks, then lo blocks
+    static constexpr uint32_t kVTile = DV * kBK * 2;         // V^T: DV rows of 64 cached rows
+    static constexpr uint32_t kVBytes = kParts * kVTile;     // hi, lo
     static constexpr uint32_t kStageBytes = kKBytes + kVBytes;
     static constexpr uint32_t kPTile = kBQ * kBK * 2;
     static constexpr uint32_t kPBytes = 2 * kPTile;          // hi, lo
-    static constexpr int kStages = 2;
+    static constexpr int kStages = PAIR ? 2 : 3;
     static constexpr size_t kSmem = kQBytes + kStages * kStageBytes + kPBytes + 1024;  // + slack for the alignment
-    // S of even tiles: columns 0..63, S of odd tiles: 64..127, O of even tiles: 128..128+D-1, O of odd tiles after it
-    static constexpr int kTmemCols = D > 64 ? 512 : 256;
+    // S of even tiles: columns 0..63, S of odd tiles: 64..127, O of even tiles: 128..128+DV-1, O of odd tiles after it
+    static constexpr int kTmemCols = DV > 64 ? 512 : 256;
     static constexpr uint32_t kIdescS = idesc_bf16(kBQ, kBKV);
-    static constexpr uint32_t kIdescO = idesc_bf16(kBQ, D);
+    static constexpr uint32_t kIdescO = idesc_bf16(kBQ, DV);
 };
 
 struct FaParams {
-    float *out;  // [B, S, Hq, D]
+    float *out;  // [B, S, Hq, vdim] (null: not stored)
+    __nv_bfloat16 *out_hi, *out_lo;
     int S, Hq, Hkv, past, total, causal;
-    int s_pad, l_pad;  // padded extents of the split copies
+    int s_pad;  // query positions per (batch row, head) in the packed Q
+    // first row and column of a (batch row b, KV head hk) in the matrix of keys: b * k_rows_b + hk * k_rows_h, hk * k_cols_h
+    int k_rows_b, k_rows_h, k_cols_h;
+    int kb_main;           // blocks of a key from that matrix; the rest from the shared part (rows b * r_rows_b, columns from r_col0)
+    int r_rows_b, r_col0;
+    int vdim;              // values per head: rows (b * Hkv + hk) * vdim of V^T
+    const float *gate;     // gate logits gate[row * gate_ld + h] (null: no gate)
+    size_t gate_ld;
     float scale;
     DeviceStatus *status;
 };
@@ -89,13 +106,13 @@ __device__ __forceinline__ void bar_arrive(uint64_t *bar) {
 }
 
 // grid (s_pad / 128, Hq, B); 8 worker warps, warp 8 (first lane) issues the MMAs, warp 9 (first lane) the copies
-template <int D>
+template <int KB, int DV, bool PAIR>
 __global__ void __launch_bounds__(kFaThreads, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_qhi, const __grid_constant__ CUtensorMap map_qlo,
                        const __grid_constant__ CUtensorMap map_khi, const __grid_constant__ CUtensorMap map_klo,
                        const __grid_constant__ CUtensorMap map_vhi, const __grid_constant__ CUtensorMap map_vlo, const FaParams p) {
-    using G = FaGeom<D>;
-    constexpr int kKB = G::kKB, kDH = D / 2;  // a worker thread owns half a row of the context
+    using G = FaGeom<KB, DV, PAIR>;
+    constexpr int kKB = G::kKB, kDH = DV / 2;  // a worker thread owns half a row of the context
     extern __shared__ unsigned char smem_raw[];
     // the 128-byte swizzle pattern repeats every 1024 bytes: tiles must start on that boundary
     unsigned char *q_s = reinterpret_cast<unsigned char *>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -150,8 +167,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_qhi, const __grid
         if ((tid & 31) == 0) {
             // ---- TMA producer: Q once, then K and V^T of tile j + 2 as soon as tile j has released its half stage ----
             const int q_row0 = (b * p.Hq + h) * p.s_pad + i0;
-            const int k_row0 = (b * p.Hkv + hk) * p.l_pad;
-            const int v_row0 = (b * p.Hkv + hk) * D;
+            const int k_row0 = b * p.k_rows_b + hk * p.k_rows_h, k_col0 = hk * p.k_cols_h, r_row0 = b * p.r_rows_b;
+            const int v_row0 = (b * p.Hkv + hk) * p.vdim;
             // A stage holds K (hi, lo) and V^T (hi, lo) of one tile; the two halves are refilled separately: K as
             // soon as the tile's scores are done, V^T after its P.V.
             auto load_k = [&](int j) {
@@ -160,8 +177,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_qhi, const __grid
                 bar_expect(&k_full[s], G::kKBytes);
 #pragma unroll
                 for (int kb = 0; kb < kKB; ++kb) {
-                    tma_load_2d(st + kb * G::kKTile, &map_khi, kb * kBK, k_row0 + j * kBKV, &k_full[s]);
-                    tma_load_2d(st + (kKB + kb) * G::kKTile, &map_klo, kb * kBK, k_row0 + j * kBKV, &k_full[s]);
+                    if (PAIR || kb < p.kb_main)
+                        tma_load_2d(st + kb * G::kKTile, &map_khi, k_col0 + kb * kBK, k_row0 + j * kBKV, &k_full[s]);
+                    else  // (without pairs the second map of keys is the shared part)
+                        tma_load_2d(st + kb * G::kKTile, &map_klo, p.r_col0 + (kb - p.kb_main) * kBK, r_row0 + j * kBKV, &k_full[s]);
+                    if (PAIR) tma_load_2d(st + (kKB + kb) * G::kKTile, &map_klo, k_col0 + kb * kBK, k_row0 + j * kBKV, &k_full[s]);
                 }
             };
             auto load_v = [&](int j) {
@@ -169,13 +189,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_qhi, const __grid
                 unsigned char *st = ring + (size_t)s * G::kStageBytes;
                 bar_expect(&v_full[s], G::kVBytes);
                 tma_load_2d(st + G::kKBytes, &map_vhi, j * kBKV, v_row0, &v_full[s]);
-                tma_load_2d(st + G::kKBytes + G::kVTile, &map_vlo, j * kBKV, v_row0, &v_full[s]);
+                if (PAIR) tma_load_2d(st + G::kKBytes + G::kVTile, &map_vlo, j * kBKV, v_row0, &v_full[s]);
             };
             bar_expect(&q_bar, G::kQBytes);
 #pragma unroll
             for (int kb = 0; kb < kKB; ++kb) {
                 tma_load_2d(q_s + kb * G::kQTile, &map_qhi, kb * kBK, q_row0, &q_bar);
-                tma_load_2d(q_s + (kKB + kb) * G::kQTile, &map_qlo, kb * kBK, q_row0, &q_bar);
+                if (PAIR) tma_load_2d(q_s + (kKB + kb) * G::kQTile, &map_qlo, kb * kBK, q_row0, &q_bar);
             }
             for (int j = 0; j < nt && j < G::kStages; ++j) {
                 load_k(j);
@@ -209,8 +229,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_qhi, const __grid
 #pragma unroll
                         for (int kk = 0; kk < kBK / 16; ++kk) {  // UMMA K = 16 bf16 = 32 bytes = 2 descriptor units
                             umma_bf16(acc, qhi + 2 * kk, khi + 2 * kk, G::kIdescS, (kb > 0 || kk > 0) ? 1u : 0u);
-                            umma_bf16(acc, qlo + 2 * kk, khi + 2 * kk, G::kIdescS, 1u);
-                            umma_bf16(acc, qhi + 2 * kk, klo + 2 * kk, G::kIdescS, 1u);
+                            if (PAIR) {
+                                umma_bf16(acc, qlo + 2 * kk, khi + 2 * kk, G::kIdescS, 1u);
+                                umma_bf16(acc, qhi + 2 * kk, klo + 2 * kk, G::kIdescS, 1u);
+                            }
                         }
                     }
                 }
@@ -234,12 +256,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_qhi, const __grid
                     const uint32_t st = saddr(ring + (size_t)s * G::kStageBytes), pa = saddr(p_s);
                     const uint64_t phi = smem_desc(pa), plo = smem_desc(pa + G::kPTile);
                     const uint64_t vhi = smem_desc(st + G::kKBytes), vlo = smem_desc(st + G::kKBytes + G::kVTile);
-                    const uint32_t acc = tmem_o + (uint32_t)((j & 1) * D);
+                    const uint32_t acc = tmem_o + (uint32_t)((j & 1) * DV);
 #pragma unroll
                     for (int kk = 0; kk < kBKV / 16; ++kk) {
                         umma_bf16(acc, phi + 2 * kk, vhi + 2 * kk, G::kIdescO, kk > 0 ? 1u : 0u);
                         umma_bf16(acc, plo + 2 * kk, vhi + 2 * kk, G::kIdescO, 1u);
-                        umma_bf16(acc, phi + 2 * kk, vlo + 2 * kk, G::kIdescO, 1u);
+                        if (PAIR) umma_bf16(acc, phi + 2 * kk, vlo + 2 * kk, G::kIdescO, 1u);
                     }
                 }
                 // P.V of this tile has completed when these flip: the workers may read O and rewrite the weights, the
@@ -250,7 +272,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_qhi, const __grid
         }
         __syncwarp();
     } else {
-        // ---- workers: thread (row, half) owns 32 of the 64 scores of its row and D/2 of its context values ----
+        // ---- workers: thread (row, half) owns 32 of the 64 scores of its row and DV/2 of its context values ----
         const int row = tid & (kBQ - 1), half = tid >> 7, quad = warp & 3;
         const uint32_t lane_off = (uint32_t)(quad * 32) << 16;  // warps w and w + 4 read the same 32 lanes of tensor memory
         const int i_row = min(i0 + row, p.S - 1);
@@ -263,11 +285,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_qhi, const __grid
         float m = -INFINITY;
         unsigned char *prow_hi = p_s + (size_t)row * 128, *prow_lo = prow_hi + G::kPTile;
 
-        // ctx = ctx * factor + O of tile j (the accumulator of odd tiles sits D columns after that of even tiles)
+        // ctx = ctx * factor + O of tile j (the accumulator of odd tiles sits DV columns after that of even tiles)
         auto fold = [&](int j, float factor) {
             uint32_t v[kDH / 32][32];  // every load is issued before the one wait
 #pragma unroll
-            for (int q = 0; q < kDH / 32; ++q) tmem_ld32_issue(tmem_o + (uint32_t)((j & 1) * D) + lane_off + half * kDH + 32 * q, v[q]);
+            for (int q = 0; q < kDH / 32; ++q) tmem_ld32_issue(tmem_o + (uint32_t)((j & 1) * DV) + lane_off + half * kDH + 32 * q, v[q]);
             tmem_ld_wait();
 #pragma unroll
             for (int q = 0; q < kDH / 32; ++q)
@@ -358,11 +380,25 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_qhi, const __grid
             const int row = tid & (kBQ - 1), half = tid >> 7;
             if (i0 + row < p.S) {
                 const float inv = __fdiv_rn(1.0f, __fadd_rn(xch[0][row] + xch[1][row], 1e-9f));
-                float *o = p.out + (((size_t)b * p.S + (i0 + row)) * p.Hq + h) * D + half * kDH;
+                const size_t orow = (size_t)b * p.S + (i0 + row);
+                if constexpr (PAIR) {
+                    float *o = p.out + (orow * p.Hq + h) * DV + half * kDH;
 #pragma unroll
-                for (int e = 0; e < kDH; e += 4)
-                    *reinterpret_cast<float4 *>(o + e) = make_float4(__fmul_rn(ctx[e], inv), __fmul_rn(ctx[e + 1], inv),
-                                                                     __fmul_rn(ctx[e + 2], inv), __fmul_rn(ctx[e + 3], inv));
+                    for (int e = 0; e < kDH; e += 4)
+                        *reinterpret_cast<float4 *>(o + e) = make_float4(__fmul_rn(ctx[e], inv), __fmul_rn(ctx[e + 1], inv),
+                                                                         __fmul_rn(ctx[e + 2], inv), __fmul_rn(ctx[e + 3], inv));
+                } else {
+                    const float f = p.gate ? inv * sigmoid_f(p.gate[orow * p.gate_ld + h]) : inv;
+                    const size_t at = (orow * p.Hq + h) * p.vdim + half * kDH;
+                    const int n = min(kDH, p.vdim - half * kDH);
+#pragma unroll
+                    for (int e = 0; e < kDH; ++e)
+                        if (e < n) {
+                            const float v = ctx[e] * f;
+                            if (p.out) p.out[at + e] = v;
+                            if (p.out_hi) store_split(v, p.out_hi, p.out_lo, at + e);
+                        }
+                }
             }
         }
     } else if (tid == kFaWorkers + 32) {
@@ -432,15 +468,40 @@ fa_split_vt_kernel(const float *__restrict__ v_cache, __nv_bfloat16 *__restrict_
     }
 }
 
-template <int D>
+// Q of latent attention: u rows -> [B, H, s_pad, KB * 64] bf16: the unrotated part (dim numbers, zeros up to main), then the rotated
+// part, zeros elsewhere.  One thread per element.
+__global__ void fa_pack_latent_q_kernel(const LatentArgs a, __nv_bfloat16 *__restrict__ q, int s_pad, int main, int width, size_t n) {
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n) return;
+    const size_t e = i % width, row = i / width, s = row % s_pad, bh = row / s_pad, b = bh / a.H, h = bh % a.H;
+    float v = 0.f;
+    if (s < a.S) {
+        const float *src = a.u + (b * a.S + s) * a.u_ld + h * (a.dim + a.rot_dim);
+        if (e < (size_t)main) {
+            if (e < a.dim) v = src[e];
+        } else if (e - main < a.rot_dim) {
+            const size_t r = e - main;
+            v = src[a.dim + r];
+            if (r < a.rot_dims) {
+                const size_t at = (a.past + s) * (a.rot_dims / 2) + (r >> 1);
+                const float c = a.cos_t[at], sn = a.sin_t[at], w = src[a.dim + (r ^ 1)];
+                v = (r & 1) ? __fadd_rn(__fmul_rn(v, c), __fmul_rn(w, sn)) : __fsub_rn(__fmul_rn(v, c), __fmul_rn(w, sn));
+            }
+        }
+    }
+    q[i] = __float2bfloat16_rn(v);
+}
+
+template <int KB, int DV, bool PAIR>
 int launch_fa(lumen_ctx *ctx, const CUtensorMap *maps, const FaParams &p, dim3 grid, cudaStream_t s) {
+    using G = FaGeom<KB, DV, PAIR>;
     static bool attr_set[64] = {false};
     const int dev = ctx->device >= 0 && ctx->device < 64 ? ctx->device : 0;
     if (!attr_set[dev]) {
-        LUMEN_CUDA(ctx, cudaFuncSetAttribute(attn_prefill_tc_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)FaGeom<D>::kSmem));
+        LUMEN_CUDA(ctx, cudaFuncSetAttribute(attn_prefill_tc_kernel<KB, DV, PAIR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)G::kSmem));
         attr_set[dev] = true;
     }
-    attn_prefill_tc_kernel<D><<<grid, kFaThreads, FaGeom<D>::kSmem, s>>>(maps[0], maps[1], maps[2], maps[3], maps[4], maps[5], p);
+    attn_prefill_tc_kernel<KB, DV, PAIR><<<grid, kFaThreads, G::kSmem, s>>>(maps[0], maps[1], maps[2], maps[3], maps[4], maps[5], p);
     LUMEN_LAUNCHED(ctx);
     return LUMEN_OK;
 }
@@ -495,9 +556,79 @@ int launch_attn_prefill_tc(lumen_ctx *ctx, const AttnPrefillArgs &a, const float
     if (rc == LUMEN_OK) rc = make_map(ctx, &maps[4], vhi, a.B * a.Hkv * a.D, l_pad, (int)a.D);
     if (rc == LUMEN_OK) rc = make_map(ctx, &maps[5], vlo, a.B * a.Hkv * a.D, l_pad, (int)a.D);
     if (rc == LUMEN_OK) {
-        FaParams p{a.out, (int)a.S, (int)a.Hq, (int)a.Hkv, (int)a.past, (int)total, a.causal, (int)s_pad, (int)l_pad, a.scale, ctx->d_status};
+        FaParams p{};
+        p.out = a.out;
+        p.S = (int)a.S; p.Hq = (int)a.Hq; p.Hkv = (int)a.Hkv; p.past = (int)a.past; p.total = (int)total; p.causal = a.causal;
+        p.s_pad = (int)s_pad;
+        p.k_rows_b = (int)(a.Hkv * l_pad); p.k_rows_h = (int)l_pad; p.kb_main = (int)(a.D / kBK);
+        p.vdim = (int)a.D; p.scale = a.scale; p.status = ctx->d_status;
         const dim3 grid((unsigned)(s_pad / kBQ), (unsigned)a.Hq, (unsigned)a.B);
-        rc = a.D == 64 ? launch_fa<64>(ctx, maps, p, grid, s) : launch_fa<128>(ctx, maps, p, grid, s);
+        rc = a.D == 64 ? launch_fa<1, 64, true>(ctx, maps, p, grid, s) : launch_fa<2, 128, true>(ctx, maps, p, grid, s);
+    }
+    const int rc2 = dev_free(ctx, ws);
+    return rc != LUMEN_OK ? rc : rc2;
+}
+
+// Portions of at least 64 positions whose head fits two or three key blocks and 128 values; TMA wants 16-byte steps between
+// heads and rows.
+bool latent_prefill_usable(const LatentArgs &a) {
+    static const bool off = [] {
+        const char *e = getenv("LUMEN_NO_TC_ATTN");
+        return e && e[0] == '1';
+    }();
+    if (off || a.dt != LUMEN_BF16 || a.S < 64 || a.vdim > 128 || a.dim % 8 || a.rank % 8 || a.pitch % 8) return false;
+    if (!gemm_bf16_usable(a.rank, a.pitch, a.rank, a.cache, a.wuk)) return false;
+    const size_t kb = (a.dim + kBK - 1) / kBK + (a.rot_dim + kBK - 1) / kBK, total = a.past + a.S;
+    const size_t s_pad = (a.S + kBQ - 1) / kBQ * kBQ;
+    return kb <= 3 && a.B * a.H * s_pad < ((size_t)1 << 31) && a.B * a.max_seq < ((size_t)1 << 31) && a.B * a.H * a.vdim < ((size_t)1 << 31) &&
+           a.B * total < ((size_t)1 << 31) && a.B <= 65535 && a.H <= 65535;
+}
+
+// Keys and values of every head are expanded from the cached latents (two products per batch row), V directly as V^T.
+int launch_latent_prefill(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s) {
+    const size_t total = a.past + a.S, s_pad = (a.S + kBQ - 1) / kBQ * kBQ, lp = (total + 7) / 8 * 8;
+    const int kb_main = (int)((a.dim + kBK - 1) / kBK), kb_rot = (int)((a.rot_dim + kBK - 1) / kBK);
+    const int KB = std::max(2, kb_main + kb_rot), width = KB * kBK;
+    const size_t nq = a.B * a.H * s_pad * width, nk = (a.B * total * a.H * a.dim + 7) / 8 * 8, nv = a.B * a.H * a.vdim * lp;
+    void *ws = nullptr;
+    LUMEN_TRY(dev_alloc(ctx, (nq + nk + nv) * sizeof(__nv_bfloat16), &ws));
+    __nv_bfloat16 *q = static_cast<__nv_bfloat16 *>(ws), *k = q + nq, *vt = k + nk;
+    int rc = LUMEN_OK;
+    fa_pack_latent_q_kernel<<<(unsigned)((nq + 255) / 256), 256, 0, s>>>(a, q, (int)s_pad, kb_main * kBK, width, nq);
+    cudaError_t e = cudaGetLastError();
+    if (e != cudaSuccess) rc = cuda_fail(ctx, e, "fa_pack_latent_q_kernel launch");
+    else ctx->launches += 1;
+    const __nv_bfloat16 *cache = static_cast<const __nv_bfloat16 *>(a.cache);
+    for (size_t b = 0; b < a.B && rc == LUMEN_OK; ++b) {
+        const __nv_bfloat16 *latent = cache + b * a.max_seq * a.pitch;
+        GemmBf16Args g;
+        g.a_hi = latent; g.M = total; g.K = a.rank; g.lda = a.pitch;
+        g.w = static_cast<const __nv_bfloat16 *>(a.wuk); g.N = a.H * a.dim;
+        g.out16 = k + b * total * a.H * a.dim; g.ld16 = a.H * a.dim; g.epi = GemmBf16Args::kBf16;
+        rc = launch_gemm_bf16(ctx, g, s);
+        GemmBf16Args v;
+        v.a_hi = static_cast<const __nv_bfloat16 *>(a.wuv); v.M = a.H * a.vdim; v.K = a.rank;
+        v.w = latent; v.N = total; v.ldw = a.pitch;
+        v.out16 = vt + b * a.H * a.vdim * lp; v.ld16 = lp; v.epi = GemmBf16Args::kBf16;
+        if (rc == LUMEN_OK) rc = launch_gemm_bf16(ctx, v, s);
+    }
+    const bool wide = a.vdim > 64;
+    CUtensorMap maps[6];
+    if (rc == LUMEN_OK) rc = make_map(ctx, &maps[0], q, a.B * a.H * s_pad, width, kBQ);
+    if (rc == LUMEN_OK) rc = make_map(ctx, &maps[2], k, a.B * total, a.H * a.dim, kBKV);
+    if (rc == LUMEN_OK) rc = make_map(ctx, &maps[3], cache, a.B * a.max_seq, a.pitch, kBKV);
+    if (rc == LUMEN_OK) rc = make_map(ctx, &maps[4], vt, a.B * a.H * a.vdim, total, wide ? 128 : 64, lp);
+    if (rc == LUMEN_OK) {
+        maps[1] = maps[0];
+        maps[5] = maps[4];
+        FaParams p{};
+        p.out = a.out; p.out_hi = a.out_hi; p.out_lo = a.out_lo;
+        p.S = (int)a.S; p.Hq = p.Hkv = (int)a.H; p.past = (int)a.past; p.total = (int)total; p.causal = 1; p.s_pad = (int)s_pad;
+        p.k_rows_b = (int)total; p.k_cols_h = (int)a.dim; p.kb_main = kb_main; p.r_rows_b = (int)a.max_seq; p.r_col0 = (int)a.rank;
+        p.vdim = (int)a.vdim; p.gate = a.u + a.u_gate; p.gate_ld = a.u_ld; p.scale = a.scale; p.status = ctx->d_status;
+        const dim3 grid((unsigned)(s_pad / kBQ), (unsigned)a.H, (unsigned)a.B);
+        if (KB == 2) rc = wide ? launch_fa<2, 128, false>(ctx, maps, p, grid, s) : launch_fa<2, 64, false>(ctx, maps, p, grid, s);
+        else rc = wide ? launch_fa<3, 128, false>(ctx, maps, p, grid, s) : launch_fa<3, 64, false>(ctx, maps, p, grid, s);
     }
     const int rc2 = dev_free(ctx, ws);
     return rc != LUMEN_OK ? rc : rc2;

@@ -98,6 +98,10 @@ struct lumen_kv_cache {
     int *d_len = nullptr;  // device copy read by replayable kernels
     float *k = nullptr;    // [B,Hkv,max_seq,D]
     float *v = nullptr;
+    // Latent caches (models given as a list of layers): rows of d numbers of type dtype in k, no v.  The slab also holds the
+    // last token id of every batch row, shared by the layers.
+    lumen_dtype dtype = LUMEN_F32;
+    int *last_tok = nullptr;
     unsigned int seen_abort = 0;  // ctx->abort_gen at the last time `len` was known to equal *d_len
     bool owns_slab = true;  // false when carved out of a model-wide slab
     lumen_storage *slab = nullptr;  // shared slab (reference counted) when !owns_slab

@@ -1,0 +1,56 @@
+// Token inputs of the models given as a list of layers: embedding plus hashed bigram embedding, and the end of a step.
+#include "decoder_kernels.cuh"
+
+namespace lumen {
+namespace {
+
+template <typename T>
+__global__ void __launch_bounds__(256) embed_kernel(EmbedArgs a, DeviceStatus *status) {
+    const size_t m = blockIdx.x, b = m / a.S, s = m - b * a.S;
+    unsigned long long tok = id_to_index(a.ids[m]);
+    if (tok >= a.vocab) {
+        if (threadIdx.x == 0 && atomicCAS(&status->code, 0, LUMEN_ERR_EMBED_RANGE) == 0) {
+            status->detail0 = (int)m;
+            status->detail1 = (int)min(tok, 0x7fffffffull);
+        }
+        tok = 0;
+    }
+    const T *row = static_cast<const T *>(a.embed) + tok * a.dim;
+    const T *brow = nullptr;
+    if (a.bigram) {
+        unsigned long long r = a.buckets;
+        if (s > 0) r = (id_to_index(a.ids[m - 1]) * a.mul_prev + tok * a.mul_cur) % a.buckets;
+        else if (*a.d_len > 0) r = ((unsigned long long)a.last_tok[b] * a.mul_prev + tok * a.mul_cur) % a.buckets;
+        brow = static_cast<const T *>(a.bigram) + r * a.dim;
+    }
+    for (size_t i = threadIdx.x; i < a.dim; i += 256) {
+        float v = to_f32(row[i]);
+        if (brow) v = __fadd_rn(v, to_f32(brow[i]));
+        const size_t at = m * a.dim + i;
+        a.x[at] = v;
+        if (a.hi) store_split(v, a.hi, a.lo, at);
+    }
+}
+
+__global__ void advance_kernel(int *lens, int layers, const float *ids, int *last_tok, int B, int S) {
+    for (int l = threadIdx.x; l < layers; l += blockDim.x) lens[l] += S;
+    for (int b = threadIdx.x; b < B; b += blockDim.x) last_tok[b] = (int)id_to_index(ids[(size_t)b * S + S - 1]);
+}
+
+}  // namespace
+
+int launch_embed(lumen_ctx *ctx, const EmbedArgs &a, cudaStream_t s) {
+    const unsigned rows = (unsigned)(a.B * a.S);
+    if (a.dt == LUMEN_F32) embed_kernel<float><<<rows, 256, 0, s>>>(a, ctx->d_status);
+    else embed_kernel<__nv_bfloat16><<<rows, 256, 0, s>>>(a, ctx->d_status);
+    LUMEN_LAUNCHED(ctx);
+    return LUMEN_OK;
+}
+
+int launch_advance(lumen_ctx *ctx, int *d_lens, size_t layers, const float *ids, int *last_tok, size_t B, size_t S, cudaStream_t s) {
+    advance_kernel<<<1, 256, 0, s>>>(d_lens, (int)layers, ids, last_tok, (int)B, (int)S);
+    LUMEN_LAUNCHED(ctx);
+    return LUMEN_OK;
+}
+
+}  // namespace lumen

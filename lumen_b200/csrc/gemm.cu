@@ -6,7 +6,7 @@
 // vector-matrix kernel when the weights are f32 (bf16 weights are widened on load).
 #include <algorithm>
 
-#include "common.cuh"
+#include "decoder_kernels.cuh"
 
 namespace lumen {
 namespace {
@@ -79,6 +79,14 @@ int launch_gemm_nk(lumen_ctx *ctx, const float *a, const void *w, lumen_dtype wd
                    size_t N, const float *residual, cudaStream_t s, const TpSumArgs *tp) {
     if (M == 0 || N == 0) return LUMEN_OK;
     if (gemm_tc_usable(wdt, M, K, N, w)) return launch_gemm_tc(ctx, a, w, wdt, c, M, K, N, residual, s, tp);
+    LUMEN_TRY(launch_gemm_simt(ctx, a, w, wdt, c, M, K, N, residual, s));
+    if (tp) return launch_tp_sum(ctx, c, 1, nullptr, M, N, *tp, s);
+    return LUMEN_OK;
+}
+
+int launch_gemm_simt(lumen_ctx *ctx, const float *a, const void *w, lumen_dtype wdt, float *c, size_t M, size_t K, size_t N,
+                     const float *residual, cudaStream_t s) {
+    if (M == 0 || N == 0) return LUMEN_OK;
     dim3 grid((unsigned)((N + BN - 1) / BN), (unsigned)((M + BM - 1) / BM));
     if (wdt == LUMEN_F32)
         gemm_nk_kernel<float><<<grid, kThreads, 0, s>>>(a, static_cast<const float *>(w), c, M, K, N, residual);
@@ -86,7 +94,6 @@ int launch_gemm_nk(lumen_ctx *ctx, const float *a, const void *w, lumen_dtype wd
         gemm_nk_kernel<__nv_bfloat16>
             <<<grid, kThreads, 0, s>>>(a, static_cast<const __nv_bfloat16 *>(w), c, M, K, N, residual);
     LUMEN_LAUNCHED(ctx);
-    if (tp) return launch_tp_sum(ctx, c, 1, nullptr, M, N, *tp, s);
     return LUMEN_OK;
 }
 

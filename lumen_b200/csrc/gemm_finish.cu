@@ -7,6 +7,7 @@
 //                          over the concatenated gate and up weights (replaces two split-K sums + SiLU*mul + hi/lo split)
 #include <algorithm>
 
+#include "decoder_kernels.cuh"
 #include "row_finish.cuh"
 
 namespace lumen {
@@ -53,7 +54,79 @@ __global__ void __launch_bounds__(256) sum_swiglu_split_kernel(const float *__re
     *reinterpret_cast<uint2 *>(lo + row * inter + col) = l;
 }
 
+// One CTA per row, any row length (the row is kept in shared memory between the two passes).
+__global__ void __launch_bounds__(256) norm_add_kernel(const float *__restrict__ part, int splits, size_t rows, size_t n, const StepFinish f) {
+    extern __shared__ float row_s[];
+    __shared__ float red[8];
+    const int tid = threadIdx.x;
+    const size_t row = blockIdx.x, base = row * n, mn = rows * n;
+    float ss = 0.f;
+    for (size_t i = tid; i < n; i += 256) {
+        float v = 0.f;
+        for (int sl = 0; sl < splits; ++sl) v = __fadd_rn(v, part[(size_t)sl * mn + base + i]);
+        for (int k = 0; k < f.gather_n; ++k) v = __fadd_rn(v, f.gather_src[(size_t)f.gather_idx[row * f.gather_n + k] * n + i]);
+        if (f.extra) v = __fadd_rn(v, f.extra[base + i]);
+        row_s[i] = v;
+        ss = fmaf(v, v, ss);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if ((tid & 31) == 0) red[tid >> 5] = ss;
+    __syncthreads();
+    float t = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) t += red[w];
+    const float inv = __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(t, (float)n), f.eps)));
+    for (size_t i = tid; i < n; i += 256) {
+        const float x = __fadd_rn(f.x[base + i], __fmul_rn(__fmul_rn(row_s[i], inv), f.gain[i]));
+        f.x[base + i] = x;
+        if (f.hi) store_split(x, f.hi, f.lo, base + i);
+    }
+}
+
+// One thread per output element.
+__global__ void __launch_bounds__(256) act_finish_kernel(const float *__restrict__ part, int splits, size_t rows, size_t n, const StepFinish f) {
+    const size_t out_n = f.kind == StepFinish::kGated ? f.ff : n;
+    const size_t i = (size_t)blockIdx.x * 256 + threadIdx.x;
+    if (i >= rows * out_n) return;
+    const size_t row = i / out_n, col = i - row * out_n, mn = rows * n;
+    auto sum = [&](size_t c) {
+        float v = part[row * n + c];
+        for (int sl = 1; sl < splits; ++sl) v = __fadd_rn(v, part[(size_t)sl * mn + row * n + c]);
+        return v;
+    };
+    float v;
+    if (f.kind == StepFinish::kGated) {
+        const size_t at = col / kGateBlock * (2 * kGateBlock) + col % kGateBlock;
+        v = gated_act(sum(at), sum(at + kGateBlock), f.limit);
+    } else {
+        v = sum(col);
+        if (f.kind != StepFinish::kStore) v = gelu_tanh(v);
+        if (f.kind == StepFinish::kSideGate) {
+            const unsigned long long tok = id_to_index(f.ids[row]);
+            v *= tok < f.table_rows ? table_at(f.table, f.table_dt, tok * f.table_ld + col) : 0.f;
+        }
+    }
+    if (f.out) f.out[i] = v;
+    if (f.hi) store_split(v, f.hi, f.lo, i);
+}
+
 }  // namespace
+
+int launch_step_finish(lumen_ctx *ctx, const float *part, int splits, size_t rows, size_t n, const StepFinish &f, cudaStream_t s) {
+    if (rows == 0 || n == 0) return LUMEN_OK;
+    if (f.kind == StepFinish::kNormAdd) {
+        const size_t smem = n * sizeof(float);
+        if (smem > 200 * 1024) return set_error(ctx, LUMEN_ERR_UNSUPPORTED, "row finisher: row length %zu", n);
+        if (smem > 48 * 1024) LUMEN_CUDA(ctx, cudaFuncSetAttribute(norm_add_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        norm_add_kernel<<<(unsigned)rows, 256, smem, s>>>(part, part ? splits : 0, rows, n, f);
+    } else {
+        const size_t total = rows * (f.kind == StepFinish::kGated ? f.ff : n);
+        act_finish_kernel<<<(unsigned)((total + 255) / 256), 256, 0, s>>>(part, splits, rows, n, f);
+    }
+    LUMEN_LAUNCHED(ctx);
+    return LUMEN_OK;
+}
 
 bool row_finish_usable(size_t dim) { return dim % 8 == 0 && dim <= (size_t)kRowVecs * 1024; }
 

@@ -19,6 +19,7 @@
 // copies in flight land, frees its tensor memory and returns.
 #include <algorithm>
 
+#include "decoder_kernels.cuh"
 #include "tc_common.cuh"
 
 namespace lumen {
@@ -51,9 +52,36 @@ struct TcParams {
     int M, N, K;
     int kb_per_split;       // 64-element K blocks per blockIdx.z
     DeviceStatus *status;
+    // bf16 epilogues and grouped products (launch_gemm_bf16)
+    __nv_bfloat16 *out16;
+    size_t ld16;
+    const int4 *tiles;
+    const int *n_tiles;
+    const float *row_scale;
+    float limit;
+    int ff;
 };
 
-template <int NA, int NB, int BN, bool SWAP>
+// Eight values of one output row as bf16 (one 16-byte store when the row allows it).
+__device__ __forceinline__ void store8_bf16(__nv_bfloat16 *dst, const float (&x)[8], int n, bool vec) {
+    if (vec && n >= 8) {
+        uint4 v;
+        uint32_t *u = &v.x;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const __nv_bfloat162 p = __floats2bfloat162_rn(x[2 * j], x[2 * j + 1]);
+            u[j] = *reinterpret_cast<const uint32_t *>(&p);
+        }
+        *reinterpret_cast<uint4 *>(dst) = v;
+    } else {
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+            if (j < n) dst[j] = __float2bfloat16_rn(x[j]);
+    }
+}
+
+// EPI: GemmBf16Args::Epi.  GROUPED: blockIdx.y is a tile of p.tiles instead of a row block.
+template <int NA, int NB, int BN, bool SWAP, int EPI = 0, bool GROUPED = false>
 __global__ void __launch_bounds__(kTcThreads, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid_constant__ CUtensorMap map_alo,
                const __grid_constant__ CUtensorMap map_b, const __grid_constant__ CUtensorMap map_blo, const TcParams p) {
@@ -68,7 +96,15 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid_constan
     __shared__ int failed;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     // first row of this CTA's tile on the 128-row side and on the BN-row side (blockIdx.x walks the weight rows)
-    const int a0 = (SWAP ? blockIdx.x : blockIdx.y) * kBM, b0 = (SWAP ? blockIdx.y : blockIdx.x) * kBN;
+    int a0 = (SWAP ? blockIdx.x : blockIdx.y) * kBM, b_load = (SWAP ? blockIdx.y : blockIdx.x) * kBN, a_end = p.M;
+    const int b0 = b_load;
+    if (GROUPED) {
+        if ((int)blockIdx.y >= *p.n_tiles) return;
+        const int4 t = p.tiles[blockIdx.y];
+        a0 = t.x;
+        a_end = t.y;
+        b_load += t.z * p.N;
+    }
     // This CTA's range of 64-element K blocks: all of them, or slice blockIdx.z when K is split over the grid
     // (few output tiles and a long K: more CTAs stream the weights).  kb below counts from the slice's start.
     const int kb_all = (p.K + kBK - 1) / kBK;
@@ -106,8 +142,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid_constan
             const int kx = (kb0 + kb) * kBK;
             tma_load_2d(st, &map_ahi, kx, a0, &full[s]);
             if (NA == 2) tma_load_2d(st + kABytes, &map_alo, kx, a0, &full[s]);
-            tma_load_2d(st + NA * kABytes, &map_b, kx, b0, &full[s]);
-            if (NB == 2) tma_load_2d(st + NA * kABytes + kBBytes, &map_blo, kx, b0, &full[s]);
+            tma_load_2d(st + NA * kABytes, &map_b, kx, b_load, &full[s]);
+            if (NB == 2) tma_load_2d(st + NA * kABytes + kBBytes, &map_blo, kx, b_load, &full[s]);
         }
     } else if (tid == 32) {
         // ---- MMA issuer ----
@@ -139,6 +175,50 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid_constan
     if (have && !failed) {
         const int arow = a0 + warp * 32 + lane;  // this thread's row of the tile's 128-row side
         const bool empty_slice = nkb == 0;       // nothing was accumulated: the tile's contribution is zero
+        if constexpr (EPI == GemmBf16Args::kGated) {
+            // columns 0 .. 63 of the tile are gates, 64 .. 127 the ups that go with them: 64 columns of output
+            const float scale = p.row_scale && arow < a_end ? p.row_scale[arow] : 1.f;
+            const bool vec = (p.ld16 & 7) == 0;
+#pragma unroll 1
+            for (int c0 = 0; c0 < 64; c0 += 32) {
+                uint32_t g[32], u[32];
+                const uint32_t taddr = tmem_base + ((uint32_t)(warp * 32) << 16) + (uint32_t)c0;
+                tmem_ld32_issue(taddr, g);
+                tmem_ld32_issue(taddr + 64, u);
+                tmem_ld_wait();
+                if (arow < a_end) {
+                    const int col = b0 / 2 + c0;
+                    __nv_bfloat16 *dst = p.out16 + (size_t)arow * p.ld16 + col;
+#pragma unroll
+                    for (int j = 0; j < 32; j += 8) {
+                        float x[8];
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) x[i] = gated_act(__uint_as_float(g[j + i]) * scale, __uint_as_float(u[j + i]) * scale, p.limit);
+                        if (col + j < p.ff) store8_bf16(dst + j, x, p.ff - (col + j), vec);
+                    }
+                }
+            }
+        } else if constexpr (EPI == GemmBf16Args::kBf16 || EPI == GemmBf16Args::kGelu) {
+            const bool vec = (p.ld16 & 7) == 0;
+#pragma unroll 1
+            for (int c0 = 0; c0 < kBN; c0 += 32) {
+                uint32_t v[32];
+                tmem_ld32(tmem_base + ((uint32_t)(warp * 32) << 16) + (uint32_t)c0, v);
+                if (arow < a_end) {
+                    __nv_bfloat16 *dst = p.out16 + (size_t)arow * p.ld16 + b0 + c0;
+#pragma unroll
+                    for (int j = 0; j < 32; j += 8) {
+                        float x[8];
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) {
+                            x[i] = __uint_as_float(v[j + i]);
+                            if (EPI == GemmBf16Args::kGelu) x[i] = gelu_tanh(x[i]);
+                        }
+                        if (b0 + c0 + j < p.N) store8_bf16(dst + j, x, p.N - (b0 + c0 + j), vec);
+                    }
+                }
+            }
+        } else {
         float *cbase = p.c + (size_t)blockIdx.z * p.M * p.N;
 #pragma unroll 1
         for (int c0 = 0; c0 < kBN; c0 += 32) {
@@ -146,7 +226,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid_constan
             const uint32_t taddr = tmem_base + ((uint32_t)(warp * 32) << 16) + (uint32_t)c0;
             tmem_ld32(taddr, v);
             if (!SWAP) {
-                if (arow < p.M) {  // output row arow, columns b0 + c0 ..
+                if (arow < a_end) {  // output row arow, columns b0 + c0 ..
                     float *crow = cbase + (size_t)arow * p.N + b0 + c0;
                     const float *rrow = p.residual ? p.residual + (size_t)arow * p.N + b0 + c0 : nullptr;
 #pragma unroll
@@ -169,6 +249,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid_constan
                     }
                 }
             }
+        }
         }
     } else if (tid == 0) {
         // A wait gave up: let the copies that are still in flight land before the CTA exits (bounded).
@@ -216,22 +297,22 @@ bool gemm_tc_usable(lumen_dtype wdt, size_t M, size_t K, size_t N, const void *w
 
 namespace {
 
-template <int NA, int NB, int BN, bool SWAP>
+template <int NA, int NB, int BN, bool SWAP, int EPI = 0, bool GROUPED = false>
 int launch_tc_kernel(lumen_ctx *ctx, const CUtensorMap &mhi, const CUtensorMap &mlo, const CUtensorMap &mb, const CUtensorMap &mblo,
-                     const TcParams &p, size_t M, size_t N, cudaStream_t s) {
+                     const TcParams &p, size_t M, size_t N, cudaStream_t s, size_t row_tiles = 0) {
     using Geom = TcGeom<NA, NB, BN>;
     constexpr size_t smem = (size_t)Geom::kStages * Geom::kStageBytes + 1024;  // + slack for the alignment
     static bool attr_set[64] = {false};
     const int dev = ctx->device >= 0 && ctx->device < 64 ? ctx->device : 0;
     if (!attr_set[dev]) {
-        LUMEN_CUDA(ctx, cudaFuncSetAttribute(gemm_tc_kernel<NA, NB, BN, SWAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        LUMEN_CUDA(ctx, cudaFuncSetAttribute(gemm_tc_kernel<NA, NB, BN, SWAP, EPI, GROUPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         attr_set[dev] = true;
     }
     const int kb_all = (p.K + kBK - 1) / kBK;
     const int splits = (kb_all + p.kb_per_split - 1) / p.kb_per_split;
     const dim3 grid = SWAP ? dim3((unsigned)((N + kBM - 1) / kBM), (unsigned)((M + BN - 1) / BN), (unsigned)splits)
-                           : dim3((unsigned)((N + BN - 1) / BN), (unsigned)((M + kBM - 1) / kBM), (unsigned)splits);
-    gemm_tc_kernel<NA, NB, BN, SWAP><<<grid, kTcThreads, smem, s>>>(mhi, mlo, mb, mblo, p);
+                           : dim3((unsigned)((N + BN - 1) / BN), (unsigned)(GROUPED ? row_tiles : (M + kBM - 1) / kBM), (unsigned)splits);
+    gemm_tc_kernel<NA, NB, BN, SWAP, EPI, GROUPED><<<grid, kTcThreads, smem, s>>>(mhi, mlo, mb, mblo, p);
     LUMEN_LAUNCHED(ctx);
     return LUMEN_OK;
 }
@@ -317,8 +398,12 @@ int launch_gemm_tc(lumen_ctx *ctx, const float *a, const void *w, lumen_dtype wd
     void *partial = nullptr;
     if (rc == LUMEN_OK && splits > 1) rc = dev_alloc(ctx, (size_t)splits * M * N * sizeof(float), &partial);
     if (rc == LUMEN_OK) {
-        TcParams p{splits > 1 ? static_cast<float *>(partial) : c, splits > 1 ? nullptr : residual, (int)M, (int)N, (int)K,
-                   kb_per_split, ctx->d_status};
+        TcParams p{};
+        p.c = splits > 1 ? static_cast<float *>(partial) : c;
+        p.residual = splits > 1 ? nullptr : residual;
+        p.M = (int)M; p.N = (int)N; p.K = (int)K;
+        p.kb_per_split = kb_per_split;
+        p.status = ctx->d_status;
 #define LUMEN_TC(NA_, NB_, BN_, SW_) launch_tc_kernel<NA_, NB_, BN_, SW_>(ctx, map_hi, map_lo, map_b, map_blo, p, M, N, s)
         if (swap) rc = wsplit ? LUMEN_TC(2, 2, 64, true) : LUMEN_TC(1, 2, 64, true);
         else if (wsplit) rc = bn == 128 ? LUMEN_TC(2, 2, 128, false) : bn == 64 ? LUMEN_TC(2, 2, 64, false) : LUMEN_TC(2, 2, 32, false);
@@ -350,6 +435,77 @@ int launch_gemm_tc(lumen_ctx *ctx, const float *a, const void *w, lumen_dtype wd
         if (rc == LUMEN_OK) rc = rc3;
     }
     int rc2 = dev_free(ctx, split);
+    return rc != LUMEN_OK ? rc : rc2;
+}
+
+// ---- bf16 operands ------------------------------------------------------------------------------
+bool gemm_bf16_usable(size_t K, size_t lda, size_t ldw, const void *a, const void *w) {
+    if (!gemm_tc_usable(LUMEN_BF16, 2, K, 8, w)) return false;
+    return (lda ? lda : K) % 8 == 0 && (ldw ? ldw : K) % 8 == 0 && (reinterpret_cast<uintptr_t>(a) & 15) == 0;
+}
+
+int launch_gemm_bf16(lumen_ctx *ctx, const GemmBf16Args &g, cudaStream_t s) {
+    if (g.M == 0 || g.N == 0) return LUMEN_OK;
+    const size_t lda = g.lda ? g.lda : g.K, ldw = g.ldw ? g.ldw : g.K;
+    const bool pair = g.a_lo != nullptr, grouped = g.tiles != nullptr;
+    if (!gemm_bf16_usable(g.K, lda, ldw, g.a_hi, g.w) || (pair && g.epi != GemmBf16Args::kF32) || g.M > 0x7fffffff || g.N * g.w_groups > 0x7fffffff)
+        return set_error(ctx, LUMEN_ERR_UNSUPPORTED, "tensor-core product: %zu x %zu x %zu", g.M, g.N, g.K);
+    TcParams p{};
+    p.c = g.c; p.M = (int)g.M; p.N = (int)g.N; p.K = (int)g.K; p.status = ctx->d_status;
+    p.out16 = g.out16; p.ld16 = g.ld16; p.tiles = g.tiles; p.n_tiles = g.n_tiles; p.row_scale = g.row_scale; p.limit = g.limit;
+    p.ff = (int)g.ff;
+    const int kb_all = (int)((g.K + kBK - 1) / kBK);
+    p.kb_per_split = kb_all;
+    const bool swap = g.M <= 64 && g.epi == GemmBf16Args::kF32 && !grouped;
+    const int bn = swap ? 64 : g.epi == GemmBf16Args::kGated || grouped ? 128 : pick_bn(g.M, g.N, ctx->num_sms);
+    int splits = 1;
+    void *partial = nullptr;
+    if (g.epi == GemmBf16Args::kF32 && !grouped && g.M <= (size_t)kBM) {
+        const int tiles = (int)((g.N + (swap ? kBM : bn) - 1) / (swap ? kBM : bn));
+        splits = std::max(1, std::min(std::min(ctx->num_sms / std::max(tiles, 1), kb_all / 4), 16));
+        p.kb_per_split = (kb_all + splits - 1) / splits;
+        splits = (kb_all + p.kb_per_split - 1) / p.kb_per_split;
+        if (splits > 1) {
+            LUMEN_TRY(dev_alloc(ctx, (size_t)splits * g.M * g.N * sizeof(float), &partial));
+            p.c = static_cast<float *>(partial);
+        }
+    }
+    CUtensorMap ma, ma2, mb, mb2;
+    const __nv_bfloat16 *lo = pair ? g.a_lo : g.a_hi;
+    int rc;
+    if (swap) {
+        rc = make_map(ctx, &ma, g.w, g.N, g.K, kBM, ldw);
+        ma2 = ma;
+        if (rc == LUMEN_OK) rc = make_map(ctx, &mb, g.a_hi, g.M, g.K, bn, lda);
+        if (rc == LUMEN_OK) rc = make_map(ctx, &mb2, lo, g.M, g.K, bn, lda);
+    } else {
+        rc = make_map(ctx, &ma, g.a_hi, g.M, g.K, kBM, lda);
+        if (rc == LUMEN_OK) rc = make_map(ctx, &ma2, lo, g.M, g.K, kBM, lda);
+        if (rc == LUMEN_OK) rc = make_map(ctx, &mb, g.w, g.N * g.w_groups, g.K, bn, ldw);
+        mb2 = mb;
+    }
+#define LUMEN_TC(NA_, NB_, BN_, SW_, EPI_, GR_) launch_tc_kernel<NA_, NB_, BN_, SW_, EPI_, GR_>(ctx, ma, ma2, mb, mb2, p, g.M, g.N, s, g.max_tiles)
+    if (rc == LUMEN_OK) {
+        if (grouped) rc = g.epi == GemmBf16Args::kGated ? LUMEN_TC(1, 1, 128, false, 3, true) : LUMEN_TC(1, 1, 128, false, 0, true);
+        else if (swap) rc = pair ? LUMEN_TC(1, 2, 64, true, 0, false) : LUMEN_TC(1, 1, 64, true, 0, false);
+        else if (g.epi == GemmBf16Args::kGated) rc = LUMEN_TC(1, 1, 128, false, 3, false);
+        else if (g.epi == GemmBf16Args::kGelu) rc = bn == 128 ? LUMEN_TC(1, 1, 128, false, 2, false) : bn == 64 ? LUMEN_TC(1, 1, 64, false, 2, false) : LUMEN_TC(1, 1, 32, false, 2, false);
+        else if (g.epi == GemmBf16Args::kBf16) rc = bn == 128 ? LUMEN_TC(1, 1, 128, false, 1, false) : bn == 64 ? LUMEN_TC(1, 1, 64, false, 1, false) : LUMEN_TC(1, 1, 32, false, 1, false);
+        else if (pair) rc = bn == 128 ? LUMEN_TC(2, 1, 128, false, 0, false) : bn == 64 ? LUMEN_TC(2, 1, 64, false, 0, false) : LUMEN_TC(2, 1, 32, false, 0, false);
+        else rc = bn == 128 ? LUMEN_TC(1, 1, 128, false, 0, false) : bn == 64 ? LUMEN_TC(1, 1, 64, false, 0, false) : LUMEN_TC(1, 1, 32, false, 0, false);
+    }
+#undef LUMEN_TC
+    if (rc == LUMEN_OK && g.epi == GemmBf16Args::kF32) {
+        if (g.fin) rc = launch_step_finish(ctx, p.c, splits, g.M, g.N, *g.fin, s);
+        else if (splits > 1) {
+            const size_t mn = g.M * g.N;
+            splitk_reduce_kernel<<<(unsigned)((mn + 255) / 256), 256, 0, s>>>(p.c, nullptr, g.c, mn, splits);
+            cudaError_t e = cudaGetLastError();
+            if (e != cudaSuccess) rc = cuda_fail(ctx, e, "splitk_reduce_kernel launch");
+            else ctx->launches += 1;
+        }
+    }
+    const int rc2 = dev_free(ctx, partial);
     return rc != LUMEN_OK ? rc : rc2;
 }
 

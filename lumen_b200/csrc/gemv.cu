@@ -10,25 +10,14 @@
 // shared memory and read back as conflict-free 128-bit words.
 #include <algorithm>
 
-#include "common.cuh"
+#include "decoder_kernels.cuh"
+#include "gemv_rows.cuh"
 
 namespace lumen {
 namespace {
 
 constexpr int kThreads = 256;
 constexpr int kWarps = kThreads / 32;
-
-__device__ __forceinline__ float warp_sum(float v) {
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-    return v;
-}
-
-__device__ __forceinline__ float4 ld_stream_f4(const float4 *p) { return __ldcs(p); }
-__device__ __forceinline__ uint4 ld_stream_u4(const uint4 *p) { return __ldcs(p); }
-
-__device__ __forceinline__ float bf16_lo(uint32_t u) { return __uint_as_float(u << 16); }
-__device__ __forceinline__ float bf16_hi(uint32_t u) { return __uint_as_float(u & 0xffff0000u); }
 
 // Stage x[M,K] into shared memory, optionally RMS-normalised: xs = (x * inv_rms) * norm_w, which is
 // the element the reference's RMSNorm produces (src/layers/norm/rms_norm.rs:49-56) before its Linear.
@@ -67,139 +56,6 @@ __device__ void stage_x(float *xs, const float *__restrict__ x, int M, size_t K,
         }
     }
     __syncthreads();
-}
-
-// Accumulate one row (`wrow`, K elements) against MB staged vectors.  Vector path needs K % VEC == 0
-// and a 16-byte aligned row; otherwise the scalar path runs.
-template <typename WT, int MB>
-__device__ __forceinline__ void row_dot(const WT *__restrict__ wrow, const float *xs, size_t K, int lane, bool vec_ok,
-                                        float (&acc)[MB]) {
-    constexpr int kUnroll = 8;
-    if constexpr (sizeof(WT) == 4) {
-        if (vec_ok) {
-            const float4 *w4 = reinterpret_cast<const float4 *>(wrow);
-            const size_t n4 = K / 4;
-            for (size_t base = 0; base < n4; base += 32 * kUnroll) {
-                float4 wv[kUnroll];
-#pragma unroll
-                for (int u = 0; u < kUnroll; ++u) {
-                    size_t i = base + (size_t)u * 32 + lane;
-                    wv[u] = (i < n4) ? ld_stream_f4(w4 + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-                }
-#pragma unroll
-                for (int u = 0; u < kUnroll; ++u) {
-                    size_t i = base + (size_t)u * 32 + lane;
-                    if (i < n4) {
-#pragma unroll
-                        for (int m = 0; m < MB; ++m) {
-                            float4 xv = *reinterpret_cast<const float4 *>(xs + (size_t)m * K + i * 4);
-                            acc[m] = fmaf(wv[u].x, xv.x, acc[m]);
-                            acc[m] = fmaf(wv[u].y, xv.y, acc[m]);
-                            acc[m] = fmaf(wv[u].z, xv.z, acc[m]);
-                            acc[m] = fmaf(wv[u].w, xv.w, acc[m]);
-                        }
-                    }
-                }
-            }
-            return;
-        }
-        for (size_t k = lane; k < K; k += 32) {
-            float w = reinterpret_cast<const float *>(wrow)[k];
-#pragma unroll
-            for (int m = 0; m < MB; ++m) acc[m] = fmaf(w, xs[(size_t)m * K + k], acc[m]);
-        }
-    } else {
-        if (vec_ok) {
-            const uint4 *w8 = reinterpret_cast<const uint4 *>(wrow);
-            const size_t n8 = K / 8;
-            for (size_t base = 0; base < n8; base += 32 * kUnroll) {
-                uint4 wv[kUnroll];
-#pragma unroll
-                for (int u = 0; u < kUnroll; ++u) {
-                    size_t i = base + (size_t)u * 32 + lane;
-                    wv[u] = (i < n8) ? ld_stream_u4(w8 + i) : make_uint4(0u, 0u, 0u, 0u);
-                }
-#pragma unroll
-                for (int u = 0; u < kUnroll; ++u) {
-                    size_t i = base + (size_t)u * 32 + lane;
-                    if (i < n8) {
-#pragma unroll
-                        for (int m = 0; m < MB; ++m) {
-                            const float4 *xp = reinterpret_cast<const float4 *>(xs + (size_t)m * K + i * 8);
-                            float4 x0 = xp[0], x1 = xp[1];
-                            acc[m] = fmaf(bf16_lo(wv[u].x), x0.x, acc[m]);
-                            acc[m] = fmaf(bf16_hi(wv[u].x), x0.y, acc[m]);
-                            acc[m] = fmaf(bf16_lo(wv[u].y), x0.z, acc[m]);
-                            acc[m] = fmaf(bf16_hi(wv[u].y), x0.w, acc[m]);
-                            acc[m] = fmaf(bf16_lo(wv[u].z), x1.x, acc[m]);
-                            acc[m] = fmaf(bf16_hi(wv[u].z), x1.y, acc[m]);
-                            acc[m] = fmaf(bf16_lo(wv[u].w), x1.z, acc[m]);
-                            acc[m] = fmaf(bf16_hi(wv[u].w), x1.w, acc[m]);
-                        }
-                    }
-                }
-            }
-            return;
-        }
-        for (size_t k = lane; k < K; k += 32) {
-            float w = __bfloat162float(reinterpret_cast<const __nv_bfloat16 *>(wrow)[k]);
-#pragma unroll
-            for (int m = 0; m < MB; ++m) acc[m] = fmaf(w, xs[(size_t)m * K + k], acc[m]);
-        }
-    }
-}
-
-// RR rows of W against MB staged vectors at once: every 16 bytes of x read from shared memory feed RR rows, so
-// the shared-memory traffic per weight byte is MB / RR instead of MB (with MB = 8 and one row at a time the
-// kernel was bound by shared memory, not by HBM).  Vector path only (K % VEC == 0, 16-byte aligned rows).
-template <typename WT, int MB, int RR>
-__device__ __forceinline__ void rows_dot(const WT *const (&rows)[RR], const float *xs, size_t K, int lane, float (&acc)[RR][MB]) {
-    constexpr int VEC = 16 / sizeof(WT);
-    constexpr int kUnroll = 4;
-    const size_t nv = K / VEC;
-    for (size_t base = 0; base < nv; base += 32 * kUnroll) {
-        uint4 wv[RR][kUnroll];
-#pragma unroll
-        for (int u = 0; u < kUnroll; ++u) {
-            const size_t i = base + (size_t)u * 32 + lane;
-#pragma unroll
-            for (int r = 0; r < RR; ++r)
-                wv[r][u] = (i < nv) ? ld_stream_u4(reinterpret_cast<const uint4 *>(rows[r]) + i) : make_uint4(0u, 0u, 0u, 0u);
-        }
-#pragma unroll
-        for (int u = 0; u < kUnroll; ++u) {
-            const size_t i = base + (size_t)u * 32 + lane;
-            if (i < nv) {
-#pragma unroll
-                for (int m = 0; m < MB; ++m) {
-                    const float4 *xp = reinterpret_cast<const float4 *>(xs + (size_t)m * K + i * VEC);
-                    const float4 x0 = xp[0];
-                    if constexpr (sizeof(WT) == 4) {
-#pragma unroll
-                        for (int r = 0; r < RR; ++r) {
-                            acc[r][m] = fmaf(__uint_as_float(wv[r][u].x), x0.x, acc[r][m]);
-                            acc[r][m] = fmaf(__uint_as_float(wv[r][u].y), x0.y, acc[r][m]);
-                            acc[r][m] = fmaf(__uint_as_float(wv[r][u].z), x0.z, acc[r][m]);
-                            acc[r][m] = fmaf(__uint_as_float(wv[r][u].w), x0.w, acc[r][m]);
-                        }
-                    } else {
-                        const float4 x1 = xp[1];
-#pragma unroll
-                        for (int r = 0; r < RR; ++r) {
-                            acc[r][m] = fmaf(bf16_lo(wv[r][u].x), x0.x, acc[r][m]);
-                            acc[r][m] = fmaf(bf16_hi(wv[r][u].x), x0.y, acc[r][m]);
-                            acc[r][m] = fmaf(bf16_lo(wv[r][u].y), x0.z, acc[r][m]);
-                            acc[r][m] = fmaf(bf16_hi(wv[r][u].y), x0.w, acc[r][m]);
-                            acc[r][m] = fmaf(bf16_lo(wv[r][u].z), x1.x, acc[r][m]);
-                            acc[r][m] = fmaf(bf16_hi(wv[r][u].z), x1.y, acc[r][m]);
-                            acc[r][m] = fmaf(bf16_lo(wv[r][u].w), x1.z, acc[r][m]);
-                            acc[r][m] = fmaf(bf16_hi(wv[r][u].w), x1.w, acc[r][m]);
-                        }
-                    }
-                }
-            }
-        }
-    }
 }
 
 template <typename WT, int MB>
@@ -308,6 +164,66 @@ gemv_gate_up_kernel(const float *__restrict__ x, const WT *__restrict__ wg, cons
                 float sig = __fdiv_rn(1.0f, __fadd_rn(1.0f, expf(-g)));
                 out[(size_t)m * I + row] = __fmul_rn(__fmul_rn(g, sig), u);
             }
+        }
+    }
+}
+
+// One row whose input may still owe the norm of a sublayer's output (post-norm models): x = res + RMSNorm(y) * gain is
+// formed by every CTA while it stages x, so that the norm, the residual sum and the product are one launch.
+template <typename WT>
+__global__ void __launch_bounds__(kThreads) gemv_step_kernel(const GemvStepArgs a) {
+    extern __shared__ __align__(16) float smem[];
+    __shared__ float red[kWarps];
+    float *xs = smem;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const size_t K = a.K;
+    auto inv_rms = [&](float ss) {
+        ss = warp_sum(ss);
+        if (lane == 0) red[warp] = ss;
+        __syncthreads();
+        float t = 0.f;
+#pragma unroll
+        for (int w = 0; w < kWarps; ++w) t += red[w];
+        __syncthreads();
+        return __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(t, (float)K), a.eps)));
+    };
+    if (a.y) {
+        float ss = 0.f;
+        for (size_t k = tid; k < K; k += kThreads) {
+            const float v = a.y[k];
+            xs[k] = v;
+            ss = fmaf(v, v, ss);
+        }
+        const float inv = inv_rms(ss);
+        for (size_t k = tid; k < K; k += kThreads) {
+            const float x = __fadd_rn(a.res[k], __fmul_rn(__fmul_rn(xs[k], inv), a.gain[k]));
+            xs[k] = x;
+            if (blockIdx.x == 0) a.x_out[k] = x;
+        }
+    } else {
+        for (size_t k = tid; k < K; k += kThreads) xs[k] = a.res[k];
+    }
+    if (a.norm_w) {
+        float ss = 0.f;
+        for (size_t k = tid; k < K; k += kThreads) ss = fmaf(xs[k], xs[k], ss);  // (a thread's own elements)
+        const float inv = inv_rms(ss);
+        for (size_t k = tid; k < K; k += kThreads) xs[k] = __fmul_rn(__fmul_rn(xs[k], inv), a.norm_w[k]);
+    }
+    __syncthreads();
+    const WT *w = static_cast<const WT *>(a.w);
+    constexpr int VEC = 16 / sizeof(WT);
+    const bool vec_ok = (K % VEC == 0) && ((reinterpret_cast<uintptr_t>(w) & 15) == 0);
+    for (size_t row = (size_t)blockIdx.x * kWarps + warp; row < a.N; row += (size_t)gridDim.x * kWarps) {
+        float acc[1] = {0.f};
+        row_dot<WT, 1>(w + row * K, xs, K, lane, vec_ok, acc);
+        float v = warp_sum(acc[0]);
+        if (lane == 0) {
+            if (a.act != StepFinish::kStore) v = gelu_tanh(v);
+            if (a.act == StepFinish::kSideGate) {
+                const unsigned long long tok = id_to_index(a.ids[0]);
+                v *= tok < a.table_rows ? to_f32(static_cast<const WT *>(a.table)[tok * a.table_ld + row]) : 0.f;
+            }
+            a.out[row] = v;
         }
     }
 }
@@ -479,6 +395,21 @@ int launch_gemv_gate_up(lumen_ctx *ctx, const float *x, const void *w_gate, cons
         default: return f32 ? GU(float, 8) : GU(__nv_bfloat16, 8);
     }
 #undef GU
+}
+
+int launch_gemv_step(lumen_ctx *ctx, const GemvStepArgs &a, cudaStream_t s) {
+    const size_t smem = a.K * sizeof(float);
+    if (smem > 200 * 1024) return set_error(ctx, LUMEN_ERR_UNSUPPORTED, "gemv_step: row of %zu elements", a.K);
+    const int grid = pick_grid(ctx, a.N, smem);
+    if (a.wdt == LUMEN_F32) {
+        LUMEN_TRY(set_smem(ctx, gemv_step_kernel<float>, smem));
+        gemv_step_kernel<float><<<grid, kThreads, smem, s>>>(a);
+    } else {
+        LUMEN_TRY(set_smem(ctx, gemv_step_kernel<__nv_bfloat16>, smem));
+        gemv_step_kernel<__nv_bfloat16><<<grid, kThreads, smem, s>>>(a);
+    }
+    LUMEN_LAUNCHED(ctx);
+    return LUMEN_OK;
 }
 
 size_t gemv_kn_scratch_bytes_for(size_t K, size_t N, lumen_dtype wdt, int num_sms) {

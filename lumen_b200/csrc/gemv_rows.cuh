@@ -1,0 +1,154 @@
+// Device helpers of the streaming vector-matrix kernels (gemv.cu, moe.cu): dot products of weight rows read once from
+// HBM with 128-bit streaming loads against vectors staged in shared memory, one warp per row (or group of rows).
+#pragma once
+
+#include "common.cuh"
+
+namespace lumen {
+
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+
+__device__ __forceinline__ float4 ld_stream_f4(const float4 *p) { return __ldcs(p); }
+__device__ __forceinline__ uint4 ld_stream_u4(const uint4 *p) { return __ldcs(p); }
+
+__device__ __forceinline__ float bf16_lo(uint32_t u) { return __uint_as_float(u << 16); }
+__device__ __forceinline__ float bf16_hi(uint32_t u) { return __uint_as_float(u & 0xffff0000u); }
+
+// Accumulate one row (`wrow`, K elements) against MB staged vectors.  Vector path needs K % VEC == 0
+// and a 16-byte aligned row; otherwise the scalar path runs.
+template <typename WT, int MB>
+__device__ __forceinline__ void row_dot(const WT *__restrict__ wrow, const float *xs, size_t K, int lane, bool vec_ok,
+                                        float (&acc)[MB]) {
+    constexpr int kUnroll = 8;
+    if constexpr (sizeof(WT) == 4) {
+        if (vec_ok) {
+            const float4 *w4 = reinterpret_cast<const float4 *>(wrow);
+            const size_t n4 = K / 4;
+            for (size_t base = 0; base < n4; base += 32 * kUnroll) {
+                float4 wv[kUnroll];
+#pragma unroll
+                for (int u = 0; u < kUnroll; ++u) {
+                    size_t i = base + (size_t)u * 32 + lane;
+                    wv[u] = (i < n4) ? ld_stream_f4(w4 + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+                }
+#pragma unroll
+                for (int u = 0; u < kUnroll; ++u) {
+                    size_t i = base + (size_t)u * 32 + lane;
+                    if (i < n4) {
+#pragma unroll
+                        for (int m = 0; m < MB; ++m) {
+                            float4 xv = *reinterpret_cast<const float4 *>(xs + (size_t)m * K + i * 4);
+                            acc[m] = fmaf(wv[u].x, xv.x, acc[m]);
+                            acc[m] = fmaf(wv[u].y, xv.y, acc[m]);
+                            acc[m] = fmaf(wv[u].z, xv.z, acc[m]);
+                            acc[m] = fmaf(wv[u].w, xv.w, acc[m]);
+                        }
+                    }
+                }
+            }
+            return;
+        }
+        for (size_t k = lane; k < K; k += 32) {
+            float w = reinterpret_cast<const float *>(wrow)[k];
+#pragma unroll
+            for (int m = 0; m < MB; ++m) acc[m] = fmaf(w, xs[(size_t)m * K + k], acc[m]);
+        }
+    } else {
+        if (vec_ok) {
+            const uint4 *w8 = reinterpret_cast<const uint4 *>(wrow);
+            const size_t n8 = K / 8;
+            for (size_t base = 0; base < n8; base += 32 * kUnroll) {
+                uint4 wv[kUnroll];
+#pragma unroll
+                for (int u = 0; u < kUnroll; ++u) {
+                    size_t i = base + (size_t)u * 32 + lane;
+                    wv[u] = (i < n8) ? ld_stream_u4(w8 + i) : make_uint4(0u, 0u, 0u, 0u);
+                }
+#pragma unroll
+                for (int u = 0; u < kUnroll; ++u) {
+                    size_t i = base + (size_t)u * 32 + lane;
+                    if (i < n8) {
+#pragma unroll
+                        for (int m = 0; m < MB; ++m) {
+                            const float4 *xp = reinterpret_cast<const float4 *>(xs + (size_t)m * K + i * 8);
+                            float4 x0 = xp[0], x1 = xp[1];
+                            acc[m] = fmaf(bf16_lo(wv[u].x), x0.x, acc[m]);
+                            acc[m] = fmaf(bf16_hi(wv[u].x), x0.y, acc[m]);
+                            acc[m] = fmaf(bf16_lo(wv[u].y), x0.z, acc[m]);
+                            acc[m] = fmaf(bf16_hi(wv[u].y), x0.w, acc[m]);
+                            acc[m] = fmaf(bf16_lo(wv[u].z), x1.x, acc[m]);
+                            acc[m] = fmaf(bf16_hi(wv[u].z), x1.y, acc[m]);
+                            acc[m] = fmaf(bf16_lo(wv[u].w), x1.z, acc[m]);
+                            acc[m] = fmaf(bf16_hi(wv[u].w), x1.w, acc[m]);
+                        }
+                    }
+                }
+            }
+            return;
+        }
+        for (size_t k = lane; k < K; k += 32) {
+            float w = __bfloat162float(reinterpret_cast<const __nv_bfloat16 *>(wrow)[k]);
+#pragma unroll
+            for (int m = 0; m < MB; ++m) acc[m] = fmaf(w, xs[(size_t)m * K + k], acc[m]);
+        }
+    }
+}
+
+// RR rows of W against MB staged vectors at once: every 16 bytes of x read from shared memory feed RR rows, so
+// the shared-memory traffic per weight byte is MB / RR instead of MB (with MB = 8 and one row at a time the
+// kernel was bound by shared memory, not by HBM).  Vector path only (K % VEC == 0, 16-byte aligned rows).
+template <typename WT, int MB, int RR>
+__device__ __forceinline__ void rows_dot(const WT *const (&rows)[RR], const float *xs, size_t K, int lane, float (&acc)[RR][MB]) {
+    constexpr int VEC = 16 / sizeof(WT);
+    constexpr int kUnroll = 4;
+    const size_t nv = K / VEC;
+    for (size_t base = 0; base < nv; base += 32 * kUnroll) {
+        uint4 wv[RR][kUnroll];
+#pragma unroll
+        for (int u = 0; u < kUnroll; ++u) {
+            const size_t i = base + (size_t)u * 32 + lane;
+#pragma unroll
+            for (int r = 0; r < RR; ++r)
+                wv[r][u] = (i < nv) ? ld_stream_u4(reinterpret_cast<const uint4 *>(rows[r]) + i) : make_uint4(0u, 0u, 0u, 0u);
+        }
+#pragma unroll
+        for (int u = 0; u < kUnroll; ++u) {
+            const size_t i = base + (size_t)u * 32 + lane;
+            if (i < nv) {
+#pragma unroll
+                for (int m = 0; m < MB; ++m) {
+                    const float4 *xp = reinterpret_cast<const float4 *>(xs + (size_t)m * K + i * VEC);
+                    const float4 x0 = xp[0];
+                    if constexpr (sizeof(WT) == 4) {
+#pragma unroll
+                        for (int r = 0; r < RR; ++r) {
+                            acc[r][m] = fmaf(__uint_as_float(wv[r][u].x), x0.x, acc[r][m]);
+                            acc[r][m] = fmaf(__uint_as_float(wv[r][u].y), x0.y, acc[r][m]);
+                            acc[r][m] = fmaf(__uint_as_float(wv[r][u].z), x0.z, acc[r][m]);
+                            acc[r][m] = fmaf(__uint_as_float(wv[r][u].w), x0.w, acc[r][m]);
+                        }
+                    } else {
+                        const float4 x1 = xp[1];
+#pragma unroll
+                        for (int r = 0; r < RR; ++r) {
+                            acc[r][m] = fmaf(bf16_lo(wv[r][u].x), x0.x, acc[r][m]);
+                            acc[r][m] = fmaf(bf16_hi(wv[r][u].x), x0.y, acc[r][m]);
+                            acc[r][m] = fmaf(bf16_lo(wv[r][u].y), x0.z, acc[r][m]);
+                            acc[r][m] = fmaf(bf16_hi(wv[r][u].y), x0.w, acc[r][m]);
+                            acc[r][m] = fmaf(bf16_lo(wv[r][u].z), x1.x, acc[r][m]);
+                            acc[r][m] = fmaf(bf16_hi(wv[r][u].z), x1.y, acc[r][m]);
+                            acc[r][m] = fmaf(bf16_lo(wv[r][u].w), x1.z, acc[r][m]);
+                            acc[r][m] = fmaf(bf16_hi(wv[r][u].w), x1.w, acc[r][m]);
+                        }
+                    }
+                }
+            }
+        }
+    }
+}
+
+}  // namespace lumen

@@ -174,9 +174,9 @@ class KVCacheInner:
         return int(self.ctx._lib.lumen_kv_len(self.h))
 
     def read(self):
-        """Host copies of the `k` and `v` slabs."""
-        k = np.empty(self.shape, np.float32)
-        v = np.empty(self.shape, np.float32)
+        """Host copies of the `k` and `v` slabs (an f32 latent cache has rows in `k` only; its `v` stays zero)."""
+        k = np.zeros(self.shape, np.float32)
+        v = np.zeros(self.shape, np.float32)
         self.ctx.check(self.ctx._lib.lumen_kv_read(self.h, k.ctypes.data, v.ctypes.data))
         return k, v
 

@@ -69,8 +69,8 @@ class SafeTensorsFile:
             pass
 
 
-def load_llama_weights(path, model, verbose: bool = False) -> list:
-    """Fill `model` (a `LlamaModel`) from `path`.  Returns the names that were not found in the file."""
+def load_weights(path, model, verbose: bool = False) -> list:
+    """Fill `model` (any `LanguageModel`) from `path`.  Returns the names that were not found in the file."""
     missing = []
     with SafeTensorsFile(path) as f:
         present = set(f.names())
@@ -87,6 +87,9 @@ def load_llama_weights(path, model, verbose: bool = False) -> list:
             if verbose:
                 print(f"Loaded: {name}")
     return missing
+
+
+load_llama_weights = load_weights  # the reference's name (loader.rs:10)
 
 
 def save_safetensors(path, tensors: dict) -> None:
