@@ -358,6 +358,107 @@ def run_micro(args):
     return 0
 
 
+# Layer geometries of --micro layers: the model given as a list of layers beside the closest LlamaModel (bf16 weights, random, a
+# small vocabulary so that the layers dominate).  Feed-forwards of equal parameters: 2 x ff (dense) = 3 x intermediate.
+LAYER_CASES = {
+    "dense_2048": dict(width=2048, layers=8, heads=16, rank=512, ff=8448, llama=dict(intermediate_size=5632, num_key_value_heads=8)),
+    "dense_4096": dict(width=4096, layers=4, heads=32, rank=512, ff=16512, llama=dict(intermediate_size=11008, num_key_value_heads=8)),
+    # routed: a token uses 6 of 64 experts and the shared one, 3 x (6 x 1408 + 2816) x 2048 parameters = LlamaModel with 11264
+    "moe_2048": dict(width=2048, layers=4, heads=16, rank=512, moe=dict(experts=64, top=6, ff=1408, shared=2816),
+                     llama=dict(intermediate_size=11264, num_key_value_heads=8)),
+}
+
+
+def layer_models(L, case: str, max_seq: int):
+    """(FegetarConfig, LlamaConfig) of a case: heads of 128 (+ 64 rotated), values of 128."""
+    c = LAYER_CASES[case]
+    mixer = dict(heads=c["heads"], dim=128, rot_dim=64, vdim=128, kv_rank=c["rank"], scale=192 ** -0.5, rot=dict(base=10000.0, dims=64))
+    if "moe" in c:
+        m = c["moe"]
+        mlp = dict(kind="moe", router=dict(experts=m["experts"], top=m["top"]), expert=dict(ff=m["ff"], limit=7.0),
+                   shared=dict(ff=m["shared"], limit=7.0))
+    else:
+        mlp = dict(kind="dense", ff=c["ff"])
+    d = dict(architecture="Fegetar", vocab=4096, width=c["width"], norm=dict(eps=1e-5), token_side=dict(dim=256),
+             embedding=dict(bigram=dict(buckets=65521, mul_prev=31, mul_cur=7)),
+             layers=[dict(type="latent_attention", mixer=mixer, mlp=mlp)] * c["layers"])
+    return L.FegetarConfig.from_dict(d, max_seq, "bf16"), L.LlamaConfig(
+        vocab_size=4096, hidden_size=c["width"], num_hidden_layers=c["layers"], num_attention_heads=c["heads"], head_dim=128,
+        max_seq_len=max_seq, weight_dtype="bf16", **c["llama"])
+
+
+def run_layers(args):
+    """--micro layers: prefill and batch-1 decode of both models of every case, one JSON line per measurement.  Device ids and
+    logits, CUDA events around whole steps; the weights of a case exceed L2."""
+    import torch
+    import lumen_b200 as L
+    from lumen_b200.synth import f32_to_bf16_bits
+    torch.cuda.set_device(0)
+    ctx = L.Context(0)
+    stream = torch.cuda.ExternalStream(ctx.stream, device=torch.device("cuda", 0))
+    hbm, kind = measured_hbm_peak()
+    try:
+        tpeak = float(json.loads((ROOT / "MEASURED_PEAKS.json").read_text())["bf16_tflops"])
+    except Exception:
+        tpeak = 1590.0
+    cases = [args.layers_case] if args.layers_case else list(LAYER_CASES)
+    phases = [args.layers_phase] if args.layers_phase else ["prefill", "decode"]
+    models = [args.layers_model] if args.layers_model else ["fegetar", "llama"]
+    lens = [int(x) for x in args.layers_lens.split(",")]
+    rng = np.random.default_rng(0)
+    base = f32_to_bf16_bits(rng.standard_normal(1 << 22, dtype=np.float32) * np.float32(0.02))
+    sampler = ClockSampler(0)
+    sampler.start()
+    sampler.active = True
+    for case in cases:
+        max_seq = max(lens) + 96
+        for name, cfg in zip(("fegetar", "llama"), layer_models(L, case, max_seq)):
+            if name not in models:
+                continue
+            model = (L.FegetarModel if name == "fegetar" else L.LlamaModel)(cfg, ctx)
+            for i, (n, shape) in enumerate(sorted(cfg.param_shapes().items())):
+                size = int(np.prod(shape))
+                if len(shape) == 1:
+                    model.set_param(n, np.ones(shape, np.float32))
+                else:
+                    model.set_param(n, np.resize(np.roll(base, 7919 * i), size).reshape(shape), as_bf16_bits=True)
+            caches = model.init_kv_caches(1)
+            ids = L.Tensor.from_array_no_grad(rng.integers(0, 4096, max_seq).astype(np.float32), ctx)
+            logits = L.Tensor.from_array_no_grad(np.zeros(max(lens) * 4096, np.float32), ctx)
+            layer_params = sum(int(np.prod(s)) for n, s in cfg.param_shapes().items()
+                               if len(s) == 2 and n not in ("embed", "bigram", "side.embed", "model.embed_tokens.weight") and ".mlp.e" not in n)
+            if "moe" in LAYER_CASES[case] and name == "fegetar":
+                m = LAYER_CASES[case]["moe"]
+                layer_params += LAYER_CASES[case]["layers"] * 3 * m["top"] * m["ff"] * cfg.width
+            heads, n_layers = LAYER_CASES[case]["heads"], LAYER_CASES[case]["layers"]
+            qk, vd = (192, 128) if name == "fegetar" else (128, 128)
+            row_bytes = 576 * 2 if name == "fegetar" else 2 * LAYER_CASES[case]["llama"]["num_key_value_heads"] * 128 * 4
+            with L.no_grad():
+                for n in lens:
+                    if "prefill" in phases:
+                        def step():
+                            model.reset_kv_caches(caches)
+                            model.forward_device(ids.data_ptr, 1, n, caches, logits.data_ptr)
+                        ms = _event_time_ms(ctx, stream, step, iters=5 if not args.layers_once else 1, warm=3 if not args.layers_once else 1)
+                        flops = 2.0 * n * layer_params + n_layers * heads * n * (n + 1) / 2 * 2 * (qk + vd)
+                        print(json.dumps({"micro": "layers_prefill", "case": case, "model": name, "positions": n, "ms": ms, "tokens_per_s": n / ms * 1e3,
+                                          "tflops": flops / ms / 1e9, "frac_of_measured_bf16": flops / ms / 1e9 / tpeak}), flush=True)
+                    if "decode" in phases:
+                        model.reset_kv_caches(caches)
+                        model.forward_device(ids.data_ptr, 1, n, caches, logits.data_ptr)
+                        ms = _event_time_ms(ctx, stream, lambda: model.forward_device(ids.data_ptr, 1, 1, caches, logits.data_ptr),
+                                            iters=64 if not args.layers_once else 2, warm=8 if not args.layers_once else 2)
+                        nbytes = model.weight_bytes_per_step + n_layers * row_bytes * (n + 40)
+                        gbs = nbytes / ms / 1e6
+                        print(json.dumps({"micro": "layers_decode", "case": case, "model": name, "context": n, "ms": ms, "tokens_per_s": 1e3 / ms,
+                                          "weight_mb": model.weight_bytes_per_step / 1e6, "gbs": gbs, "frac_of_measured_hbm": gbs / hbm, "peak_kind": kind,
+                                          "persistent_kernel": name == "llama" and os.environ.get("LUMEN_NO_MEGA") != "1"}), flush=True)
+            del model, caches, ids, logits
+    sampler.stop()
+    print(json.dumps({"micro": "layers_clocks", **sampler.summary()}), flush=True)
+    return 0
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -372,7 +473,7 @@ def main():
     ap.add_argument("--profile-layers", type=int, default=0,
                     help="profiling aid: truncate the model to this many layers so that a profiler capture stays "
                          "small; the printed line is then marked and is not a benchmark value")
-    ap.add_argument("--micro", choices=["gemv", "attn", "gemm", "prefill"], default=None,
+    ap.add_argument("--micro", choices=["gemv", "attn", "gemm", "prefill", "layers"], default=None,
                     help="secondary measurements instead of the decode benchmark: the vector-matrix sweep or "
                          "decode attention over a static cache (one JSON line per case)")
     ap.add_argument("--batch", type=int, default=1,
@@ -385,12 +486,19 @@ def main():
     ap.add_argument("--no-extra", action="store_true", help="N > 1: skip the short Llama-2-7B run reported beside the headline")
     ap.add_argument("--prefill-chunk", type=int, default=0,
                     help="prefill the prompt in slices of this many positions (0: one forward)")
+    ap.add_argument("--layers-case", choices=list(LAYER_CASES), default=None, help="--micro layers: one case only")
+    ap.add_argument("--layers-model", choices=["fegetar", "llama"], default=None, help="--micro layers: one model only")
+    ap.add_argument("--layers-phase", choices=["prefill", "decode"], default=None, help="--micro layers: one phase only")
+    ap.add_argument("--layers-lens", default="512,2048,8192", help="--micro layers: prompt lengths / contexts")
+    ap.add_argument("--layers-once", action="store_true", help="--micro layers: very few steps (profiling aid, not a measurement)")
     args = ap.parse_args()
     global PROMPT_LEN
     PROMPT_LEN = args.prompt_len
     args.warmup = max(args.warmup, 3)
     if args.dtype is None:
         args.dtype = WORKLOADS[args.workload][2]
+    if args.micro == "layers":
+        return run_layers(args)
     if args.micro:
         return run_micro(args)
     if args.impl == "reference":

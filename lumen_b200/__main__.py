@@ -17,13 +17,13 @@ def generate(args) -> int:
     if args.text is not None:
         from .tokenizer import LlamaTokenizer
         tok = LlamaTokenizer.from_file(f"{args.model}/tokenizer.json")
-        ids = tok.encode(args.text)
+        ids = tok.encode(args.text, True)
     else:
         ids = [int(t) for t in args.ids.replace(",", " ").split()]
     session = ChatSession(model, lambda p: p, lambda p: p, stop_ids=args.stop or (), temperature=args.temperature, top_p=args.top_p,
                           repetition_penalty=args.repetition_penalty, max_gen=args.max_new)
     out = session.turn(ids)
-    print(tok.decode(out) if tok else " ".join(str(t) for t in out))
+    print(tok.decode(out, True) if tok else " ".join(str(t) for t in out))
     return 0
 
 
