@@ -72,6 +72,14 @@ int check_device_status(lumen_ctx *ctx) {
     return LUMEN_OK;
 }
 
+bool pdl_enabled() {
+    static const bool on = [] {
+        const char *e = getenv("LUMEN_NO_PDL");
+        return !(e && e[0] == '1');
+    }();
+    return on;
+}
+
 int kv_resync_len(lumen_kv_cache *c) {
     if (!c || !c->ctx || c->seen_abort == c->ctx->abort_gen) return LUMEN_OK;
     lumen_ctx *ctx = c->ctx;

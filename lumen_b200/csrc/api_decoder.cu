@@ -53,10 +53,10 @@ struct Workspace {
     void *qf = nullptr;
     float *part_ctx = nullptr, *part_ml = nullptr;
     // experts
-    float *z = nullptr, *weight = nullptr, *row_scale = nullptr, *yexp = nullptr, *vec_act = nullptr;
+    float *z = nullptr, *weight = nullptr, *row_scale = nullptr, *vec_act = nullptr;
     int *sel = nullptr, *pos = nullptr, *src = nullptr, *n_tiles = nullptr;
     int4 *tiles = nullptr;
-    __nv_bfloat16 *xperm = nullptr, *aperm = nullptr;
+    __nv_bfloat16 *xperm = nullptr, *aperm = nullptr, *yexp = nullptr;
     float *ids = nullptr, *logits = nullptr, *h_ids = nullptr, *h_logits = nullptr;
     size_t h_logits_elems = 0;
 };
@@ -345,7 +345,7 @@ int lumen_decoder::ensure_workspace(size_t M) {
                  o_nx = take(M * W * 4), o_last = take(M * W * 4), o_att = take(M * att * 4), o_act = take(M * act * 4), o_sd = take(M * sd * 4),
                  o_xh = take(bf ? M * W * 2 : 0), o_xl = take(bf ? M * W * 2 : 0), o_ah = take(bf ? M * att * 2 : 0), o_gh = take(bf ? M * act * 2 : 0),
                  o_sh = take(bf ? M * sd * 2 : 0), o_q = take(M * q * esz), o_pc = take(ctx_rows * rank * 4), o_pm = take(ctx_rows * 8),
-                 o_z = take(M * zmax * 4), o_wt = take(M * topmax * 4), o_rs = take(M * topmax * 4), o_ye = take(bf ? M * topmax * W * 4 : 0),
+                 o_z = take(M * zmax * 4), o_wt = take(M * topmax * 4), o_rs = take(M * topmax * 4), o_ye = take(bf ? M * topmax * W * 2 : 0),
                  o_va = take(M * vact * 4), o_sel = take(M * topmax * 4), o_pos = take(M * topmax * 4), o_src = take(M * topmax * 4), o_nt = take(4),
                  o_tiles = take(tiles * sizeof(int4)), o_xp = take(bf ? M * permx * 2 : 0), o_ap = take(bf ? M * perma * 2 : 0),
                  o_ids = take(M * 4), o_lg = take(M * V * 4);
@@ -358,7 +358,7 @@ int lumen_decoder::ensure_workspace(size_t M) {
     ws.att.f = f(o_att); ws.act.f = f(o_act); ws.side.f = f(o_sd);
     if (bf) { ws.xa.hi = h(o_xh); ws.xa.lo = h(o_xl); ws.att.hi = h(o_ah); ws.act.hi = h(o_gh); ws.side.hi = h(o_sh); }
     ws.qf = ws.base + o_q; ws.part_ctx = f(o_pc); ws.part_ml = f(o_pm);
-    ws.z = f(o_z); ws.weight = f(o_wt); ws.row_scale = f(o_rs); ws.yexp = f(o_ye); ws.vec_act = f(o_va);
+    ws.z = f(o_z); ws.weight = f(o_wt); ws.row_scale = f(o_rs); ws.yexp = h(o_ye); ws.vec_act = f(o_va);
     ws.sel = i(o_sel); ws.pos = i(o_pos); ws.src = i(o_src); ws.n_tiles = i(o_nt); ws.tiles = reinterpret_cast<int4 *>(ws.base + o_tiles);
     ws.xperm = h(o_xp); ws.aperm = h(o_ap); ws.ids = f(o_ids); ws.logits = f(o_lg);
     LUMEN_CUDA(ctx, cudaMallocHost(&ws.h_ids, std::max<size_t>(M, 1) * sizeof(float)));
@@ -481,16 +481,17 @@ int lumen_decoder::step_rows(size_t B, size_t S, lumen_kv_cache **caches, bool l
     EmbedArgs e;
     e.ids = ws.ids; e.embed = embed; e.bigram = bigram; e.dt = dt; e.B = B; e.S = S; e.vocab = V; e.dim = W;
     e.buckets = cfg.bigram_buckets; e.mul_prev = cfg.bigram_mul_prev; e.mul_cur = cfg.bigram_mul_cur;
-    e.d_len = caches[0]->d_len; e.last_tok = caches[0]->last_tok; e.x = ws.x[0]; e.hi = ws.xa.hi; e.lo = ws.xa.lo;
+    e.d_len = caches[0]->d_len; e.last_tok = caches[0]->last_tok; e.x = ws.x[0]; e.hi = ws.xa.hi;
     LUMEN_TRY(launch_embed(ctx, e, s));
     // What the products of this step read of an activation: bf16 on the tensor cores, f32 otherwise.
     auto target = [&](StepFinish &f, const Act &a, size_t K) {
         if (on_tensor_cores(M, K)) f.hi = a.hi;
         else f.out = a.f;
     };
-    auto norm_add = [&](const float *gain) {
+    auto norm_add = [&](const float *gain, bool pair = false) {
         StepFinish f;
-        f.kind = StepFinish::kNormAdd; f.x = ws.x[0]; f.gain = gain; f.eps = cfg.norm_eps; f.hi = ws.xa.hi; f.lo = ws.xa.lo;
+        f.kind = StepFinish::kNormAdd; f.x = ws.x[0]; f.gain = gain; f.eps = cfg.norm_eps; f.hi = ws.xa.hi;
+        if (pair) f.lo = ws.xa.lo;
         return f;
     };
     // Products whose activation is applied in the epilogue: enough rows that K is not split.
@@ -512,7 +513,7 @@ int lumen_decoder::step_rows(size_t B, size_t S, lumen_kv_cache **caches, bool l
             LUMEN_TRY(latent_mma_usable(a) ? launch_latent_mma(ctx, a, s) : launch_latent_scores(ctx, a, s));
             LUMEN_TRY(launch_latent_value(ctx, a, s));
         }
-        StepFinish f1 = norm_add(w.norm1);
+        StepFinish f1 = norm_add(w.norm1, k.mlp_kind == LUMEN_MLP_MOE);  // (the router reads the pair)
         LUMEN_TRY(product(ws.att, av, w.o, M, av, W, ws.y, &f1));
         if (k.mlp_kind == LUMEN_MLP_DENSE) {
             if (epilogue && on_tensor_cores(M, W) && on_tensor_cores(M, k.ff)) {
@@ -545,7 +546,8 @@ int lumen_decoder::step_rows(size_t B, size_t S, lumen_kv_cache **caches, bool l
                 LUMEN_TRY(launch_gemm_bf16(ctx, g, s));
                 GemmBf16Args d;
                 d.a_hi = ws.aperm; d.M = M * k.top; d.K = k.expert_ff; d.w = reinterpret_cast<const __nv_bfloat16 *>(w.edown);
-                d.N = W; d.w_groups = k.experts; d.tiles = ws.tiles; d.n_tiles = ws.n_tiles; d.max_tiles = g.max_tiles; d.c = ws.yexp;
+                d.N = W; d.w_groups = k.experts; d.tiles = ws.tiles; d.n_tiles = ws.n_tiles; d.max_tiles = g.max_tiles; d.out16 = ws.yexp; d.ld16 = W;
+                d.epi = GemmBf16Args::kBf16;
                 LUMEN_TRY(launch_gemm_bf16(ctx, d, s));
                 f2.gather_src = ws.yexp; f2.gather_idx = ws.pos; f2.gather_n = (int)k.top;
                 if (k.shared_ff) {
@@ -616,7 +618,12 @@ int lumen_decoder::run_forward(size_t b, size_t s, lumen_kv_cache **caches, bool
         for (size_t l = 0; l < L; ++l) key = key * 7 + (unsigned)latent_pick_splits(latent_args(l, caches[l], b, 1), caches[l]->len + 1, ctx->num_sms);
         const bool one = b == 1 && W * 4 <= 200 * 1024;
         rc = run_graphed(std::make_tuple(b, (int)key, (const void *)caches[0]->k),
-                         [&] { return one ? step_row(caches) : step_rows(b, 1, caches, last_only); });
+                         [&] {
+                             ctx->pdl = one;
+                             const int r = one ? step_row(caches) : step_rows(b, 1, caches, last_only);
+                             ctx->pdl = false;
+                             return r;
+                         });
     } else {
         rc = step_rows(b, s, caches, last_only);
     }

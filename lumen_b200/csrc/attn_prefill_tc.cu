@@ -469,27 +469,40 @@ fa_split_vt_kernel(const float *__restrict__ v_cache, __nv_bfloat16 *__restrict_
 }
 
 // Q of latent attention: u rows -> [B, H, s_pad, KB * 64] bf16: the unrotated part (dim numbers, zeros up to main), then the rotated
-// part, zeros elsewhere.  One thread per element.
+// part, zeros elsewhere.  One thread per 8 elements (dim and main are multiples of 8).
 __global__ void fa_pack_latent_q_kernel(const LatentArgs a, __nv_bfloat16 *__restrict__ q, int s_pad, int main, int width, size_t n) {
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= n) return;
-    const size_t e = i % width, row = i / width, s = row % s_pad, bh = row / s_pad, b = bh / a.H, h = bh % a.H;
-    float v = 0.f;
-    if (s < a.S) {
-        const float *src = a.u + (b * a.S + s) * a.u_ld + h * (a.dim + a.rot_dim);
-        if (e < (size_t)main) {
-            if (e < a.dim) v = src[e];
-        } else if (e - main < a.rot_dim) {
-            const size_t r = e - main;
-            v = src[a.dim + r];
-            if (r < a.rot_dims) {
-                const size_t at = (a.past + s) * (a.rot_dims / 2) + (r >> 1);
-                const float c = a.cos_t[at], sn = a.sin_t[at], w = src[a.dim + (r ^ 1)];
-                v = (r & 1) ? __fadd_rn(__fmul_rn(v, c), __fmul_rn(w, sn)) : __fsub_rn(__fmul_rn(v, c), __fmul_rn(w, sn));
+    const unsigned groups = (unsigned)width / 8, row = (unsigned)(i / groups);
+    const int e = (int)(i - (size_t)row * groups) * 8, s = (int)(row % (unsigned)s_pad);
+    const unsigned bh = row / (unsigned)s_pad, b = bh / (unsigned)a.H, h = bh - b * (unsigned)a.H;
+    float v[8];
+#pragma unroll
+    for (int k = 0; k < 8; ++k) v[k] = 0.f;
+    if (s < (int)a.S) {
+        const float *src = a.u + ((size_t)b * a.S + s) * a.u_ld + h * (a.dim + a.rot_dim);
+        if (e < main) {
+            if (e < (int)a.dim)
+#pragma unroll
+                for (int k = 0; k < 8; ++k) v[k] = src[e + k];
+        } else {
+            const int r0 = e - main, rot_dim = (int)a.rot_dim, rot_dims = (int)a.rot_dims;
+#pragma unroll
+            for (int k = 0; k < 8; k += 2) {
+                const int r = r0 + k;
+                const float x = r < rot_dim ? src[a.dim + r] : 0.f, y = r + 1 < rot_dim ? src[a.dim + r + 1] : 0.f;
+                v[k] = x;
+                v[k + 1] = y;
+                if (r < rot_dims) {  // (rot_dims is even: a pair turns as a whole)
+                    const size_t at = (a.past + s) * (size_t)(rot_dims / 2) + (r >> 1);
+                    const float c = a.cos_t[at], sn = a.sin_t[at];
+                    v[k] = __fsub_rn(__fmul_rn(x, c), __fmul_rn(y, sn));
+                    v[k + 1] = __fadd_rn(__fmul_rn(y, c), __fmul_rn(x, sn));
+                }
             }
         }
     }
-    q[i] = __float2bfloat16_rn(v);
+    reinterpret_cast<uint4 *>(q)[i] = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
 }
 
 template <int KB, int DV, bool PAIR>
@@ -594,7 +607,7 @@ int launch_latent_prefill(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s) {
     LUMEN_TRY(dev_alloc(ctx, (nq + nk + nv) * sizeof(__nv_bfloat16), &ws));
     __nv_bfloat16 *q = static_cast<__nv_bfloat16 *>(ws), *k = q + nq, *vt = k + nk;
     int rc = LUMEN_OK;
-    fa_pack_latent_q_kernel<<<(unsigned)((nq + 255) / 256), 256, 0, s>>>(a, q, (int)s_pad, kb_main * kBK, width, nq);
+    fa_pack_latent_q_kernel<<<(unsigned)((nq / 8 + 255) / 256), 256, 0, s>>>(a, q, (int)s_pad, kb_main * kBK, width, nq / 8);
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) rc = cuda_fail(ctx, e, "fa_pack_latent_q_kernel launch");
     else ctx->launches += 1;

@@ -38,6 +38,7 @@ struct lumen_ctx {
     lumen::DeviceStatus *d_status = nullptr;
     lumen::DeviceStatus *h_status = nullptr;  // pinned mirror
     char err[512] = {0};
+    bool pdl = false;  // launch_pdl may overlap kernels now (set by steps that consist of such launches alone)
     unsigned long long launches = 0;  // kernels enqueued so far (graph replays add their node count)
     // Persistent decode kernel: 16 device bytes whose second word is the cross-CTA abort flag, and the
     // epoch from which the next launch derives the tags of its exchanged activations.
@@ -131,6 +132,29 @@ int cuda_fail(lumen_ctx *ctx, cudaError_t e, const char *what);
         int rc__ = (call);              \
         if (rc__ != LUMEN_OK) return rc__; \
     } while (0)
+
+// Launches a kernel that may start while its predecessor on the stream still runs (programmatic dependent launch; captured
+// into graphs as such).  The kernel calls pdl_wait() before it touches anything a predecessor writes - until then it may
+// read weights - and pdl_launch() once its own successor may start the same way.  Every kernel launched so waits, so the end of a
+// kernel implies the end of all before it.  Plain launches unless ctx->pdl is set; LUMEN_NO_PDL=1: always plain.
+#ifdef __CUDACC__
+__device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+__device__ __forceinline__ void pdl_launch() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
+#endif
+bool pdl_enabled();
+template <typename... KA, typename... A>
+int launch_pdl(lumen_ctx *ctx, void (*kernel)(KA...), dim3 grid, dim3 block, size_t smem, cudaStream_t s, A... args) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid; cfg.blockDim = block; cfg.dynamicSmemBytes = smem; cfg.stream = s;
+    cudaLaunchAttribute attr = {};
+    attr.id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr.val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = &attr;
+    cfg.numAttrs = ctx->pdl && pdl_enabled() ? 1 : 0;
+    LUMEN_CUDA(ctx, cudaLaunchKernelEx(&cfg, kernel, args...));
+    ctx->launches += 1;
+    return LUMEN_OK;
+}
 
 int check_device_status(lumen_ctx *ctx);
 // Brings the host mirror of a cache's length back in line with the device copy after a device-side abort

@@ -7,6 +7,8 @@ namespace {
 template <typename T>
 __global__ void __launch_bounds__(256) embed_kernel(EmbedArgs a, DeviceStatus *status) {
     const size_t m = blockIdx.x, b = m / a.S, s = m - b * a.S;
+    pdl_launch();
+    pdl_wait();
     unsigned long long tok = id_to_index(a.ids[m]);
     if (tok >= a.vocab) {
         if (threadIdx.x == 0 && atomicCAS(&status->code, 0, LUMEN_ERR_EMBED_RANGE) == 0) {
@@ -33,6 +35,7 @@ __global__ void __launch_bounds__(256) embed_kernel(EmbedArgs a, DeviceStatus *s
 }
 
 __global__ void advance_kernel(int *lens, int layers, const float *ids, int *last_tok, int B, int S) {
+    pdl_wait();
     for (int l = threadIdx.x; l < layers; l += blockDim.x) lens[l] += S;
     for (int b = threadIdx.x; b < B; b += blockDim.x) last_tok[b] = (int)id_to_index(ids[(size_t)b * S + S - 1]);
 }
@@ -41,16 +44,11 @@ __global__ void advance_kernel(int *lens, int layers, const float *ids, int *las
 
 int launch_embed(lumen_ctx *ctx, const EmbedArgs &a, cudaStream_t s) {
     const unsigned rows = (unsigned)(a.B * a.S);
-    if (a.dt == LUMEN_F32) embed_kernel<float><<<rows, 256, 0, s>>>(a, ctx->d_status);
-    else embed_kernel<__nv_bfloat16><<<rows, 256, 0, s>>>(a, ctx->d_status);
-    LUMEN_LAUNCHED(ctx);
-    return LUMEN_OK;
+    return launch_pdl(ctx, a.dt == LUMEN_F32 ? embed_kernel<float> : embed_kernel<__nv_bfloat16>, rows, 256, 0, s, a, ctx->d_status);
 }
 
 int launch_advance(lumen_ctx *ctx, int *d_lens, size_t layers, const float *ids, int *last_tok, size_t B, size_t S, cudaStream_t s) {
-    advance_kernel<<<1, 256, 0, s>>>(d_lens, (int)layers, ids, last_tok, (int)B, (int)S);
-    LUMEN_LAUNCHED(ctx);
-    return LUMEN_OK;
+    return launch_pdl(ctx, advance_kernel, 1, 256, 0, s, d_lens, (int)layers, ids, last_tok, (int)B, (int)S);
 }
 
 }  // namespace lumen

@@ -27,7 +27,7 @@ int launch_advance(lumen_ctx *ctx, int *d_lens, size_t layers, const float *ids,
 struct StepFinish {
     enum Kind {
         kStore,     // out = sum
-        kNormAdd,   // x += RMSNorm(sum + extra + gathered rows) * gain; (hi, lo) = split(x)
+        kNormAdd,   // x += RMSNorm(sum + gathered rows) * gain; (hi, lo) = split(x)
         kGelu,      // out = gelu_tanh(sum)
         kSideGate,  // out = gelu_tanh(sum) * table[id, col]
         kGated,     // sum holds gate and up in blocks of 64 columns: out = clamped SwiGLU (see gated_act)
@@ -35,8 +35,7 @@ struct StepFinish {
     float *x = nullptr;
     const float *gain = nullptr;
     float eps = 0.f;
-    const float *extra = nullptr;       // [rows, n] one more addend
-    const float *gather_src = nullptr;  // rows gather_idx[row, 0 .. gather_n) of this matrix are added too
+    const __nv_bfloat16 *gather_src = nullptr;  // rows gather_idx[row, 0 .. gather_n) of this matrix are added too
     const int *gather_idx = nullptr;
     int gather_n = 0;
     const float *ids = nullptr;         // kSideGate
@@ -48,7 +47,7 @@ struct StepFinish {
     float *out = nullptr;
     __nv_bfloat16 *hi = nullptr, *lo = nullptr;
 };
-// part: [splits][rows][n] (null with kNormAdd: nothing but extra / gathered rows).
+// part: [splits][rows][n] (null with kNormAdd: nothing but gathered rows).
 int launch_step_finish(lumen_ctx *ctx, const float *part, int splits, size_t rows, size_t n, const StepFinish &f, cudaStream_t s);
 
 // ---- products -----------------------------------------------------------------------------------

@@ -56,18 +56,34 @@ __global__ void __launch_bounds__(256) sum_swiglu_split_kernel(const float *__re
 
 // One CTA per row, any row length (the row is kept in shared memory between the two passes).
 __global__ void __launch_bounds__(256) norm_add_kernel(const float *__restrict__ part, int splits, size_t rows, size_t n, const StepFinish f) {
-    extern __shared__ float row_s[];
+    extern __shared__ __align__(16) float row_s[];
     __shared__ float red[8];
     const int tid = threadIdx.x;
     const size_t row = blockIdx.x, base = row * n, mn = rows * n;
     float ss = 0.f;
-    for (size_t i = tid; i < n; i += 256) {
-        float v = 0.f;
-        for (int sl = 0; sl < splits; ++sl) v = __fadd_rn(v, part[(size_t)sl * mn + base + i]);
-        for (int k = 0; k < f.gather_n; ++k) v = __fadd_rn(v, f.gather_src[(size_t)f.gather_idx[row * f.gather_n + k] * n + i]);
-        if (f.extra) v = __fadd_rn(v, f.extra[base + i]);
-        row_s[i] = v;
-        ss = fmaf(v, v, ss);
+    const bool vec = n % 4 == 0;
+    if (vec) {
+        for (size_t i = tid; i < n / 4; i += 256) {
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+            for (int sl = 0; sl < splits; ++sl) v = add4(v, reinterpret_cast<const float4 *>(part + (size_t)sl * mn + base)[i]);
+#pragma unroll 4
+            for (int k = 0; k < f.gather_n; ++k) {
+                const uint2 g = reinterpret_cast<const uint2 *>(f.gather_src + (size_t)f.gather_idx[row * f.gather_n + k] * n)[i];
+                v = add4(v, make_float4(__uint_as_float(g.x << 16), __uint_as_float(g.x & 0xffff0000u), __uint_as_float(g.y << 16),
+                                        __uint_as_float(g.y & 0xffff0000u)));
+            }
+            reinterpret_cast<float4 *>(row_s)[i] = v;
+            ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+        }
+    } else {
+        for (size_t i = tid; i < n; i += 256) {
+            float v = 0.f;
+            for (int sl = 0; sl < splits; ++sl) v = __fadd_rn(v, part[(size_t)sl * mn + base + i]);
+            for (int k = 0; k < f.gather_n; ++k) v = __fadd_rn(v, __bfloat162float(f.gather_src[(size_t)f.gather_idx[row * f.gather_n + k] * n + i]));
+            row_s[i] = v;
+            ss = fmaf(v, v, ss);
+        }
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
@@ -77,6 +93,22 @@ __global__ void __launch_bounds__(256) norm_add_kernel(const float *__restrict__
 #pragma unroll
     for (int w = 0; w < 8; ++w) t += red[w];
     const float inv = __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(t, (float)n), f.eps)));
+    if (vec) {
+        for (size_t i = tid; i < n / 4; i += 256) {
+            const float4 v = reinterpret_cast<const float4 *>(row_s)[i], g = reinterpret_cast<const float4 *>(f.gain)[i];
+            float4 *xp = reinterpret_cast<float4 *>(f.x + base) + i;
+            const float4 x = add4(*xp, make_float4(__fmul_rn(__fmul_rn(v.x, inv), g.x), __fmul_rn(__fmul_rn(v.y, inv), g.y),
+                                                   __fmul_rn(__fmul_rn(v.z, inv), g.z), __fmul_rn(__fmul_rn(v.w, inv), g.w)));
+            *xp = x;
+            if (f.hi) {
+                uint2 h, l;
+                split4(x, &h, &l);
+                reinterpret_cast<uint2 *>(f.hi + base)[i] = h;
+                if (f.lo) reinterpret_cast<uint2 *>(f.lo + base)[i] = l;
+            }
+        }
+        return;
+    }
     for (size_t i = tid; i < n; i += 256) {
         const float x = __fadd_rn(f.x[base + i], __fmul_rn(__fmul_rn(row_s[i], inv), f.gain[i]));
         f.x[base + i] = x;

@@ -30,7 +30,7 @@ using namespace tc;
 constexpr int kBM = 128;  // tile rows of A
 constexpr int kTcThreads = 128;
 constexpr uint32_t kABytes = kBM * kBK * 2;
-// The tile is 128 x BN: BN = 128, or 64 / 32 for outputs narrower than that.  The 128-row side ("A") and the BN-row
+// The tile is 128 x BN: BN = 128, or 64 / 32 for outputs narrower than that (256 for single bf16 operands, launch_gemm_bf16).  The 128-row side ("A") and the BN-row
 // side ("B") each arrive as one or two bf16 matrices (a bf16 matrix, or the hi and lo parts of an f32 one):
 //   plain:   A = activations (hi, lo), B = weights (bf16: one part; f32: hi, lo)   -> tile rows are output rows
 //   swapped: A = weights (bf16: one part; f32: hi, lo), B = activations (hi, lo)   -> tile rows are output columns
@@ -176,13 +176,13 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid_constan
         const int arow = a0 + warp * 32 + lane;  // this thread's row of the tile's 128-row side
         const bool empty_slice = nkb == 0;       // nothing was accumulated: the tile's contribution is zero
         if constexpr (EPI == GemmBf16Args::kGated) {
-            // columns 0 .. 63 of the tile are gates, 64 .. 127 the ups that go with them: 64 columns of output
+            // in every 128 columns of the tile 64 are gates, and 64 the ups that go with them: 64 columns of output
             const float scale = p.row_scale && arow < a_end ? p.row_scale[arow] : 1.f;
             const bool vec = (p.ld16 & 7) == 0;
 #pragma unroll 1
-            for (int c0 = 0; c0 < 64; c0 += 32) {
+            for (int c0 = 0; c0 < kBN / 2; c0 += 32) {  // gate columns of a wider tile: 0 .. 63, 128 .. 191
                 uint32_t g[32], u[32];
-                const uint32_t taddr = tmem_base + ((uint32_t)(warp * 32) << 16) + (uint32_t)c0;
+                const uint32_t taddr = tmem_base + ((uint32_t)(warp * 32) << 16) + (uint32_t)(c0 + (c0 & ~63));
                 tmem_ld32_issue(taddr, g);
                 tmem_ld32_issue(taddr + 64, u);
                 tmem_ld_wait();
@@ -220,6 +220,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid_constan
             }
         } else {
         float *cbase = p.c + (size_t)blockIdx.z * p.M * p.N;
+        const bool vec4 = (p.N & 3) == 0 && ((reinterpret_cast<uintptr_t>(cbase) | reinterpret_cast<uintptr_t>(p.residual)) & 15) == 0;
 #pragma unroll 1
         for (int c0 = 0; c0 < kBN; c0 += 32) {
             uint32_t v[32];
@@ -229,6 +230,19 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid_constan
                 if (arow < a_end) {  // output row arow, columns b0 + c0 ..
                     float *crow = cbase + (size_t)arow * p.N + b0 + c0;
                     const float *rrow = p.residual ? p.residual + (size_t)arow * p.N + b0 + c0 : nullptr;
+                    if (vec4 && b0 + c0 + 32 <= p.N) {
+#pragma unroll
+                        for (int j = 0; j < 32; j += 4) {
+                            float4 x = empty_slice ? make_float4(0.f, 0.f, 0.f, 0.f)
+                                                   : make_float4(__uint_as_float(v[j]), __uint_as_float(v[j + 1]), __uint_as_float(v[j + 2]), __uint_as_float(v[j + 3]));
+                            if (rrow) {
+                                const float4 r = *reinterpret_cast<const float4 *>(rrow + j);
+                                x = make_float4(__fadd_rn(r.x, x.x), __fadd_rn(r.y, x.y), __fadd_rn(r.z, x.z), __fadd_rn(r.w, x.w));
+                            }
+                            *reinterpret_cast<float4 *>(crow + j) = x;
+                        }
+                        continue;
+                    }
 #pragma unroll
                     for (int j = 0; j < 32; ++j) {
                         if (b0 + c0 + j < p.N) {
@@ -448,7 +462,8 @@ int launch_gemm_bf16(lumen_ctx *ctx, const GemmBf16Args &g, cudaStream_t s) {
     if (g.M == 0 || g.N == 0) return LUMEN_OK;
     const size_t lda = g.lda ? g.lda : g.K, ldw = g.ldw ? g.ldw : g.K;
     const bool pair = g.a_lo != nullptr, grouped = g.tiles != nullptr;
-    if (!gemm_bf16_usable(g.K, lda, ldw, g.a_hi, g.w) || (pair && g.epi != GemmBf16Args::kF32) || g.M > 0x7fffffff || g.N * g.w_groups > 0x7fffffff)
+    if (!gemm_bf16_usable(g.K, lda, ldw, g.a_hi, g.w) || (pair && g.epi != GemmBf16Args::kF32) ||
+        (grouped && g.epi != GemmBf16Args::kGated && g.epi != GemmBf16Args::kBf16) || g.M > 0x7fffffff || g.N * g.w_groups > 0x7fffffff)
         return set_error(ctx, LUMEN_ERR_UNSUPPORTED, "tensor-core product: %zu x %zu x %zu", g.M, g.N, g.K);
     TcParams p{};
     p.c = g.c; p.M = (int)g.M; p.N = (int)g.N; p.K = (int)g.K; p.status = ctx->d_status;
@@ -457,7 +472,12 @@ int launch_gemm_bf16(lumen_ctx *ctx, const GemmBf16Args &g, cudaStream_t s) {
     const int kb_all = (int)((g.K + kBK - 1) / kBK);
     p.kb_per_split = kb_all;
     const bool swap = g.M <= 64 && g.epi == GemmBf16Args::kF32 && !grouped;
-    const int bn = swap ? 64 : g.epi == GemmBf16Args::kGated || grouped ? 128 : pick_bn(g.M, g.N, ctx->num_sms);
+    // 256-wide tiles read each activation tile half as often and keep the tensor pipe busier, unless they leave the last wave
+    // of CTAs emptier than that is worth (a 256-wide tile takes about 1.5 times as long as a 128-wide one)
+    const size_t row_tiles = grouped ? g.max_tiles : (g.M + kBM - 1) / kBM;
+    auto waves = [&](size_t width) { return (row_tiles * ((g.N + width - 1) / width) + ctx->num_sms - 1) / ctx->num_sms; };
+    const bool wide = !swap && !pair && g.M > (size_t)kBM && g.N > 128 && 3 * waves(256) <= 2 * waves(128);
+    const int bn = swap ? 64 : wide ? 256 : g.epi == GemmBf16Args::kGated || grouped ? 128 : pick_bn(g.M, g.N, ctx->num_sms);
     int splits = 1;
     void *partial = nullptr;
     if (g.epi == GemmBf16Args::kF32 && !grouped && g.M <= (size_t)kBM) {
@@ -486,7 +506,12 @@ int launch_gemm_bf16(lumen_ctx *ctx, const GemmBf16Args &g, cudaStream_t s) {
     }
 #define LUMEN_TC(NA_, NB_, BN_, SW_, EPI_, GR_) launch_tc_kernel<NA_, NB_, BN_, SW_, EPI_, GR_>(ctx, ma, ma2, mb, mb2, p, g.M, g.N, s, g.max_tiles)
     if (rc == LUMEN_OK) {
-        if (grouped) rc = g.epi == GemmBf16Args::kGated ? LUMEN_TC(1, 1, 128, false, 3, true) : LUMEN_TC(1, 1, 128, false, 0, true);
+        if (grouped && wide) rc = g.epi == GemmBf16Args::kGated ? LUMEN_TC(1, 1, 256, false, 3, true) : LUMEN_TC(1, 1, 256, false, 1, true);
+        else if (grouped) rc = g.epi == GemmBf16Args::kGated ? LUMEN_TC(1, 1, 128, false, 3, true) : LUMEN_TC(1, 1, 128, false, 1, true);
+        else if (wide) rc = g.epi == GemmBf16Args::kGated  ? LUMEN_TC(1, 1, 256, false, 3, false)
+                            : g.epi == GemmBf16Args::kGelu ? LUMEN_TC(1, 1, 256, false, 2, false)
+                            : g.epi == GemmBf16Args::kBf16 ? LUMEN_TC(1, 1, 256, false, 1, false)
+                                                           : LUMEN_TC(1, 1, 256, false, 0, false);
         else if (swap) rc = pair ? LUMEN_TC(1, 2, 64, true, 0, false) : LUMEN_TC(1, 1, 64, true, 0, false);
         else if (g.epi == GemmBf16Args::kGated) rc = LUMEN_TC(1, 1, 128, false, 3, false);
         else if (g.epi == GemmBf16Args::kGelu) rc = bn == 128 ? LUMEN_TC(1, 1, 128, false, 2, false) : bn == 64 ? LUMEN_TC(1, 1, 64, false, 2, false) : LUMEN_TC(1, 1, 32, false, 2, false);

@@ -176,7 +176,14 @@ __global__ void __launch_bounds__(kThreads) gemv_step_kernel(const GemvStepArgs 
     __shared__ float red[kWarps];
     float *xs = smem;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const size_t K = a.K;
+    const size_t K = a.K, row0 = (size_t)blockIdx.x * kWarps + warp;
+    const WT *w = static_cast<const WT *>(a.w);
+    constexpr int VEC = 16 / sizeof(WT);
+    const bool vec_ok = (K % VEC == 0) && ((reinterpret_cast<uintptr_t>(w) & 15) == 0);
+    uint4 pre[8];
+    if (vec_ok && row0 < a.N) row_ahead<WT>(w + row0 * K, K, lane, pre);
+    pdl_launch();
+    pdl_wait();
     auto inv_rms = [&](float ss) {
         ss = warp_sum(ss);
         if (lane == 0) red[warp] = ss;
@@ -189,33 +196,65 @@ __global__ void __launch_bounds__(kThreads) gemv_step_kernel(const GemvStepArgs 
     };
     if (a.y) {
         float ss = 0.f;
-        for (size_t k = tid; k < K; k += kThreads) {
-            const float v = a.y[k];
-            xs[k] = v;
-            ss = fmaf(v, v, ss);
+        if (K % 4 == 0) {  // res and the gains are requested before the sum of y^2 is needed
+            constexpr int kHold = 4;  // float4 per thread held in registers: rows of up to 4096
+            const float4 *y4 = reinterpret_cast<const float4 *>(a.y), *r4 = reinterpret_cast<const float4 *>(a.res), *g4 = reinterpret_cast<const float4 *>(a.gain);
+            float4 *x4 = reinterpret_cast<float4 *>(xs), *o4 = reinterpret_cast<float4 *>(a.x_out);
+            const size_t n4 = K / 4;
+            float4 r[kHold], g[kHold];
+#pragma unroll
+            for (int i = 0; i < kHold; ++i)
+                if (tid + kThreads * i < n4) {
+                    r[i] = r4[tid + kThreads * i];
+                    g[i] = g4[tid + kThreads * i];
+                }
+            for (size_t k = tid; k < n4; k += kThreads) {
+                const float4 v = y4[k];
+                x4[k] = v;
+                ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+            }
+            const float inv = inv_rms(ss);
+            auto settle = [&](size_t k, float4 res, float4 gain) {
+                const float4 v = x4[k];
+                const float4 x = make_float4(__fadd_rn(res.x, __fmul_rn(__fmul_rn(v.x, inv), gain.x)), __fadd_rn(res.y, __fmul_rn(__fmul_rn(v.y, inv), gain.y)),
+                                             __fadd_rn(res.z, __fmul_rn(__fmul_rn(v.z, inv), gain.z)), __fadd_rn(res.w, __fmul_rn(__fmul_rn(v.w, inv), gain.w)));
+                x4[k] = x;
+                if (blockIdx.x == 0) o4[k] = x;
+            };
+#pragma unroll
+            for (int i = 0; i < kHold; ++i)
+                if (tid + kThreads * i < n4) settle(tid + kThreads * i, r[i], g[i]);
+            for (size_t k = tid + kThreads * kHold; k < n4; k += kThreads) settle(k, r4[k], g4[k]);
+        } else {
+            for (size_t k = tid; k < K; k += kThreads) {
+                const float v = a.y[k];
+                xs[k] = v;
+                ss = fmaf(v, v, ss);
+            }
+            const float inv = inv_rms(ss);
+            for (size_t k = tid; k < K; k += kThreads) {
+                const float x = __fadd_rn(a.res[k], __fmul_rn(__fmul_rn(xs[k], inv), a.gain[k]));
+                xs[k] = x;
+                if (blockIdx.x == 0) a.x_out[k] = x;
+            }
         }
-        const float inv = inv_rms(ss);
-        for (size_t k = tid; k < K; k += kThreads) {
-            const float x = __fadd_rn(a.res[k], __fmul_rn(__fmul_rn(xs[k], inv), a.gain[k]));
-            xs[k] = x;
-            if (blockIdx.x == 0) a.x_out[k] = x;
-        }
+    } else if (K % 4 == 0) {
+        for (size_t k = tid; k < K / 4; k += kThreads) reinterpret_cast<float4 *>(xs)[k] = reinterpret_cast<const float4 *>(a.res)[k];
     } else {
         for (size_t k = tid; k < K; k += kThreads) xs[k] = a.res[k];
     }
     if (a.norm_w) {
+        __syncthreads();
         float ss = 0.f;
-        for (size_t k = tid; k < K; k += kThreads) ss = fmaf(xs[k], xs[k], ss);  // (a thread's own elements)
+        for (size_t k = tid; k < K; k += kThreads) ss = fmaf(xs[k], xs[k], ss);
         const float inv = inv_rms(ss);
         for (size_t k = tid; k < K; k += kThreads) xs[k] = __fmul_rn(__fmul_rn(xs[k], inv), a.norm_w[k]);
     }
     __syncthreads();
-    const WT *w = static_cast<const WT *>(a.w);
-    constexpr int VEC = 16 / sizeof(WT);
-    const bool vec_ok = (K % VEC == 0) && ((reinterpret_cast<uintptr_t>(w) & 15) == 0);
-    for (size_t row = (size_t)blockIdx.x * kWarps + warp; row < a.N; row += (size_t)gridDim.x * kWarps) {
+    for (size_t row = row0; row < a.N; row += (size_t)gridDim.x * kWarps) {
         float acc[1] = {0.f};
-        row_dot<WT, 1>(w + row * K, xs, K, lane, vec_ok, acc);
+        if (vec_ok && row == row0) acc[0] = row_dot_ahead<WT>(w + row * K, xs, K, lane, pre);
+        else row_dot<WT, 1>(w + row * K, xs, K, lane, vec_ok, acc);
         float v = warp_sum(acc[0]);
         if (lane == 0) {
             if (a.act != StepFinish::kStore) v = gelu_tanh(v);
@@ -403,13 +442,10 @@ int launch_gemv_step(lumen_ctx *ctx, const GemvStepArgs &a, cudaStream_t s) {
     const int grid = pick_grid(ctx, a.N, smem);
     if (a.wdt == LUMEN_F32) {
         LUMEN_TRY(set_smem(ctx, gemv_step_kernel<float>, smem));
-        gemv_step_kernel<float><<<grid, kThreads, smem, s>>>(a);
-    } else {
-        LUMEN_TRY(set_smem(ctx, gemv_step_kernel<__nv_bfloat16>, smem));
-        gemv_step_kernel<__nv_bfloat16><<<grid, kThreads, smem, s>>>(a);
+        return launch_pdl(ctx, gemv_step_kernel<float>, grid, kThreads, smem, s, a);
     }
-    LUMEN_LAUNCHED(ctx);
-    return LUMEN_OK;
+    LUMEN_TRY(set_smem(ctx, gemv_step_kernel<__nv_bfloat16>, smem));
+    return launch_pdl(ctx, gemv_step_kernel<__nv_bfloat16>, grid, kThreads, smem, s, a);
 }
 
 size_t gemv_kn_scratch_bytes_for(size_t K, size_t N, lumen_dtype wdt, int num_sms) {

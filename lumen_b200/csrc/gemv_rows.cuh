@@ -98,6 +98,66 @@ __device__ __forceinline__ void row_dot(const WT *__restrict__ wrow, const float
     }
 }
 
+// The first 8 x 32 vectors of a row requested ahead of time (while an earlier kernel still runs), the rest of the row handed to the
+// L2; row_dot_ahead then is row_dot<WT, 1> whose first batch is in registers.
+template <typename WT>
+__device__ __forceinline__ void row_ahead(const WT *__restrict__ wrow, size_t K, int lane, uint4 (&pre)[8]) {
+    constexpr int VEC = 16 / sizeof(WT);
+    const size_t nv = K / VEC;
+#pragma unroll
+    for (int u = 0; u < 8; ++u) {
+        const size_t i = (size_t)u * 32 + lane;
+        pre[u] = i < nv ? ld_stream_u4(reinterpret_cast<const uint4 *>(wrow) + i) : make_uint4(0u, 0u, 0u, 0u);
+    }
+    for (size_t off = 4096 + (size_t)lane * 128; off < K * sizeof(WT); off += 4096)
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char *>(wrow) + off));
+}
+template <typename WT>
+__device__ __forceinline__ float vec_dot(uint4 w, const float *x, float acc) {
+    const float4 x0 = *reinterpret_cast<const float4 *>(x);
+    if constexpr (sizeof(WT) == 4) {
+        acc = fmaf(__uint_as_float(w.x), x0.x, acc);
+        acc = fmaf(__uint_as_float(w.y), x0.y, acc);
+        acc = fmaf(__uint_as_float(w.z), x0.z, acc);
+        return fmaf(__uint_as_float(w.w), x0.w, acc);
+    } else {
+        const float4 x1 = *reinterpret_cast<const float4 *>(x + 4);
+        acc = fmaf(bf16_lo(w.x), x0.x, acc);
+        acc = fmaf(bf16_hi(w.x), x0.y, acc);
+        acc = fmaf(bf16_lo(w.y), x0.z, acc);
+        acc = fmaf(bf16_hi(w.y), x0.w, acc);
+        acc = fmaf(bf16_lo(w.z), x1.x, acc);
+        acc = fmaf(bf16_hi(w.z), x1.y, acc);
+        acc = fmaf(bf16_lo(w.w), x1.z, acc);
+        return fmaf(bf16_hi(w.w), x1.w, acc);
+    }
+}
+template <typename WT>
+__device__ __forceinline__ float row_dot_ahead(const WT *__restrict__ wrow, const float *xs, size_t K, int lane, const uint4 (&pre)[8]) {
+    constexpr int VEC = 16 / sizeof(WT);
+    const size_t nv = K / VEC;
+    float acc = 0.f;
+#pragma unroll
+    for (int u = 0; u < 8; ++u) {
+        const size_t i = (size_t)u * 32 + lane;
+        if (i < nv) acc = vec_dot<WT>(pre[u], xs + i * VEC, acc);
+    }
+    for (size_t base = 256; base < nv; base += 256) {
+        uint4 wv[8];
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+            const size_t i = base + (size_t)u * 32 + lane;
+            wv[u] = i < nv ? ld_stream_u4(reinterpret_cast<const uint4 *>(wrow) + i) : make_uint4(0u, 0u, 0u, 0u);
+        }
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+            const size_t i = base + (size_t)u * 32 + lane;
+            if (i < nv) acc = vec_dot<WT>(wv[u], xs + i * VEC, acc);
+        }
+    }
+    return acc;
+}
+
 // RR rows of W against MB staged vectors at once: every 16 bytes of x read from shared memory feed RR rows, so
 // the shared-memory traffic per weight byte is MB / RR instead of MB (with MB = 8 and one row at a time the
 // kernel was bound by shared memory, not by HBM).  Vector path only (K % VEC == 0, 16-byte aligned rows).

@@ -63,6 +63,20 @@ __global__ void __launch_bounds__(kThreads) latent_absorb_kernel(const LatentArg
     __shared__ float part[kSlices][kAbsorbCols];
     const int tid = threadIdx.x;
     const size_t h = blockIdx.x, m = blockIdx.z;
+    // the first weight vectors of this thread are requested while the projections still run
+    constexpr int kAhead = 4, kQ = sizeof(T) / 2;
+    const int cg = tid % kColGroups, slice = tid / kColGroups;
+    const size_t r0 = (size_t)blockIdx.y * kAbsorbCols + cg * 8;
+    const T *w = static_cast<const T *>(a.wuk) + h * a.dim * a.rank + r0;
+    const bool vec = a.rank % 8 == 0, mine = (int)blockIdx.y < chunks && r0 < a.rank;
+    uint4 pre[kAhead][kQ];
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i)
+        if (vec && mine && slice + i * kSlices < a.dim)
+#pragma unroll
+            for (int k = 0; k < kQ; ++k) pre[i][k] = ld_stream_u4(reinterpret_cast<const uint4 *>(w + (slice + i * kSlices) * a.rank) + k);
+    pdl_launch();
+    pdl_wait();
     if ((int)blockIdx.y == chunks) {
         if (h == 0) append_row<T>(a, m, &part[0][0], tid);
         return;
@@ -74,28 +88,33 @@ __global__ void __launch_bounds__(kThreads) latent_absorb_kernel(const LatentArg
         for (size_t i = a.rank + tid; i < a.pitch; i += kThreads)
             out[i] = from_f32<T>(i < a.rank + a.rot_dim ? rotated(q + a.dim, i - a.rank, a.rot_dims, a.cos_t + pos * half, a.sin_t + pos * half) : 0.f);
     }
-    const int cg = tid % kColGroups, slice = tid / kColGroups;
-    const size_t r0 = (size_t)blockIdx.y * kAbsorbCols + cg * 8;
     float acc[8];
 #pragma unroll
     for (int j = 0; j < 8; ++j) acc[j] = 0.f;
-    const T *w = static_cast<const T *>(a.wuk) + h * a.dim * a.rank + r0;
-    if (a.rank % 8 == 0) {
-        if (r0 < a.rank) {
-#pragma unroll 4
-            for (size_t d = slice; d < a.dim; d += kSlices) {
-                const float x = q[d];
-                if constexpr (sizeof(T) == 4) {
-                    const float4 w0 = __ldcs(reinterpret_cast<const float4 *>(w + d * a.rank)), w1 = __ldcs(reinterpret_cast<const float4 *>(w + d * a.rank) + 1);
-                    acc[0] = fmaf(w0.x, x, acc[0]); acc[1] = fmaf(w0.y, x, acc[1]); acc[2] = fmaf(w0.z, x, acc[2]); acc[3] = fmaf(w0.w, x, acc[3]);
-                    acc[4] = fmaf(w1.x, x, acc[4]); acc[5] = fmaf(w1.y, x, acc[5]); acc[6] = fmaf(w1.z, x, acc[6]); acc[7] = fmaf(w1.w, x, acc[7]);
-                } else {
-                    const uint4 v = __ldcs(reinterpret_cast<const uint4 *>(w + d * a.rank));
-                    acc[0] = fmaf(bf16_lo(v.x), x, acc[0]); acc[1] = fmaf(bf16_hi(v.x), x, acc[1]);
-                    acc[2] = fmaf(bf16_lo(v.y), x, acc[2]); acc[3] = fmaf(bf16_hi(v.y), x, acc[3]);
-                    acc[4] = fmaf(bf16_lo(v.z), x, acc[4]); acc[5] = fmaf(bf16_hi(v.z), x, acc[5]);
-                    acc[6] = fmaf(bf16_lo(v.w), x, acc[6]); acc[7] = fmaf(bf16_hi(v.w), x, acc[7]);
+    if (vec) {
+        auto add = [&](const uint4 (&v)[kQ], float x) {
+            if constexpr (sizeof(T) == 4) {
+#pragma unroll
+                for (int k = 0; k < kQ; ++k) {
+                    acc[4 * k] = fmaf(__uint_as_float(v[k].x), x, acc[4 * k]); acc[4 * k + 1] = fmaf(__uint_as_float(v[k].y), x, acc[4 * k + 1]);
+                    acc[4 * k + 2] = fmaf(__uint_as_float(v[k].z), x, acc[4 * k + 2]); acc[4 * k + 3] = fmaf(__uint_as_float(v[k].w), x, acc[4 * k + 3]);
                 }
+            } else {
+                acc[0] = fmaf(bf16_lo(v[0].x), x, acc[0]); acc[1] = fmaf(bf16_hi(v[0].x), x, acc[1]);
+                acc[2] = fmaf(bf16_lo(v[0].y), x, acc[2]); acc[3] = fmaf(bf16_hi(v[0].y), x, acc[3]);
+                acc[4] = fmaf(bf16_lo(v[0].z), x, acc[4]); acc[5] = fmaf(bf16_hi(v[0].z), x, acc[5]);
+                acc[6] = fmaf(bf16_lo(v[0].w), x, acc[6]); acc[7] = fmaf(bf16_hi(v[0].w), x, acc[7]);
+            }
+        };
+        if (mine) {
+#pragma unroll
+            for (int i = 0; i < kAhead; ++i)
+                if (slice + i * kSlices < a.dim) add(pre[i], q[slice + i * kSlices]);
+            for (size_t d = slice + kAhead * kSlices; d < a.dim; d += kSlices) {
+                uint4 v[kQ];
+#pragma unroll
+                for (int k = 0; k < kQ; ++k) v[k] = ld_stream_u4(reinterpret_cast<const uint4 *>(w + d * a.rank) + k);
+                add(v, q[d]);
             }
         }
     } else {
@@ -129,6 +148,8 @@ __global__ void __launch_bounds__(kScoreWarps * 32) latent_scores_kernel(const L
     __shared__ float wm[kScoreWarps], wl[kScoreWarps];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int rank = (int)a.rank, width = (int)(a.rank + a.rot_dim);
+    pdl_wait();
+    pdl_launch();
     for (size_t row = blockIdx.y; row < a.B * a.S * a.H; row += gridDim.y) {
         const size_t m = row / a.H, b = m / a.S, past = (size_t)*a.d_len, total = past + a.S;
         const size_t seen = past + (m - b * a.S) + 1;
@@ -199,11 +220,20 @@ constexpr int kValueRows = 16;
 template <typename T>
 __global__ void __launch_bounds__(kThreads) latent_value_kernel(const LatentArgs a) {
     extern __shared__ __align__(16) float smem[];
-    float *ctx = smem;               // [rank]
-    float *f = ctx + ((a.rank + 3) & ~(size_t)3);  // [nsplit]
+    const size_t rank4 = (a.rank + 3) & ~(size_t)3;
+    float *ctx = smem;               // [2][rank4]: halves of the pieces, summed into the first
+    float *f = ctx + 2 * rank4;      // [nsplit]
     __shared__ float inv_s;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const size_t h = blockIdx.x, m = blockIdx.z, o = (m * a.H + h) * a.nsplit;
+    constexpr int VEC = 16 / sizeof(T);
+    const bool vec_ok = a.rank % VEC == 0;
+    const size_t v0 = (size_t)blockIdx.y * kValueRows + warp, v1 = min(a.vdim, (size_t)(blockIdx.y + 1) * kValueRows);
+    const T *w = static_cast<const T *>(a.wuv) + h * a.vdim * a.rank;
+    uint4 pre[8];
+    if (vec_ok && v0 < v1) row_ahead<T>(w + v0 * a.rank, a.rank, lane, pre);
+    pdl_launch();
+    pdl_wait();
     if (warp == 0) {
         float M = -INFINITY;
         for (int s = lane; s < a.nsplit; s += 32) M = fmaxf(M, a.part_ml[(o + s) * 2]);
@@ -220,21 +250,33 @@ __global__ void __launch_bounds__(kThreads) latent_value_kernel(const LatentArgs
     }
     __syncthreads();
     const float inv = inv_s;
-    for (size_t r = tid; r < a.rank; r += kThreads) {
-        float v = 0.f;
-#pragma unroll 4
-        for (int s = 0; s < a.nsplit; ++s)
-            if (f[s] != 0.f) v = fmaf(a.part_ctx[(o + s) * a.rank + r], f[s], v);
-        ctx[r] = v * inv;
+    if (a.rank % 4 == 0) {  // two groups of 128 threads, each with every other piece; a thread owns four adjacent columns
+        const int half = tid >> 7;
+        for (size_t c = tid & 127; c < a.rank / 4; c += 128) {
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+            for (int s = half; s < a.nsplit; s += 2) {
+                const float4 p = reinterpret_cast<const float4 *>(a.part_ctx + (o + s) * a.rank)[c];
+                const float w = f[s];
+                v.x = fmaf(p.x, w, v.x); v.y = fmaf(p.y, w, v.y); v.z = fmaf(p.z, w, v.z); v.w = fmaf(p.w, w, v.w);
+            }
+            reinterpret_cast<float4 *>(ctx + half * rank4)[c] = make_float4(v.x * inv, v.y * inv, v.z * inv, v.w * inv);
+        }
+        __syncthreads();
+        for (size_t r = tid; r < a.rank; r += kThreads) ctx[r] += ctx[rank4 + r];
+    } else {
+        for (size_t r = tid; r < a.rank; r += kThreads) {
+            float v = 0.f;
+            for (int s = 0; s < a.nsplit; ++s) v = fmaf(a.part_ctx[(o + s) * a.rank + r], f[s], v);
+            ctx[r] = v * inv;
+        }
     }
     __syncthreads();
     const float gate = sigmoid_f(a.u[m * a.u_ld + a.u_gate + h]);
-    constexpr int VEC = 16 / sizeof(T);
-    const bool vec_ok = a.rank % VEC == 0;
-    const size_t v1 = min(a.vdim, (size_t)(blockIdx.y + 1) * kValueRows);
-    for (size_t v = (size_t)blockIdx.y * kValueRows + warp; v < v1; v += kWarps) {
+    for (size_t v = v0; v < v1; v += kWarps) {
         float acc[1] = {0.f};
-        row_dot<T, 1>(static_cast<const T *>(a.wuv) + (h * a.vdim + v) * a.rank, ctx, a.rank, lane, vec_ok, acc);
+        if (vec_ok && v == v0) acc[0] = row_dot_ahead<T>(w + v * a.rank, ctx, a.rank, lane, pre);
+        else row_dot<T, 1>(w + v * a.rank, ctx, a.rank, lane, vec_ok, acc);
         const float y = warp_sum(acc[0]) * gate;
         if (lane == 0) {
             const size_t at = (m * a.H + h) * a.vdim + v;
@@ -251,14 +293,12 @@ int launch_scores_t(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s) {
 #define LUMEN_SCORES(NI_)                                                                                                                \
     do {                                                                                                                                 \
         if (smem > 48 * 1024) LUMEN_CUDA(ctx, cudaFuncSetAttribute(latent_scores_kernel<T, NI_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
-        latent_scores_kernel<T, NI_><<<grid, kScoreWarps * 32, smem, s>>>(a);                                                            \
+        return launch_pdl(ctx, latent_scores_kernel<T, NI_>, grid, kScoreWarps * 32, smem, s, a);                                         \
     } while (0)
     if (a.rank <= 128) LUMEN_SCORES(4);
-    else if (a.rank <= 512) LUMEN_SCORES(16);
-    else LUMEN_SCORES(32);
+    if (a.rank <= 512) LUMEN_SCORES(16);
+    LUMEN_SCORES(32);
 #undef LUMEN_SCORES
-    LUMEN_LAUNCHED(ctx);
-    return LUMEN_OK;
 }
 
 }  // namespace
@@ -275,10 +315,7 @@ int launch_latent_absorb(lumen_ctx *ctx, const LatentArgs &a, bool append, cudaS
     if (rows > 65535) return set_error(ctx, LUMEN_ERR_UNSUPPORTED, "latent attention: %zu rows in one step", rows);
     const int chunks = (int)((a.rank + kAbsorbCols - 1) / kAbsorbCols);
     const dim3 grid((unsigned)a.H, (unsigned)(chunks + (append ? 1 : 0)), (unsigned)rows);
-    if (a.dt == LUMEN_F32) latent_absorb_kernel<float><<<grid, kThreads, 0, s>>>(a, chunks);
-    else latent_absorb_kernel<__nv_bfloat16><<<grid, kThreads, 0, s>>>(a, chunks);
-    LUMEN_LAUNCHED(ctx);
-    return LUMEN_OK;
+    return launch_pdl(ctx, a.dt == LUMEN_F32 ? latent_absorb_kernel<float> : latent_absorb_kernel<__nv_bfloat16>, grid, kThreads, 0, s, a, chunks);
 }
 
 int launch_latent_scores(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s) {
@@ -289,12 +326,9 @@ int launch_latent_scores(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s) {
 int launch_latent_value(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s) {
     const size_t rows = a.B * a.S;
     if (rows > 65535) return set_error(ctx, LUMEN_ERR_UNSUPPORTED, "latent attention: %zu rows in one step", rows);
-    const size_t smem = (((a.rank + 3) & ~(size_t)3) + a.nsplit) * sizeof(float);
+    const size_t smem = (2 * ((a.rank + 3) & ~(size_t)3) + a.nsplit) * sizeof(float);
     const dim3 grid((unsigned)a.H, (unsigned)((a.vdim + kValueRows - 1) / kValueRows), (unsigned)rows);
-    if (a.dt == LUMEN_F32) latent_value_kernel<float><<<grid, kThreads, smem, s>>>(a);
-    else latent_value_kernel<__nv_bfloat16><<<grid, kThreads, smem, s>>>(a);
-    LUMEN_LAUNCHED(ctx);
-    return LUMEN_OK;
+    return launch_pdl(ctx, a.dt == LUMEN_F32 ? latent_value_kernel<float> : latent_value_kernel<__nv_bfloat16>, grid, kThreads, smem, s, a);
 }
 
 }  // namespace lumen

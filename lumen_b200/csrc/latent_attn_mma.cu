@@ -63,6 +63,8 @@ __global__ void __launch_bounds__(kThreads, 1) latent_attn_mma_kernel(const Late
     __nv_bfloat16 *ph = reinterpret_cast<__nv_bfloat16 *>(smem + g.p), *pl = ph + kRows * kLdP;
     float *m_s = reinterpret_cast<float *>(smem + g.stats), *l_s = m_s + kRows, *f_s = l_s + kRows;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    pdl_wait();
+    pdl_launch();
     const int H = (int)a.H, n_rows = (int)(a.S * a.H), row0 = blockIdx.y * kRows, b = blockIdx.z, split = blockIdx.x;
     const int past = *a.d_len, total = past + (int)a.S;
     const int tiles_all = (total + kBN - 1) / kBN, per = (tiles_all + a.nsplit - 1) / a.nsplit;
@@ -272,9 +274,8 @@ int launch_t(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s) {
         set[dev] = smem;
     }
     const size_t rows = a.S * a.H;
-    latent_attn_mma_kernel<MT, NT><<<dim3((unsigned)a.nsplit, (unsigned)((rows + MT * 16 - 1) / (MT * 16)), (unsigned)a.B), kThreads, smem, s>>>(a);
-    LUMEN_LAUNCHED(ctx);
-    return LUMEN_OK;
+    return launch_pdl(ctx, latent_attn_mma_kernel<MT, NT>, dim3((unsigned)a.nsplit, (unsigned)((rows + MT * 16 - 1) / (MT * 16)), (unsigned)a.B), kThreads,
+                      smem, s, a);
 }
 
 constexpr size_t kSmemLimit = 227 * 1024;
@@ -298,8 +299,8 @@ int latent_pick_splits(const LatentArgs &a, size_t total, int num_sms) {
     const size_t rows = a.S * a.H, blocks = a.B * (mma ? (rows + row_tiles(a) * 16 - 1) / (row_tiles(a) * 16) : rows);
     const size_t want = std::min<size_t>({(total + kBN - 1) / kBN, std::max<size_t>(1, (size_t)num_sms * (mma ? 1 : 8) / std::max<size_t>(blocks, 1)), 64});
     int n = 1;
-    while ((size_t)n < want) n <<= 1;
-    return std::min(n, 64);
+    while ((size_t)n * 2 <= want) n <<= 1;
+    return n;
 }
 
 int launch_latent_mma(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s) {

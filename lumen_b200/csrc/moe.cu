@@ -55,6 +55,8 @@ __global__ void __launch_bounds__(kThreads) moe_gate_up_kernel(const MoeArgs a) 
     const size_t m = blockIdx.y, K = a.W;
     float *xs = smem, *sc = xs + ((K + 3) & ~(size_t)3), *weight = sc + E;
     int *sel = reinterpret_cast<int *>(weight + top);
+    pdl_launch();
+    pdl_wait();
     for (size_t k = tid; k < K; k += kThreads) xs[k] = a.x[m * K + k];
     for (int e = tid; e < E; e += kThreads) sc[e] = sigmoid_f(a.z[m * E + e]);
     __syncthreads();
@@ -99,6 +101,8 @@ __global__ void __launch_bounds__(kThreads) moe_down_kernel(const MoeArgs a) {
     const int top = (int)a.top;
     const size_t m = blockIdx.y, ff4 = (a.ff + 3) & ~(size_t)3;
     const size_t routed = (size_t)top * a.ff, total = routed + a.shared_ff;
+    pdl_launch();
+    pdl_wait();
     for (size_t i = tid; i < total; i += kThreads) {
         const size_t slot = i < routed ? i / a.ff : (size_t)top;
         act[slot * ff4 + (i - slot * a.ff)] = a.act[m * total + i];
@@ -108,6 +112,33 @@ __global__ void __launch_bounds__(kThreads) moe_down_kernel(const MoeArgs a) {
     const bool vec_ok = a.ff % VEC == 0, svec_ok = a.shared_ff % VEC == 0;
     for (size_t n = (size_t)blockIdx.x * kWarps + warp; n < a.W; n += (size_t)gridDim.x * kWarps) {
         float acc[1] = {0.f};
+        if (vec_ok && svec_ok) {  // the experts' rows and the shared one as one sequence of vectors, eight in flight per lane
+            const size_t nv = a.ff / VEC, routed_v = nv * top, all = routed_v + a.shared_ff / VEC;
+            for (size_t base = 0; base < all; base += 256) {
+                uint4 wv[8];
+                const float *xp[8];
+#pragma unroll
+                for (int u = 0; u < 8; ++u) {
+                    const size_t i = base + (size_t)u * 32 + lane;
+                    xp[u] = nullptr;
+                    if (i < routed_v) {
+                        const unsigned slot = (unsigned)i / (unsigned)nv, at = (unsigned)i - slot * (unsigned)nv;
+                        const size_t e = (size_t)a.sel[m * top + slot];
+                        wv[u] = ld_stream_u4(reinterpret_cast<const uint4 *>(static_cast<const WT *>(a.down) + (e * a.W + n) * a.ff) + at);
+                        xp[u] = act + slot * ff4 + at * VEC;
+                    } else if (i < all) {
+                        wv[u] = ld_stream_u4(reinterpret_cast<const uint4 *>(static_cast<const WT *>(a.shared_down) + n * a.shared_ff) + (i - routed_v));
+                        xp[u] = act + top * ff4 + (i - routed_v) * VEC;
+                    }
+                }
+#pragma unroll
+                for (int u = 0; u < 8; ++u)
+                    if (xp[u]) acc[0] = vec_dot<WT>(wv[u], xp[u], acc[0]);
+            }
+            const float v = warp_sum(acc[0]);
+            if (lane == 0) a.y[m * a.W + n] = v;
+            continue;
+        }
         for (int k = 0; k < top; ++k) {
             const size_t e = (size_t)a.sel[m * top + k];
             row_dot<WT, 1>(static_cast<const WT *>(a.down) + (e * a.W + n) * a.ff, act + k * ff4, a.ff, lane, vec_ok, acc);
@@ -178,11 +209,8 @@ int launch_vec_t(lumen_ctx *ctx, const MoeArgs &a, cudaStream_t s) {
         const size_t per_sm = std::max<size_t>(1, std::min<size_t>(8, 227 * 1024 / (smem + 1024)));
         return (unsigned)std::max<size_t>(1, std::min((rows + kWarps - 1) / kWarps, (size_t)ctx->num_sms * per_sm));
     };
-    moe_gate_up_kernel<WT><<<dim3(blocks(a.top * a.ff + a.shared_ff, s1), (unsigned)a.M), kThreads, s1, s>>>(a);
-    LUMEN_LAUNCHED(ctx);
-    moe_down_kernel<WT><<<dim3(blocks(a.W, s2), (unsigned)a.M), kThreads, s2, s>>>(a);
-    LUMEN_LAUNCHED(ctx);
-    return LUMEN_OK;
+    LUMEN_TRY(launch_pdl(ctx, moe_gate_up_kernel<WT>, dim3(blocks(a.top * a.ff + a.shared_ff, s1), (unsigned)a.M), kThreads, s1, s, a));
+    return launch_pdl(ctx, moe_down_kernel<WT>, dim3(blocks(a.W, s2), (unsigned)a.M), kThreads, s2, s, a);
 }
 
 }  // namespace

@@ -4,7 +4,7 @@ from __future__ import annotations
 import numpy as np
 
 
-def mixer(heads=3, dim=24, rot_dim=8, vdim=40, kv_rank=48, rot_dims=None, base=500.0, scale=0.2):
+def mixer(heads=3, dim=24, rot_dim=8, vdim=40, kv_rank=48, rot_dims=None, base=500.0, scale=0.1):
     return dict(heads=heads, dim=dim, rot_dim=rot_dim, vdim=vdim, kv_rank=kv_rank, scale=scale,
                 rot=dict(base=base, dims=rot_dim if rot_dims is None else rot_dims))
 
@@ -79,3 +79,17 @@ def row_err(got, want):
     d -= d.mean(-1, keepdims=True)
     w = want - want.mean(-1, keepdims=True)
     return np.sqrt((d * d).mean(-1)) / np.sqrt((w * w).mean())
+
+
+FLOOR = {"f32": 4e-6, "bf16": 6e-3}
+
+
+def tolerance(ids, cfg, p, dtype, want, rows=None):
+    """Three times what rounding alone does to this model and these tokens (see row_err), and at least a floor."""
+    import fegetar_plain as plain
+    if dtype == "f32":
+        near = plain.forward(ids, cfg, p, dtype=np.float32)
+    else:
+        near = plain.forward(ids, cfg, p, rounding=plain.to_bf16)
+    err = row_err(near, want)
+    return max(3 * float((err if rows is None else err[rows]).max()), FLOOR[dtype])

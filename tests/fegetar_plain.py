@@ -3,10 +3,25 @@ code shared with the product.  Test infrastructure.
 
 `cfg` is a config.json dictionary, `p` the parameters by name.  `without` plants one mistake (its name) so that a test can
 show that the mistake would be seen.
+
+`forward` can also run in float32, or with the input of every product rounded to bfloat16: what these two differ from the
+float64 result by is the error that rounding alone causes in a model, and the measure of the tests' tolerances.
 """
 from __future__ import annotations
 
 import numpy as np
+
+_ROUND = None  # applied to the inputs of products (None: exact)
+
+
+def product(x, w):
+    return (x if _ROUND is None else _ROUND(x)) @ w.T
+
+
+def to_bf16(x):
+    u = np.ascontiguousarray(x, dtype=np.float32).view(np.uint32)
+    u = (u + np.uint32(0x7FFF) + ((u >> np.uint32(16)) & np.uint32(1))) & np.uint32(0xFFFF0000)
+    return u.view(np.float32).reshape(np.shape(x)).astype(np.asarray(x).dtype)
 
 
 def rms_norm(x, gain, eps):
@@ -49,15 +64,15 @@ def latent_attention(h, m, p, pre, eps, without=None, hidden_key=None):
     """`hidden_key`: a position that nobody but itself sees (a planted mistake)."""
     T, H, d, r, vd, rank = len(h), m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
     pos = np.arange(T)
-    q = (h @ p[pre + "q"].T).reshape(T, H, d + r)
-    down = h @ p[pre + "dkv"].T
+    q = (product(h, p[pre + "q"])).reshape(T, H, d + r)
+    down = product(h, p[pre + "dkv"])
     c = down[:, :rank] if without == "latent norm" else rms_norm(down[:, :rank], p[pre + "dkv.norm"], eps)
     k_rot = rotate(down[:, rank:], pos, m["rot"], without)
     q_rot = rotate(q[..., d:], pos, m["rot"], None if without == "position" else without)
-    k = (c @ p[pre + "uk"].T).reshape(T, H, d)
-    v = (c @ p[pre + "uv"].T).reshape(T, H, vd)
-    gate = sigmoid(h @ p[pre + "g"].T)
-    out = np.zeros((T, H, vd))
+    k = product(c, p[pre + "uk"]).reshape(T, H, d)
+    v = product(c, p[pre + "uv"]).reshape(T, H, vd)
+    gate = sigmoid(product(h, p[pre + "g"]))
+    out = np.zeros((T, H, vd), h.dtype)
     for i in range(T):
         s = (np.einsum("hd,jhd->hj", q[i, :, :d], k[:i + 1]) + np.einsum("hr,jr->hj", q_rot[i], k_rot[:i + 1])) * m["scale"]
         if hidden_key is not None and hidden_key < i:
@@ -67,17 +82,17 @@ def latent_attention(h, m, p, pre, eps, without=None, hidden_key=None):
         out[i] = np.einsum("hj,jhv->hv", w, v[:i + 1])
         if without != "gate":
             out[i] *= gate[i][:, None]
-    return out.reshape(T, H * vd) @ p[pre + "o"].T
+    return product(out.reshape(T, H * vd), p[pre + "o"])
 
 
 def dense(h, p, pre):
-    return gelu_tanh(h @ p[pre + "up"].T) @ p[pre + "down"].T
+    return product(gelu_tanh(product(h, p[pre + "up"])), p[pre + "down"])
 
 
 def expert(h, p, pre, limit):
-    g = np.minimum(h @ p[pre + ".gate"].T, limit)
-    u = np.clip(h @ p[pre + ".up"].T, -limit, limit)
-    return (g * sigmoid(1.702 * g) * (u + 1)) @ p[pre + ".down"].T
+    g = np.minimum(product(h, p[pre + ".gate"]), limit)
+    u = np.clip(product(h, p[pre + ".up"]), -limit, limit)
+    return product(g * sigmoid(1.702 * g) * (u + 1), p[pre + ".down"])
 
 
 def router_scores(h, p, pre):
@@ -101,14 +116,23 @@ def moe(h, mlp, p, pre, without=None):
 
 def side_input(x, tokens, layer, dim, p, pre, eps):
     e = p["side.embed"][tokens][:, layer * dim:(layer + 1) * dim]
-    y = (gelu_tanh(x @ p[pre + "gate"].T) * e) @ p[pre + "proj"].T
+    y = product(gelu_tanh(product(x, p[pre + "gate"])) * e, p[pre + "proj"])
     return rms_norm(y, p[pre + "norm"], eps)
 
 
-def forward(tokens, cfg, p, without=None, hidden_key=None, streams=None):
-    """Logits [T, vocab] of one sequence.  `streams`: a list that receives the residual after every layer."""
+def forward(tokens, cfg, p, without=None, hidden_key=None, dtype=np.float64, rounding=None):
+    """Logits [T, vocab] of one sequence."""
+    global _ROUND
     tokens = np.asarray(tokens, dtype=np.int64)
-    p = {k: np.asarray(v, dtype=np.float64) for k, v in p.items()}
+    p = {k: np.asarray(v, dtype=dtype) for k, v in p.items()}
+    _ROUND = rounding
+    try:
+        return _forward(tokens, cfg, p, without, hidden_key)
+    finally:
+        _ROUND = None
+
+
+def _forward(tokens, cfg, p, without, hidden_key):
     eps = cfg["norm"]["eps"]
     x = embed_tokens(tokens, cfg, p, without)
     for i, layer in enumerate(cfg["layers"]):
@@ -122,6 +146,4 @@ def forward(tokens, cfg, p, without=None, hidden_key=None, streams=None):
             x = x + rms_norm(y, one + p[pre + "norm2"], eps)
         if cfg.get("token_side") and without != "side":
             x = x + side_input(x, tokens, i, cfg["token_side"]["dim"], p, pre + "side.", eps)
-        if streams is not None:
-            streams.append(x)
     return rms_norm(x, 1.0 + p["final.norm"], eps) @ p["head"].T

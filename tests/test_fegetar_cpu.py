@@ -20,7 +20,7 @@ def test_config_reader_takes_every_size(L):
     assert (c.bigram_buckets, c.bigram_mul_prev, c.bigram_mul_cur) == (37, 5, 3)
     a, b, n = c.layers[0], c.layers[1], c.layers[2]
     assert (a.heads, a.dim, a.rot_dim, a.vdim, a.kv_rank, a.rot_dims, a.rot_base, a.mlp_kind, a.ff) == (3, 24, 8, 40, 48, 8, 500.0, 1, 88)
-    assert a.scale == pytest.approx(0.2)
+    assert a.scale == pytest.approx(0.1)
     assert (b.heads, b.rot_dims, b.mlp_kind, b.experts, b.top, b.expert_ff, b.shared_ff) == (2, 4, 2, 6, 2, 40, 56)
     assert (b.expert_limit, b.shared_limit) == (1.5, pytest.approx(0.8))
     assert n.mlp_kind == 0 and n.kv_rank == 40
