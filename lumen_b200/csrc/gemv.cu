@@ -169,19 +169,23 @@ gemv_gate_up_kernel(const float *__restrict__ x, const WT *__restrict__ wg, cons
 }
 
 // One row whose input may still owe the norm of a sublayer's output (post-norm models): x = res + RMSNorm(y) * gain is
-// formed by every CTA while it stages x, so that the norm, the residual sum and the product are one launch.
-template <typename WT>
+// formed by every CTA while it stages x, so that the norm, the residual sum and the product are one launch.  WPR warps share a
+// weight row (a slice of K each) where there are too few rows to keep enough loads in flight.
+template <typename WT, int WPR>
 __global__ void __launch_bounds__(kThreads) gemv_step_kernel(const GemvStepArgs a) {
     extern __shared__ __align__(16) float smem[];
     __shared__ float red[kWarps];
     float *xs = smem;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const size_t K = a.K, row0 = (size_t)blockIdx.x * kWarps + warp;
+    constexpr int VEC = 16 / sizeof(WT), kRows = kWarps / WPR;
+    const int part = warp % WPR;
+    const size_t K = a.K, row0 = (size_t)blockIdx.x * kRows + warp / WPR;
     const WT *w = static_cast<const WT *>(a.w);
-    constexpr int VEC = 16 / sizeof(WT);
     const bool vec_ok = (K % VEC == 0) && ((reinterpret_cast<uintptr_t>(w) & 15) == 0);
+    // this warp's slice of K, in whole vectors
+    const size_t per = (K / VEC + WPR - 1) / WPR * VEC, k0 = min(K, part * per), kn = min(K - k0, per);
     uint4 pre[8];
-    if (vec_ok && row0 < a.N) row_ahead<WT>(w + row0 * K, K, lane, pre);
+    if (vec_ok && row0 < a.N) row_ahead<WT>(w + row0 * K + k0, kn, lane, pre);
     pdl_launch();
     pdl_wait();
     auto inv_rms = [&](float ss) {
@@ -251,12 +255,28 @@ __global__ void __launch_bounds__(kThreads) gemv_step_kernel(const GemvStepArgs 
         for (size_t k = tid; k < K; k += kThreads) xs[k] = __fmul_rn(__fmul_rn(xs[k], inv), a.norm_w[k]);
     }
     __syncthreads();
-    for (size_t row = row0; row < a.N; row += (size_t)gridDim.x * kWarps) {
+    for (size_t base = (size_t)blockIdx.x * kRows; base < a.N; base += (size_t)gridDim.x * kRows) {
+        const size_t row = base + warp / WPR;
         float acc[1] = {0.f};
-        if (vec_ok && row == row0) acc[0] = row_dot_ahead<WT>(w + row * K, xs, K, lane, pre);
-        else row_dot<WT, 1>(w + row * K, xs, K, lane, vec_ok, acc);
+        if (row < a.N) {
+            if (!vec_ok) {
+                if (part == 0) row_dot<WT, 1>(w + row * K, xs, K, lane, false, acc);
+            } else if (row == row0) {
+                acc[0] = row_dot_ahead<WT>(w + row * K + k0, xs + k0, kn, lane, pre);
+            } else {
+                row_dot<WT, 1>(w + row * K + k0, xs + k0, kn, lane, true, acc);
+            }
+        }
         float v = warp_sum(acc[0]);
-        if (lane == 0) {
+        if (WPR > 1) {  // the row's slices meet in its first warp
+            if (lane == 0) red[warp] = v;
+            __syncthreads();
+            v = 0.f;
+#pragma unroll
+            for (int i = 0; i < WPR; ++i) v += red[(warp / WPR) * WPR + i];
+            __syncthreads();
+        }
+        if (lane == 0 && part == 0 && row < a.N) {
             if (a.act != StepFinish::kStore) v = gelu_tanh(v);
             if (a.act == StepFinish::kSideGate) {
                 const unsigned long long tok = id_to_index(a.ids[0]);
@@ -439,13 +459,24 @@ int launch_gemv_gate_up(lumen_ctx *ctx, const float *x, const void *w_gate, cons
 int launch_gemv_step(lumen_ctx *ctx, const GemvStepArgs &a, cudaStream_t s) {
     const size_t smem = a.K * sizeof(float);
     if (smem > 200 * 1024) return set_error(ctx, LUMEN_ERR_UNSUPPORTED, "gemv_step: row of %zu elements", a.K);
-    const int grid = pick_grid(ctx, a.N, smem);
+    // warps per row: enough warps for about three CTAs per SM, a slice of at least 1 KB each
+    const size_t row_bytes = a.K * (a.wdt == LUMEN_F32 ? 4 : 2), want = (size_t)ctx->num_sms * 3 * kWarps;
+    const int wpr = a.N * 4 <= want && row_bytes >= 4096 ? 4 : a.N * 2 <= want && row_bytes >= 2048 ? 2 : row_bytes >= 8192 && a.N * 2 <= 2 * want ? 2 : 1;
+    const int grid = pick_grid(ctx, a.N * wpr, smem);
+#define LUMEN_STEP(T_, W_)                                                                     \
+    do {                                                                                       \
+        LUMEN_TRY(set_smem(ctx, gemv_step_kernel<T_, W_>, smem));                              \
+        return launch_pdl(ctx, gemv_step_kernel<T_, W_>, grid, kThreads, smem, s, a);          \
+    } while (0)
     if (a.wdt == LUMEN_F32) {
-        LUMEN_TRY(set_smem(ctx, gemv_step_kernel<float>, smem));
-        return launch_pdl(ctx, gemv_step_kernel<float>, grid, kThreads, smem, s, a);
+        if (wpr == 4) LUMEN_STEP(float, 4);
+        if (wpr == 2) LUMEN_STEP(float, 2);
+        LUMEN_STEP(float, 1);
     }
-    LUMEN_TRY(set_smem(ctx, gemv_step_kernel<__nv_bfloat16>, smem));
-    return launch_pdl(ctx, gemv_step_kernel<__nv_bfloat16>, grid, kThreads, smem, s, a);
+    if (wpr == 4) LUMEN_STEP(__nv_bfloat16, 4);
+    if (wpr == 2) LUMEN_STEP(__nv_bfloat16, 2);
+    LUMEN_STEP(__nv_bfloat16, 1);
+#undef LUMEN_STEP
 }
 
 size_t gemv_kn_scratch_bytes_for(size_t K, size_t N, lumen_dtype wdt, int num_sms) {

@@ -67,10 +67,10 @@ __global__ void __launch_bounds__(kThreads, 1) latent_attn_mma_kernel(const Late
     pdl_launch();
     const int H = (int)a.H, n_rows = (int)(a.S * a.H), row0 = blockIdx.y * kRows, b = blockIdx.z, split = blockIdx.x;
     const int past = *a.d_len, total = past + (int)a.S;
-    const int tiles_all = (total + kBN - 1) / kBN, per = (tiles_all + a.nsplit - 1) / a.nsplit;
+    const int tiles_all = (total + kBN - 1) / kBN;
     // the last query row of this block sees up to past + its position
     const int seen = past + min(row0 + kRows - 1, n_rows - 1) / H + 1;
-    const int j0 = split * per * kBN, j1 = min(seen, j0 + per * kBN);
+    const int j0 = (int)((long long)split * tiles_all / a.nsplit) * kBN, j1 = min(seen, (int)((long long)(split + 1) * tiles_all / a.nsplit) * kBN);
     const int nt = j1 > j0 ? (j1 - j0 + kBN - 1) / kBN : 0;
     const __nv_bfloat16 *cache = static_cast<const __nv_bfloat16 *>(a.cache) + (size_t)b * a.max_seq * pitch;
     const int vec = pitch / 8;

@@ -94,58 +94,75 @@ __global__ void __launch_bounds__(kThreads) moe_gate_up_kernel(const MoeArgs a) 
     }
 }
 
+// Four warps share an output row: the chosen experts' rows and the shared one form one sequence of vectors.
+constexpr int kDownWarps = 4, kDownRows = kWarps / kDownWarps;
 template <typename WT>
 __global__ void __launch_bounds__(kThreads) moe_down_kernel(const MoeArgs a) {
-    extern __shared__ __align__(16) float act[];  // every expert's activations, each on a 16-byte boundary
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int top = (int)a.top;
-    const size_t m = blockIdx.y, ff4 = (a.ff + 3) & ~(size_t)3;
-    const size_t routed = (size_t)top * a.ff, total = routed + a.shared_ff;
+    extern __shared__ __align__(16) float act[];  // every expert's activations, each on a 16-byte boundary; then the experts' numbers
+    __shared__ float red[kWarps];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, part = warp % kDownWarps;
+    const int top = (int)a.top, ff = (int)a.ff, sff = (int)a.shared_ff, ff4 = (ff + 3) & ~3;
+    const size_t m = blockIdx.y, total = (size_t)top * ff + sff;
+    int *sel = reinterpret_cast<int *>(act + top * ff4 + ((sff + 3) & ~3));
+    constexpr int VEC = 16 / sizeof(WT);
+    const bool vec_ok = ff % VEC == 0 && sff % VEC == 0;
     pdl_launch();
     pdl_wait();
-    for (size_t i = tid; i < total; i += kThreads) {
-        const size_t slot = i < routed ? i / a.ff : (size_t)top;
-        act[slot * ff4 + (i - slot * a.ff)] = a.act[m * total + i];
+    const float *src = a.act + m * total;
+    if (ff4 == ff && total % 4 == 0) {
+        for (size_t i = tid; i < total / 4; i += kThreads) reinterpret_cast<float4 *>(act)[i] = reinterpret_cast<const float4 *>(src)[i];
+    } else {
+        for (int k = 0; k <= top; ++k)
+            for (int i = tid; i < (k < top ? ff : sff); i += kThreads) act[k * ff4 + i] = src[k * ff + i];
     }
+    if (tid < top) sel[tid] = a.sel[m * top + tid];
+    for (int k = kThreads + tid; k < top; k += kThreads) sel[k] = a.sel[m * top + k];
     __syncthreads();
-    constexpr int VEC = 16 / sizeof(WT);
-    const bool vec_ok = a.ff % VEC == 0, svec_ok = a.shared_ff % VEC == 0;
-    for (size_t n = (size_t)blockIdx.x * kWarps + warp; n < a.W; n += (size_t)gridDim.x * kWarps) {
+    const unsigned nv = (unsigned)(ff / VEC), routed = nv * top, all = routed + (unsigned)(sff / VEC);
+    for (size_t base = (size_t)blockIdx.x * kDownRows; base < a.W; base += (size_t)gridDim.x * kDownRows) {
+        const size_t n = base + warp / kDownWarps;
         float acc[1] = {0.f};
-        if (vec_ok && svec_ok) {  // the experts' rows and the shared one as one sequence of vectors, eight in flight per lane
-            const size_t nv = a.ff / VEC, routed_v = nv * top, all = routed_v + a.shared_ff / VEC;
-            for (size_t base = 0; base < all; base += 256) {
-                uint4 wv[8];
-                const float *xp[8];
+        if (n < a.W) {
+            const WT *shared_row = static_cast<const WT *>(a.shared_down) + n * sff;
+            if (vec_ok) {
+                for (unsigned i0 = part * 256; i0 < all; i0 += kDownWarps * 256) {
+                    uint4 wv[8];
+                    unsigned xo[8];
 #pragma unroll
-                for (int u = 0; u < 8; ++u) {
-                    const size_t i = base + (size_t)u * 32 + lane;
-                    xp[u] = nullptr;
-                    if (i < routed_v) {
-                        const unsigned slot = (unsigned)i / (unsigned)nv, at = (unsigned)i - slot * (unsigned)nv;
-                        const size_t e = (size_t)a.sel[m * top + slot];
-                        wv[u] = ld_stream_u4(reinterpret_cast<const uint4 *>(static_cast<const WT *>(a.down) + (e * a.W + n) * a.ff) + at);
-                        xp[u] = act + slot * ff4 + at * VEC;
-                    } else if (i < all) {
-                        wv[u] = ld_stream_u4(reinterpret_cast<const uint4 *>(static_cast<const WT *>(a.shared_down) + n * a.shared_ff) + (i - routed_v));
-                        xp[u] = act + top * ff4 + (i - routed_v) * VEC;
+                    for (int u = 0; u < 8; ++u) {
+                        const unsigned i = i0 + u * 32 + lane;
+                        xo[u] = 0;
+                        wv[u] = make_uint4(0u, 0u, 0u, 0u);
+                        if (i < routed) {
+                            const unsigned slot = i / nv, at = i - slot * nv;
+                            wv[u] = ld_stream_u4(reinterpret_cast<const uint4 *>(static_cast<const WT *>(a.down) + ((size_t)sel[slot] * a.W + n) * ff) + at);
+                            xo[u] = slot * ff4 + at * VEC;
+                        } else if (i < all) {
+                            wv[u] = ld_stream_u4(reinterpret_cast<const uint4 *>(shared_row) + (i - routed));
+                            xo[u] = top * ff4 + (i - routed) * VEC;
+                        }
                     }
-                }
 #pragma unroll
-                for (int u = 0; u < 8; ++u)
-                    if (xp[u]) acc[0] = vec_dot<WT>(wv[u], xp[u], acc[0]);
+                    for (int u = 0; u < 8; ++u)
+                        if (i0 + u * 32 + lane < all) acc[0] = vec_dot<WT>(wv[u], act + xo[u], acc[0]);
+                }
+            } else {
+                for (int k = part; k <= top; k += kDownWarps) {
+                    if (k < top) row_dot<WT, 1>(static_cast<const WT *>(a.down) + ((size_t)sel[k] * a.W + n) * ff, act + k * ff4, ff, lane, false, acc);
+                    else if (sff) row_dot<WT, 1>(shared_row, act + top * ff4, sff, lane, false, acc);
+                }
             }
-            const float v = warp_sum(acc[0]);
-            if (lane == 0) a.y[m * a.W + n] = v;
-            continue;
         }
-        for (int k = 0; k < top; ++k) {
-            const size_t e = (size_t)a.sel[m * top + k];
-            row_dot<WT, 1>(static_cast<const WT *>(a.down) + (e * a.W + n) * a.ff, act + k * ff4, a.ff, lane, vec_ok, acc);
-        }
-        if (a.shared_ff) row_dot<WT, 1>(static_cast<const WT *>(a.shared_down) + n * a.shared_ff, act + top * ff4, a.shared_ff, lane, svec_ok, acc);
         const float v = warp_sum(acc[0]);
-        if (lane == 0) a.y[m * a.W + n] = v;
+        if (lane == 0) red[warp] = v;
+        __syncthreads();
+        if (lane == 0 && part == 0 && n < a.W) {
+            float y = 0.f;
+#pragma unroll
+            for (int i = 0; i < kDownWarps; ++i) y += red[warp + i];
+            a.y[m * a.W + n] = y;
+        }
+        __syncthreads();
     }
 }
 
@@ -198,19 +215,19 @@ __global__ void __launch_bounds__(128) gather_rows_kernel(const __nv_bfloat16 *_
 }
 
 size_t gate_up_smem(const MoeArgs &a) { return (((a.W + 3) & ~(size_t)3) + a.experts + 2 * a.top) * sizeof(float); }
-size_t down_smem(const MoeArgs &a) { return (a.top * ((a.ff + 3) & ~(size_t)3) + a.shared_ff + 4) * sizeof(float); }
+size_t down_smem(const MoeArgs &a) { return (a.top * (((a.ff + 3) & ~(size_t)3) + 1) + a.shared_ff + 4) * sizeof(float); }
 
 template <typename WT>
 int launch_vec_t(lumen_ctx *ctx, const MoeArgs &a, cudaStream_t s) {
     const size_t s1 = gate_up_smem(a), s2 = down_smem(a);
     if (s1 > 48 * 1024) LUMEN_CUDA(ctx, cudaFuncSetAttribute(moe_gate_up_kernel<WT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1));
     if (s2 > 48 * 1024) LUMEN_CUDA(ctx, cudaFuncSetAttribute(moe_down_kernel<WT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2));
-    auto blocks = [&](size_t rows, size_t smem) {
+    auto blocks = [&](size_t rows, size_t smem, size_t per_cta) {
         const size_t per_sm = std::max<size_t>(1, std::min<size_t>(8, 227 * 1024 / (smem + 1024)));
-        return (unsigned)std::max<size_t>(1, std::min((rows + kWarps - 1) / kWarps, (size_t)ctx->num_sms * per_sm));
+        return (unsigned)std::max<size_t>(1, std::min((rows + per_cta - 1) / per_cta, (size_t)ctx->num_sms * per_sm));
     };
-    LUMEN_TRY(launch_pdl(ctx, moe_gate_up_kernel<WT>, dim3(blocks(a.top * a.ff + a.shared_ff, s1), (unsigned)a.M), kThreads, s1, s, a));
-    return launch_pdl(ctx, moe_down_kernel<WT>, dim3(blocks(a.W, s2), (unsigned)a.M), kThreads, s2, s, a);
+    LUMEN_TRY(launch_pdl(ctx, moe_gate_up_kernel<WT>, dim3(blocks(a.top * a.ff + a.shared_ff, s1, kWarps), (unsigned)a.M), kThreads, s1, s, a));
+    return launch_pdl(ctx, moe_down_kernel<WT>, dim3(blocks(a.W, s2, kDownRows), (unsigned)a.M), kThreads, s2, s, a);
 }
 
 }  // namespace
