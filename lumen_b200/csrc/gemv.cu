@@ -172,7 +172,7 @@ gemv_gate_up_kernel(const float *__restrict__ x, const WT *__restrict__ wg, cons
 // formed by every CTA while it stages x, so that the norm, the residual sum and the product are one launch.  WPR warps share a
 // weight row (a slice of K each) where there are too few rows to keep enough loads in flight.
 template <typename WT, int WPR>
-__global__ void __launch_bounds__(kThreads) gemv_step_kernel(const GemvStepArgs a) {
+__global__ void __launch_bounds__(kThreads, 4) gemv_step_kernel(const GemvStepArgs a) {
     extern __shared__ __align__(16) float smem[];
     __shared__ float red[kWarps];
     float *xs = smem;
@@ -183,9 +183,9 @@ __global__ void __launch_bounds__(kThreads) gemv_step_kernel(const GemvStepArgs 
     const WT *w = static_cast<const WT *>(a.w);
     const bool vec_ok = (K % VEC == 0) && ((reinterpret_cast<uintptr_t>(w) & 15) == 0);
     // this warp's slice of K, in whole vectors
-    const size_t per = (K / VEC + WPR - 1) / WPR * VEC, k0 = min(K, part * per), kn = min(K - k0, per);
-    uint4 pre[8];
-    if (vec_ok && row0 < a.N) row_ahead<WT>(w + row0 * K + k0, kn, lane, pre);
+    const int nv = (int)(K / VEC), per = (nv + WPR - 1) / WPR, v0 = min(nv, part * per), vn = min(nv - v0, per);
+    uint4 pre[kAhead];
+    if (vec_ok && row0 < a.N) row_ahead(reinterpret_cast<const uint4 *>(w + row0 * K) + v0, vn, lane, pre);
     pdl_launch();
     pdl_wait();
     auto inv_rms = [&](float ss) {
@@ -198,76 +198,84 @@ __global__ void __launch_bounds__(kThreads) gemv_step_kernel(const GemvStepArgs 
         __syncthreads();
         return __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(t, (float)K), a.eps)));
     };
+    // 32-bit indices and no unrolling: registers decide how many CTAs an SM holds
+    const int k_n = (int)K;
     if (a.y) {
         float ss = 0.f;
-        if (K % 4 == 0) {  // res and the gains are requested before the sum of y^2 is needed
-            constexpr int kHold = 4;  // float4 per thread held in registers: rows of up to 4096
+        if (k_n % 4 == 0) {  // the thread's first part of res and the gains is requested before the sum of y^2 is needed
             const float4 *y4 = reinterpret_cast<const float4 *>(a.y), *r4 = reinterpret_cast<const float4 *>(a.res), *g4 = reinterpret_cast<const float4 *>(a.gain);
-            float4 *x4 = reinterpret_cast<float4 *>(xs), *o4 = reinterpret_cast<float4 *>(a.x_out);
-            const size_t n4 = K / 4;
-            float4 r[kHold], g[kHold];
-#pragma unroll
-            for (int i = 0; i < kHold; ++i)
-                if (tid + kThreads * i < n4) {
-                    r[i] = r4[tid + kThreads * i];
-                    g[i] = g4[tid + kThreads * i];
-                }
-            for (size_t k = tid; k < n4; k += kThreads) {
+            float4 *x4 = reinterpret_cast<float4 *>(xs);
+            const int n4 = k_n / 4;
+            float4 r = make_float4(0.f, 0.f, 0.f, 0.f), g = r;
+            if (tid < n4) {
+                r = r4[tid];
+                g = g4[tid];
+            }
+#pragma unroll 1
+            for (int k = tid; k < n4; k += kThreads) {
                 const float4 v = y4[k];
                 x4[k] = v;
                 ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
             }
             const float inv = inv_rms(ss);
-            auto settle = [&](size_t k, float4 res, float4 gain) {
+#pragma unroll 1
+            for (int k = tid; k < n4; k += kThreads) {
                 const float4 v = x4[k];
-                const float4 x = make_float4(__fadd_rn(res.x, __fmul_rn(__fmul_rn(v.x, inv), gain.x)), __fadd_rn(res.y, __fmul_rn(__fmul_rn(v.y, inv), gain.y)),
-                                             __fadd_rn(res.z, __fmul_rn(__fmul_rn(v.z, inv), gain.z)), __fadd_rn(res.w, __fmul_rn(__fmul_rn(v.w, inv), gain.w)));
+                const float4 x = make_float4(__fadd_rn(r.x, __fmul_rn(__fmul_rn(v.x, inv), g.x)), __fadd_rn(r.y, __fmul_rn(__fmul_rn(v.y, inv), g.y)),
+                                             __fadd_rn(r.z, __fmul_rn(__fmul_rn(v.z, inv), g.z)), __fadd_rn(r.w, __fmul_rn(__fmul_rn(v.w, inv), g.w)));
+                if (k + kThreads < n4) {
+                    r = r4[k + kThreads];
+                    g = g4[k + kThreads];
+                }
                 x4[k] = x;
-                if (blockIdx.x == 0) o4[k] = x;
-            };
-#pragma unroll
-            for (int i = 0; i < kHold; ++i)
-                if (tid + kThreads * i < n4) settle(tid + kThreads * i, r[i], g[i]);
-            for (size_t k = tid + kThreads * kHold; k < n4; k += kThreads) settle(k, r4[k], g4[k]);
+                if (blockIdx.x == 0) reinterpret_cast<float4 *>(a.x_out)[k] = x;
+            }
         } else {
-            for (size_t k = tid; k < K; k += kThreads) {
+#pragma unroll 1
+            for (int k = tid; k < k_n; k += kThreads) {
                 const float v = a.y[k];
                 xs[k] = v;
                 ss = fmaf(v, v, ss);
             }
             const float inv = inv_rms(ss);
-            for (size_t k = tid; k < K; k += kThreads) {
+#pragma unroll 1
+            for (int k = tid; k < k_n; k += kThreads) {
                 const float x = __fadd_rn(a.res[k], __fmul_rn(__fmul_rn(xs[k], inv), a.gain[k]));
                 xs[k] = x;
                 if (blockIdx.x == 0) a.x_out[k] = x;
             }
         }
-    } else if (K % 4 == 0) {
-        for (size_t k = tid; k < K / 4; k += kThreads) reinterpret_cast<float4 *>(xs)[k] = reinterpret_cast<const float4 *>(a.res)[k];
+    } else if (k_n % 4 == 0) {
+#pragma unroll 2
+        for (int k = tid; k < k_n / 4; k += kThreads) reinterpret_cast<float4 *>(xs)[k] = reinterpret_cast<const float4 *>(a.res)[k];
     } else {
-        for (size_t k = tid; k < K; k += kThreads) xs[k] = a.res[k];
+#pragma unroll 1
+        for (int k = tid; k < k_n; k += kThreads) xs[k] = a.res[k];
     }
     if (a.norm_w) {
         __syncthreads();
         float ss = 0.f;
-        for (size_t k = tid; k < K; k += kThreads) ss = fmaf(xs[k], xs[k], ss);
+#pragma unroll 1
+        for (int k = tid; k < k_n; k += kThreads) ss = fmaf(xs[k], xs[k], ss);
         const float inv = inv_rms(ss);
-        for (size_t k = tid; k < K; k += kThreads) xs[k] = __fmul_rn(__fmul_rn(xs[k], inv), a.norm_w[k]);
+#pragma unroll 1
+        for (int k = tid; k < k_n; k += kThreads) xs[k] = __fmul_rn(__fmul_rn(xs[k], inv), a.norm_w[k]);
     }
     __syncthreads();
+#pragma unroll 1
     for (size_t base = (size_t)blockIdx.x * kRows; base < a.N; base += (size_t)gridDim.x * kRows) {
         const size_t row = base + warp / WPR;
-        float acc[1] = {0.f};
+        float v = 0.f;
         if (row < a.N) {
-            if (!vec_ok) {
-                if (part == 0) row_dot<WT, 1>(w + row * K, xs, K, lane, false, acc);
-            } else if (row == row0) {
-                acc[0] = row_dot_ahead<WT>(w + row * K + k0, xs + k0, kn, lane, pre);
-            } else {
-                row_dot<WT, 1>(w + row * K + k0, xs + k0, kn, lane, true, acc);
+            if (vec_ok) {
+                const uint4 *wrow = reinterpret_cast<const uint4 *>(w + row * K) + v0;
+                if (row != row0) batch_load(wrow, 0, vn, lane, pre);
+                v = row_dot_ahead<WT>(wrow, xs + v0 * VEC, vn, lane, pre);
+            } else if (part == 0) {
+                v = row_dot_scalar<WT>(w + row * K, xs, (int)K, lane);
             }
         }
-        float v = warp_sum(acc[0]);
+        v = warp_sum(v);
         if (WPR > 1) {  // the row's slices meet in its first warp
             if (lane == 0) red[warp] = v;
             __syncthreads();

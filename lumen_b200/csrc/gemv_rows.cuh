@@ -98,19 +98,20 @@ __device__ __forceinline__ void row_dot(const WT *__restrict__ wrow, const float
     }
 }
 
-// The first 8 x 32 vectors of a row requested ahead of time (while an earlier kernel still runs), the rest of the row handed to the
-// L2; row_dot_ahead then is row_dot<WT, 1> whose first batch is in registers.
-template <typename WT>
-__device__ __forceinline__ void row_ahead(const WT *__restrict__ wrow, size_t K, int lane, uint4 (&pre)[8]) {
-    constexpr int VEC = 16 / sizeof(WT);
-    const size_t nv = K / VEC;
+// A row in batches of kAhead x 32 vectors with the next batch always in flight.  The first batch is requested ahead of time (while
+// an earlier kernel still runs) and the rest of the row handed to the L2.  n: vectors of the row.
+constexpr int kAhead = 4;  // (registers: more would reduce the CTAs an SM holds)
+__device__ __forceinline__ void batch_load(const uint4 *__restrict__ row, int base, int n, int lane, uint4 (&v)[kAhead]) {
 #pragma unroll
-    for (int u = 0; u < 8; ++u) {
-        const size_t i = (size_t)u * 32 + lane;
-        pre[u] = i < nv ? ld_stream_u4(reinterpret_cast<const uint4 *>(wrow) + i) : make_uint4(0u, 0u, 0u, 0u);
+    for (int u = 0; u < kAhead; ++u) {
+        const int i = base + u * 32 + lane;
+        v[u] = i < n ? ld_stream_u4(row + i) : make_uint4(0u, 0u, 0u, 0u);
     }
-    for (size_t off = 4096 + (size_t)lane * 128; off < K * sizeof(WT); off += 4096)
-        asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char *>(wrow) + off));
+}
+__device__ __forceinline__ void row_ahead(const uint4 *__restrict__ row, int n, int lane, uint4 (&pre)[kAhead]) {
+    batch_load(row, 0, n, lane, pre);
+#pragma unroll 1
+    for (int i = kAhead * 32 + lane * 8; i < n; i += 256) asm volatile("prefetch.global.L2 [%0];" ::"l"(row + i));
 }
 template <typename WT>
 __device__ __forceinline__ float vec_dot(uint4 w, const float *x, float acc) {
@@ -133,27 +134,33 @@ __device__ __forceinline__ float vec_dot(uint4 w, const float *x, float acc) {
     }
 }
 template <typename WT>
-__device__ __forceinline__ float row_dot_ahead(const WT *__restrict__ wrow, const float *xs, size_t K, int lane, const uint4 (&pre)[8]) {
+__device__ __forceinline__ float row_dot_ahead(const uint4 *__restrict__ row, const float *xs, int n, int lane, uint4 (&cur)[kAhead]) {
     constexpr int VEC = 16 / sizeof(WT);
-    const size_t nv = K / VEC;
     float acc = 0.f;
+#pragma unroll 1
+    for (int base = 0; base < n; base += kAhead * 32) {
+        uint4 next[kAhead];
+        batch_load(row, base + kAhead * 32, n, lane, next);
 #pragma unroll
-    for (int u = 0; u < 8; ++u) {
-        const size_t i = (size_t)u * 32 + lane;
-        if (i < nv) acc = vec_dot<WT>(pre[u], xs + i * VEC, acc);
+        for (int u = 0; u < kAhead; ++u) {
+            const int i = base + u * 32 + lane;
+            if (i < n) acc = vec_dot<WT>(cur[u], xs + i * VEC, acc);
+        }
+#pragma unroll
+        for (int u = 0; u < kAhead; ++u) cur[u] = next[u];
     }
-    for (size_t base = 256; base < nv; base += 256) {
-        uint4 wv[8];
-#pragma unroll
-        for (int u = 0; u < 8; ++u) {
-            const size_t i = base + (size_t)u * 32 + lane;
-            wv[u] = i < nv ? ld_stream_u4(reinterpret_cast<const uint4 *>(wrow) + i) : make_uint4(0u, 0u, 0u, 0u);
-        }
-#pragma unroll
-        for (int u = 0; u < 8; ++u) {
-            const size_t i = base + (size_t)u * 32 + lane;
-            if (i < nv) acc = vec_dot<WT>(wv[u], xs + i * VEC, acc);
-        }
+    return acc;
+}
+// Any row length and alignment.
+template <typename WT>
+__device__ __forceinline__ float row_dot_scalar(const WT *__restrict__ row, const float *xs, int K, int lane) {
+    float acc = 0.f;
+#pragma unroll 1
+    for (int k = lane; k < K; k += 32) {
+        float w;
+        if constexpr (sizeof(WT) == 4) w = row[k];
+        else w = __bfloat162float(row[k]);
+        acc = fmaf(w, xs[k], acc);
     }
     return acc;
 }

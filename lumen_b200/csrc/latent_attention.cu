@@ -64,7 +64,7 @@ __global__ void __launch_bounds__(kThreads) latent_absorb_kernel(const LatentArg
     const int tid = threadIdx.x;
     const size_t h = blockIdx.x, m = blockIdx.z;
     // the first weight vectors of this thread are requested while the projections still run
-    constexpr int kAhead = 4, kQ = sizeof(T) / 2;
+    constexpr int kQ = sizeof(T) / 2;
     const int cg = tid % kColGroups, slice = tid / kColGroups;
     const size_t r0 = (size_t)blockIdx.y * kAbsorbCols + cg * 8;
     const T *w = static_cast<const T *>(a.wuk) + h * a.dim * a.rank + r0;
@@ -230,8 +230,9 @@ __global__ void __launch_bounds__(kThreads) latent_value_kernel(const LatentArgs
     const bool vec_ok = a.rank % VEC == 0;
     const size_t v0 = (size_t)blockIdx.y * kValueRows + warp, v1 = min(a.vdim, (size_t)(blockIdx.y + 1) * kValueRows);
     const T *w = static_cast<const T *>(a.wuv) + h * a.vdim * a.rank;
-    uint4 pre[8];
-    if (vec_ok && v0 < v1) row_ahead<T>(w + v0 * a.rank, a.rank, lane, pre);
+    uint4 pre[kAhead];
+    const int nv = (int)(a.rank / VEC);
+    if (vec_ok && v0 < v1) row_ahead(reinterpret_cast<const uint4 *>(w + v0 * a.rank), nv, lane, pre);
     pdl_launch();
     pdl_wait();
     if (warp == 0) {
@@ -274,10 +275,15 @@ __global__ void __launch_bounds__(kThreads) latent_value_kernel(const LatentArgs
     __syncthreads();
     const float gate = sigmoid_f(a.u[m * a.u_ld + a.u_gate + h]);
     for (size_t v = v0; v < v1; v += kWarps) {
-        float acc[1] = {0.f};
-        if (vec_ok && v == v0) acc[0] = row_dot_ahead<T>(w + v * a.rank, ctx, a.rank, lane, pre);
-        else row_dot<T, 1>(w + v * a.rank, ctx, a.rank, lane, vec_ok, acc);
-        const float y = warp_sum(acc[0]) * gate;
+        float d;
+        if (vec_ok) {
+            const uint4 *wrow = reinterpret_cast<const uint4 *>(w + v * a.rank);
+            if (v != v0) batch_load(wrow, 0, nv, lane, pre);
+            d = row_dot_ahead<T>(wrow, ctx, nv, lane, pre);
+        } else {
+            d = row_dot_scalar<T>(w + v * a.rank, ctx, (int)a.rank, lane);
+        }
+        const float y = warp_sum(d) * gate;
         if (lane == 0) {
             const size_t at = (m * a.H + h) * a.vdim + v;
             if (a.out) a.out[at] = y;

@@ -86,8 +86,8 @@ __global__ void __launch_bounds__(kThreads) moe_gate_up_kernel(const MoeArgs a) 
         if (vec_ok) {
             rows_dot<WT, 1, 2>(rows, xs, K, lane, acc);
         } else {
-            row_dot<WT, 1>(rows[0], xs, K, lane, false, acc[0]);
-            row_dot<WT, 1>(rows[1], xs, K, lane, false, acc[1]);
+            acc[0][0] = row_dot_scalar<WT>(rows[0], xs, (int)K, lane);
+            acc[1][0] = row_dot_scalar<WT>(rows[1], xs, (int)K, lane);
         }
         const float g = warp_sum(acc[0][0]) * w, u = warp_sum(acc[1][0]) * w;
         if (lane == 0) a.act[m * total + i] = gated_act(g, u, limit);
@@ -97,7 +97,7 @@ __global__ void __launch_bounds__(kThreads) moe_gate_up_kernel(const MoeArgs a) 
 // Four warps share an output row: the chosen experts' rows and the shared one form one sequence of vectors.
 constexpr int kDownWarps = 4, kDownRows = kWarps / kDownWarps;
 template <typename WT>
-__global__ void __launch_bounds__(kThreads) moe_down_kernel(const MoeArgs a) {
+__global__ void __launch_bounds__(kThreads, 3) moe_down_kernel(const MoeArgs a) {
     extern __shared__ __align__(16) float act[];  // every expert's activations, each on a 16-byte boundary; then the experts' numbers
     __shared__ float red[kWarps];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, part = warp % kDownWarps;
@@ -127,7 +127,7 @@ __global__ void __launch_bounds__(kThreads) moe_down_kernel(const MoeArgs a) {
             if (vec_ok) {
                 for (unsigned i0 = part * 256; i0 < all; i0 += kDownWarps * 256) {
                     uint4 wv[8];
-                    unsigned xo[8];
+                    int xo[8];
 #pragma unroll
                     for (int u = 0; u < 8; ++u) {
                         const unsigned i = i0 + u * 32 + lane;
@@ -148,8 +148,8 @@ __global__ void __launch_bounds__(kThreads) moe_down_kernel(const MoeArgs a) {
                 }
             } else {
                 for (int k = part; k <= top; k += kDownWarps) {
-                    if (k < top) row_dot<WT, 1>(static_cast<const WT *>(a.down) + ((size_t)sel[k] * a.W + n) * ff, act + k * ff4, ff, lane, false, acc);
-                    else if (sff) row_dot<WT, 1>(shared_row, act + top * ff4, sff, lane, false, acc);
+                    if (k < top) acc[0] += row_dot_scalar<WT>(static_cast<const WT *>(a.down) + ((size_t)sel[k] * a.W + n) * ff, act + k * ff4, ff, lane);
+                    else if (sff) acc[0] += row_dot_scalar<WT>(shared_row, act + top * ff4, sff, lane);
                 }
             }
         }
