@@ -155,6 +155,14 @@ int latent_pick_splits(const LatentArgs &a, size_t total, int num_sms);
 bool latent_mma_usable(const LatentArgs &a);
 int launch_latent_scores(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s);
 int launch_latent_mma(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s);
+// Cached rows a piece is made of: pieces of one tile each while there are fewer tiles than pieces, else about equal shares.
+constexpr int kLatentTile = 64;
+#ifdef __CUDACC__
+__device__ __forceinline__ int latent_pieces(int total, int nsplit) { return min(nsplit, (total + kLatentTile - 1) / kLatentTile); }
+__device__ __forceinline__ int latent_piece_start(int total, int pieces, int i) {  // first cached row of piece i (i == pieces: the end)
+    return (int)((long long)i * ((total + kLatentTile - 1) / kLatentTile) / pieces) * kLatentTile;
+}
+#endif
 // Pieces merged, W_uv and the output gate applied.
 int launch_latent_value(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s);
 // Whole portions on the tensor cores over expanded keys and values (bf16); the cache already holds the rows.

@@ -99,7 +99,8 @@ __device__ __forceinline__ void row_dot(const WT *__restrict__ wrow, const float
 }
 
 // A row in batches of kAhead x 32 vectors with the next batch always in flight.  The first batch is requested ahead of time (while
-// an earlier kernel still runs) and the rest of the row handed to the L2.  n: vectors of the row.
+// an earlier kernel still runs) and the next few KB of the row handed to the L2 (not more: all rows of a large matrix at once
+// would push one another out).  n: vectors of the row.
 constexpr int kAhead = 4;  // (registers: more would reduce the CTAs an SM holds)
 __device__ __forceinline__ void batch_load(const uint4 *__restrict__ row, int base, int n, int lane, uint4 (&v)[kAhead]) {
 #pragma unroll
@@ -111,7 +112,7 @@ __device__ __forceinline__ void batch_load(const uint4 *__restrict__ row, int ba
 __device__ __forceinline__ void row_ahead(const uint4 *__restrict__ row, int n, int lane, uint4 (&pre)[kAhead]) {
     batch_load(row, 0, n, lane, pre);
 #pragma unroll 1
-    for (int i = kAhead * 32 + lane * 8; i < n; i += 256) asm volatile("prefetch.global.L2 [%0];" ::"l"(row + i));
+    for (int i = kAhead * 32 + lane * 8; i < min(n, 512); i += 256) asm volatile("prefetch.global.L2 [%0];" ::"l"(row + i));
 }
 template <typename WT>
 __device__ __forceinline__ float vec_dot(uint4 w, const float *x, float acc) {

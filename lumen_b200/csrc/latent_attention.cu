@@ -153,8 +153,9 @@ __global__ void __launch_bounds__(kScoreWarps * 32) latent_scores_kernel(const L
     for (size_t row = blockIdx.y; row < a.B * a.S * a.H; row += gridDim.y) {
         const size_t m = row / a.H, b = m / a.S, past = (size_t)*a.d_len, total = past + a.S;
         const size_t seen = past + (m - b * a.S) + 1;
-        const size_t chunk = (total + a.nsplit - 1) / a.nsplit;
-        const size_t j0 = blockIdx.x * chunk, j1 = min(seen, j0 + chunk);
+        const int pieces = latent_pieces((int)total, a.nsplit);
+        if ((int)blockIdx.x >= pieces) return;
+        const size_t j0 = latent_piece_start((int)total, pieces, blockIdx.x), j1 = min(seen, (size_t)latent_piece_start((int)total, pieces, blockIdx.x + 1));
         const T *qsrc = static_cast<const T *>(a.qf) + row * a.pitch;
         __syncthreads();
         for (int i = tid; i < width; i += kScoreWarps * 32) q[i] = to_f32(qsrc[i]);
@@ -216,13 +217,13 @@ __global__ void __launch_bounds__(kScoreWarps * 32) latent_scores_kernel(const L
 }
 
 // grid (heads, chunks of value rows, rows)
-constexpr int kValueRows = 16;
+constexpr int kValueRows = 16, kValueThreads = 512, kValueGroups = kValueThreads / 128;
 template <typename T>
-__global__ void __launch_bounds__(kThreads) latent_value_kernel(const LatentArgs a) {
+__global__ void __launch_bounds__(kValueThreads) latent_value_kernel(const LatentArgs a) {
     extern __shared__ __align__(16) float smem[];
     const size_t rank4 = (a.rank + 3) & ~(size_t)3;
-    float *ctx = smem;               // [2][rank4]: halves of the pieces, summed into the first
-    float *f = ctx + 2 * rank4;      // [nsplit]
+    float *ctx = smem;                        // [groups][rank4]: shares of the pieces, summed into the first
+    float *f = ctx + kValueGroups * rank4;    // [nsplit]
     __shared__ float inv_s;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const size_t h = blockIdx.x, m = blockIdx.z, o = (m * a.H + h) * a.nsplit;
@@ -235,13 +236,14 @@ __global__ void __launch_bounds__(kThreads) latent_value_kernel(const LatentArgs
     if (vec_ok && v0 < v1) row_ahead(reinterpret_cast<const uint4 *>(w + v0 * a.rank), nv, lane, pre);
     pdl_launch();
     pdl_wait();
+    const int pieces = latent_pieces(*a.d_len + (int)a.S, a.nsplit);
     if (warp == 0) {
         float M = -INFINITY;
-        for (int s = lane; s < a.nsplit; s += 32) M = fmaxf(M, a.part_ml[(o + s) * 2]);
+        for (int s = lane; s < pieces; s += 32) M = fmaxf(M, a.part_ml[(o + s) * 2]);
 #pragma unroll
         for (int k = 16; k > 0; k >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, k));
         float l = 0.f;
-        for (int s = lane; s < a.nsplit; s += 32) {
+        for (int s = lane; s < pieces; s += 32) {
             const float ms = a.part_ml[(o + s) * 2], w = ms == -INFINITY ? 0.f : expf(ms - M);
             f[s] = w;
             l = fmaf(a.part_ml[(o + s) * 2 + 1], w, l);
@@ -251,30 +253,35 @@ __global__ void __launch_bounds__(kThreads) latent_value_kernel(const LatentArgs
     }
     __syncthreads();
     const float inv = inv_s;
-    if (a.rank % 4 == 0) {  // two groups of 128 threads, each with every other piece; a thread owns four adjacent columns
-        const int half = tid >> 7;
+    if (a.rank % 4 == 0) {  // groups of 128 threads, each with every fourth piece; a thread owns four adjacent columns
+        const int group = tid >> 7;
         for (size_t c = tid & 127; c < a.rank / 4; c += 128) {
             float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 8
-            for (int s = half; s < a.nsplit; s += 2) {
+            for (int s = group; s < pieces; s += kValueGroups) {
                 const float4 p = reinterpret_cast<const float4 *>(a.part_ctx + (o + s) * a.rank)[c];
                 const float w = f[s];
                 v.x = fmaf(p.x, w, v.x); v.y = fmaf(p.y, w, v.y); v.z = fmaf(p.z, w, v.z); v.w = fmaf(p.w, w, v.w);
             }
-            reinterpret_cast<float4 *>(ctx + half * rank4)[c] = make_float4(v.x * inv, v.y * inv, v.z * inv, v.w * inv);
+            reinterpret_cast<float4 *>(ctx + group * rank4)[c] = make_float4(v.x * inv, v.y * inv, v.z * inv, v.w * inv);
         }
         __syncthreads();
-        for (size_t r = tid; r < a.rank; r += kThreads) ctx[r] += ctx[rank4 + r];
+        for (size_t r = tid; r < a.rank; r += kValueThreads) {
+            float v = ctx[r];
+#pragma unroll
+            for (int g = 1; g < kValueGroups; ++g) v += ctx[g * rank4 + r];
+            ctx[r] = v;
+        }
     } else {
-        for (size_t r = tid; r < a.rank; r += kThreads) {
+        for (size_t r = tid; r < a.rank; r += kValueThreads) {
             float v = 0.f;
-            for (int s = 0; s < a.nsplit; ++s) v = fmaf(a.part_ctx[(o + s) * a.rank + r], f[s], v);
+            for (int s = 0; s < pieces; ++s) v = fmaf(a.part_ctx[(o + s) * a.rank + r], f[s], v);
             ctx[r] = v * inv;
         }
     }
     __syncthreads();
     const float gate = sigmoid_f(a.u[m * a.u_ld + a.u_gate + h]);
-    for (size_t v = v0; v < v1; v += kWarps) {
+    for (size_t v = v0; v < v1; v += kValueThreads / 32) {
         float d;
         if (vec_ok) {
             const uint4 *wrow = reinterpret_cast<const uint4 *>(w + v * a.rank);
@@ -332,9 +339,9 @@ int launch_latent_scores(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s) {
 int launch_latent_value(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s) {
     const size_t rows = a.B * a.S;
     if (rows > 65535) return set_error(ctx, LUMEN_ERR_UNSUPPORTED, "latent attention: %zu rows in one step", rows);
-    const size_t smem = (2 * ((a.rank + 3) & ~(size_t)3) + a.nsplit) * sizeof(float);
+    const size_t smem = (kValueGroups * ((a.rank + 3) & ~(size_t)3) + a.nsplit) * sizeof(float);
     const dim3 grid((unsigned)a.H, (unsigned)((a.vdim + kValueRows - 1) / kValueRows), (unsigned)rows);
-    return launch_pdl(ctx, a.dt == LUMEN_F32 ? latent_value_kernel<float> : latent_value_kernel<__nv_bfloat16>, grid, kThreads, smem, s, a);
+    return launch_pdl(ctx, a.dt == LUMEN_F32 ? latent_value_kernel<float> : latent_value_kernel<__nv_bfloat16>, grid, kValueThreads, smem, s, a);
 }
 
 }  // namespace lumen

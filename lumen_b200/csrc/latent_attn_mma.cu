@@ -15,7 +15,7 @@ namespace lumen {
 namespace {
 
 constexpr int kWarps = 8, kThreads = kWarps * 32;
-constexpr int kBN = 64;            // cached rows per tile
+constexpr int kBN = kLatentTile;   // cached rows per tile
 constexpr int kLdS = kBN + 4;      // floats between score rows
 constexpr int kLdP = kBN + 8;      // bf16 between weight rows (16 bytes more than a multiple of 128)
 
@@ -67,10 +67,11 @@ __global__ void __launch_bounds__(kThreads, 1) latent_attn_mma_kernel(const Late
     pdl_launch();
     const int H = (int)a.H, n_rows = (int)(a.S * a.H), row0 = blockIdx.y * kRows, b = blockIdx.z, split = blockIdx.x;
     const int past = *a.d_len, total = past + (int)a.S;
-    const int tiles_all = (total + kBN - 1) / kBN;
+    const int pieces = latent_pieces(total, a.nsplit);  // later pieces are empty, and not read by the merge
+    if (split >= pieces) return;
     // the last query row of this block sees up to past + its position
     const int seen = past + min(row0 + kRows - 1, n_rows - 1) / H + 1;
-    const int j0 = (int)((long long)split * tiles_all / a.nsplit) * kBN, j1 = min(seen, (int)((long long)(split + 1) * tiles_all / a.nsplit) * kBN);
+    const int j0 = latent_piece_start(total, pieces, split), j1 = min(seen, latent_piece_start(total, pieces, split + 1));
     const int nt = j1 > j0 ? (j1 - j0 + kBN - 1) / kBN : 0;
     const __nv_bfloat16 *cache = static_cast<const __nv_bfloat16 *>(a.cache) + (size_t)b * a.max_seq * pitch;
     const int vec = pitch / 8;
@@ -292,15 +293,15 @@ bool latent_mma_usable(const LatentArgs &a) {
            a.S * a.H <= 16 * 65535;
 }
 
-// Pieces of the context: about one CTA per SM over query-row blocks and batch rows, at least one tile each; powers of two so
-// that a handful of captured graphs covers every context length.
+// Pieces of the context: about one CTA per SM over query-row blocks and batch rows; powers of two so that a handful of captured
+// graphs covers every context length (with fewer tiles than pieces the last pieces stay empty).
 int latent_pick_splits(const LatentArgs &a, size_t total, int num_sms) {
     const bool mma = latent_mma_usable(a);
     const size_t rows = a.S * a.H, blocks = a.B * (mma ? (rows + row_tiles(a) * 16 - 1) / (row_tiles(a) * 16) : rows);
     const size_t want = std::min<size_t>({(total + kBN - 1) / kBN, std::max<size_t>(1, (size_t)num_sms * (mma ? 1 : 8) / std::max<size_t>(blocks, 1)), 64});
     int n = 1;
-    while ((size_t)n * 2 <= want) n <<= 1;
-    return n;
+    while ((size_t)n < want) n <<= 1;
+    return std::min(n, 64);
 }
 
 int launch_latent_mma(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s) {
