@@ -198,20 +198,15 @@ __global__ void __launch_bounds__(kThreads, 4) gemv_step_kernel(const GemvStepAr
         __syncthreads();
         return __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(t, (float)K), a.eps)));
     };
-    // 32-bit indices and no unrolling: registers decide how many CTAs an SM holds
+    // 32-bit indices and little unrolling: registers decide how many CTAs an SM holds
     const int k_n = (int)K;
     if (a.y) {
         float ss = 0.f;
-        if (k_n % 4 == 0) {  // the thread's first part of res and the gains is requested before the sum of y^2 is needed
+        if (k_n % 4 == 0) {
             const float4 *y4 = reinterpret_cast<const float4 *>(a.y), *r4 = reinterpret_cast<const float4 *>(a.res), *g4 = reinterpret_cast<const float4 *>(a.gain);
             float4 *x4 = reinterpret_cast<float4 *>(xs);
             const int n4 = k_n / 4;
-            float4 r = make_float4(0.f, 0.f, 0.f, 0.f), g = r;
-            if (tid < n4) {
-                r = r4[tid];
-                g = g4[tid];
-            }
-#pragma unroll 1
+#pragma unroll 4
             for (int k = tid; k < n4; k += kThreads) {
                 const float4 v = y4[k];
                 x4[k] = v;
@@ -219,16 +214,24 @@ __global__ void __launch_bounds__(kThreads, 4) gemv_step_kernel(const GemvStepAr
             }
             const float inv = inv_rms(ss);
 #pragma unroll 1
-            for (int k = tid; k < n4; k += kThreads) {
-                const float4 v = x4[k];
-                const float4 x = make_float4(__fadd_rn(r.x, __fmul_rn(__fmul_rn(v.x, inv), g.x)), __fadd_rn(r.y, __fmul_rn(__fmul_rn(v.y, inv), g.y)),
-                                             __fadd_rn(r.z, __fmul_rn(__fmul_rn(v.z, inv), g.z)), __fadd_rn(r.w, __fmul_rn(__fmul_rn(v.w, inv), g.w)));
-                if (k + kThreads < n4) {
-                    r = r4[k + kThreads];
-                    g = g4[k + kThreads];
+            for (int k0 = tid; k0 < n4; k0 += 2 * kThreads) {  // two at a time: both loads before a store that might alias
+                float4 r[2], g[2];
+#pragma unroll
+                for (int i = 0; i < 2; ++i)
+                    if (k0 + i * kThreads < n4) {
+                        r[i] = r4[k0 + i * kThreads];
+                        g[i] = g4[k0 + i * kThreads];
+                    }
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    const int k = k0 + i * kThreads;
+                    if (k >= n4) break;
+                    const float4 v = x4[k];
+                    const float4 x = make_float4(__fadd_rn(r[i].x, __fmul_rn(__fmul_rn(v.x, inv), g[i].x)), __fadd_rn(r[i].y, __fmul_rn(__fmul_rn(v.y, inv), g[i].y)),
+                                                 __fadd_rn(r[i].z, __fmul_rn(__fmul_rn(v.z, inv), g[i].z)), __fadd_rn(r[i].w, __fmul_rn(__fmul_rn(v.w, inv), g[i].w)));
+                    x4[k] = x;
+                    if (blockIdx.x == 0) reinterpret_cast<float4 *>(a.x_out)[k] = x;
                 }
-                x4[k] = x;
-                if (blockIdx.x == 0) reinterpret_cast<float4 *>(a.x_out)[k] = x;
             }
         } else {
 #pragma unroll 1
@@ -246,7 +249,7 @@ __global__ void __launch_bounds__(kThreads, 4) gemv_step_kernel(const GemvStepAr
             }
         }
     } else if (k_n % 4 == 0) {
-#pragma unroll 2
+#pragma unroll 6
         for (int k = tid; k < k_n / 4; k += kThreads) reinterpret_cast<float4 *>(xs)[k] = reinterpret_cast<const float4 *>(a.res)[k];
     } else {
 #pragma unroll 1

@@ -293,15 +293,16 @@ bool latent_mma_usable(const LatentArgs &a) {
            a.S * a.H <= 16 * 65535;
 }
 
+constexpr int kMaxPieces = 128;
 // Pieces of the context: about one CTA per SM over query-row blocks and batch rows; powers of two so that a handful of captured
 // graphs covers every context length (with fewer tiles than pieces the last pieces stay empty).
 int latent_pick_splits(const LatentArgs &a, size_t total, int num_sms) {
     const bool mma = latent_mma_usable(a);
     const size_t rows = a.S * a.H, blocks = a.B * (mma ? (rows + row_tiles(a) * 16 - 1) / (row_tiles(a) * 16) : rows);
-    const size_t want = std::min<size_t>({(total + kBN - 1) / kBN, std::max<size_t>(1, (size_t)num_sms * (mma ? 1 : 8) / std::max<size_t>(blocks, 1)), 64});
+    const size_t want = std::min<size_t>({(total + kBN - 1) / kBN, std::max<size_t>(1, (size_t)num_sms * (mma ? 1 : 8) / std::max<size_t>(blocks, 1)), (size_t)kMaxPieces});
     int n = 1;
     while ((size_t)n < want) n <<= 1;
-    return std::min(n, 64);
+    return std::min(n, kMaxPieces);
 }
 
 int launch_latent_mma(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s) {
