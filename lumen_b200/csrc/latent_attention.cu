@@ -27,33 +27,38 @@ __device__ __forceinline__ float rotated(const float *v, size_t i, size_t rot_di
     return (i & 1) ? __fadd_rn(__fmul_rn(y, c), __fmul_rn(x, s)) : __fsub_rn(__fmul_rn(x, c), __fmul_rn(y, s));
 }
 
-template <typename T>
+// NT threads (a warp, or the whole CTA) share a row.
+template <typename T, int NT>
 __device__ __forceinline__ void append_row(const LatentArgs &a, size_t m, float *red, int tid) {
     const size_t b = m / a.S, pos = (size_t)*a.d_len + (m - b * a.S);
     const float *d = a.u + m * a.u_ld + a.u_kv;
     T *row = static_cast<T *>(a.cache) + (b * a.max_seq + pos) * a.pitch;
     float ss = 0.f;
-    for (size_t i = tid; i < a.rank; i += kThreads) ss = fmaf(d[i], d[i], ss);
+#pragma unroll 4
+    for (size_t i = tid; i < a.rank; i += NT) ss = fmaf(d[i], d[i], ss);
     ss = warp_sum(ss);
-    if ((tid & 31) == 0) red[tid >> 5] = ss;
-    __syncthreads();
-    float t = 0.f;
+    if (NT > 32) {
+        if ((tid & 31) == 0) red[tid >> 5] = ss;
+        __syncthreads();
+        ss = 0.f;
 #pragma unroll
-    for (int w = 0; w < kWarps; ++w) t += red[w];
-    const float inv = __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(t, (float)a.rank), a.eps)));
+        for (int w = 0; w < NT / 32; ++w) ss += red[w];
+    }
+    const float inv = __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)a.rank), a.eps)));
     const size_t half = a.rot_dims / 2;
-    for (size_t i = tid; i < a.pitch; i += kThreads) {
+#pragma unroll 4
+    for (size_t i = tid; i < a.rank; i += NT) row[i] = from_f32<T>(__fmul_rn(__fmul_rn(d[i], inv), a.latent_gain[i]));
+    for (size_t i = a.rank + tid; i < a.pitch; i += NT) {
         float v = 0.f;
-        if (i < a.rank) v = __fmul_rn(__fmul_rn(d[i], inv), a.latent_gain[i]);
-        else if (i < a.rank + a.rot_dim) v = rotated(d + a.rank, i - a.rank, a.rot_dims, a.cos_t + pos * half, a.sin_t + pos * half);
+        if (i < a.rank + a.rot_dim) v = rotated(d + a.rank, i - a.rank, a.rot_dims, a.cos_t + pos * half, a.sin_t + pos * half);
         row[i] = from_f32<T>(v);
     }
 }
 
 template <typename T>
 __global__ void __launch_bounds__(kThreads) latent_append_kernel(const LatentArgs a) {
-    __shared__ float red[kWarps];
-    append_row<T>(a, blockIdx.x, red, threadIdx.x);
+    const size_t m = (size_t)blockIdx.x * kWarps + (threadIdx.x >> 5);  // one warp per row
+    if (m < a.B * a.S) append_row<T, 32>(a, m, nullptr, threadIdx.x & 31);
 }
 
 // grid (heads, chunks of 64 latent columns (+ 1 when the first head's CTA there appends the cache row), rows)
@@ -78,7 +83,7 @@ __global__ void __launch_bounds__(kThreads) latent_absorb_kernel(const LatentArg
     pdl_launch();
     pdl_wait();
     if ((int)blockIdx.y == chunks) {
-        if (h == 0) append_row<T>(a, m, &part[0][0], tid);
+        if (h == 0) append_row<T, kThreads>(a, m, &part[0][0], tid);
         return;
     }
     const float *q = a.u + m * a.u_ld + h * (a.dim + a.rot_dim);
@@ -317,8 +322,8 @@ int launch_scores_t(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s) {
 }  // namespace
 
 int launch_latent_append(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s) {
-    if (a.dt == LUMEN_F32) latent_append_kernel<float><<<(unsigned)(a.B * a.S), kThreads, 0, s>>>(a);
-    else latent_append_kernel<__nv_bfloat16><<<(unsigned)(a.B * a.S), kThreads, 0, s>>>(a);
+    if (a.dt == LUMEN_F32) latent_append_kernel<float><<<(unsigned)((a.B * a.S + kWarps - 1) / kWarps), kThreads, 0, s>>>(a);
+    else latent_append_kernel<__nv_bfloat16><<<(unsigned)((a.B * a.S + kWarps - 1) / kWarps), kThreads, 0, s>>>(a);
     LUMEN_LAUNCHED(ctx);
     return LUMEN_OK;
 }
