@@ -380,7 +380,7 @@ def layer_models(L, case: str, max_seq: int):
     else:
         mlp = dict(kind="dense", ff=c["ff"])
     d = dict(architecture="Fegetar", vocab=4096, width=c["width"], norm=dict(eps=1e-5), token_side=dict(dim=256),
-             embedding=dict(bigram=dict(buckets=65521, mul_prev=31, mul_cur=7)),
+             embedding=dict(bigram=dict(buckets=65521, mul_prev=1000003, mul_cur=101)),
              layers=[dict(type="latent_attention", mixer=mixer, mlp=mlp)] * c["layers"])
     return L.FegetarConfig.from_dict(d, max_seq, "bf16"), L.LlamaConfig(
         vocab_size=4096, hidden_size=c["width"], num_hidden_layers=c["layers"], num_attention_heads=c["heads"], head_dim=128,

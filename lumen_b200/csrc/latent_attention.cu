@@ -34,7 +34,7 @@ __device__ __forceinline__ void append_row(const LatentArgs &a, size_t m, float 
     const float *d = a.u + m * a.u_ld + a.u_kv;
     T *row = static_cast<T *>(a.cache) + (b * a.max_seq + pos) * a.pitch;
     float ss = 0.f;
-#pragma unroll 4
+#pragma unroll (NT == 32 ? 16 : 4)
     for (size_t i = tid; i < a.rank; i += NT) ss = fmaf(d[i], d[i], ss);
     ss = warp_sum(ss);
     if (NT > 32) {
@@ -46,7 +46,7 @@ __device__ __forceinline__ void append_row(const LatentArgs &a, size_t m, float 
     }
     const float inv = __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)a.rank), a.eps)));
     const size_t half = a.rot_dims / 2;
-#pragma unroll 4
+#pragma unroll (NT == 32 ? 16 : 4)
     for (size_t i = tid; i < a.rank; i += NT) row[i] = from_f32<T>(__fmul_rn(__fmul_rn(d[i], inv), a.latent_gain[i]));
     for (size_t i = a.rank + tid; i < a.pitch; i += NT) {
         float v = 0.f;

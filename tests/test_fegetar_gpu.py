@@ -138,7 +138,7 @@ def test_long_decoding(L):
     cfg = _mixed()
     p, ids = F.weights(L, cfg, 8), _ids(420, 8)
     _check(L, cfg, p, ids, ([20, 1],), "f32")
-    cfg = F.config([(F.mixer(heads=6, kv_rank=128), F.dense())])
+    cfg = F.config([(F.mixer(heads=7, kv_rank=112), F.dense())])
     _check(L, cfg, F.weights(L, cfg, 8), ids, ([20, 1],), "bf16")
 
 
@@ -221,7 +221,7 @@ FAR = [(1, 0), (2, 1), (63, 0), (64, 0), (64, 63), (65, 63), (65, 64), (127, 63)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("m", [F.mixer(heads=2, dim=32, rot_dim=16, vdim=32, kv_rank=64), F.mixer(heads=2, dim=28, rot_dim=8, vdim=40, kv_rank=60),
+@pytest.mark.parametrize("m", [F.mixer(heads=2, dim=32, rot_dim=24, vdim=40, kv_rank=72), F.mixer(heads=2, dim=28, rot_dim=8, vdim=40, kv_rank=60),
                                F.mixer(heads=1, dim=36, rot_dim=10, vdim=40, kv_rank=68)])
 def test_far_keys_and_borders(L, dtype, m):
     cfg, p = _standing_out(L, m)
