@@ -266,14 +266,29 @@ int lumen_llama_decode_trace(lumen_llama *m, uint64_t *out, size_t capacity, siz
  *                      cache holds these kv_rank + rot_dim numbers per token.  The first rot_dims of the rotated part
  *                      turn in interleaved pairs (2i, 2i+1) with frequency rot_base^(-2i/rot_dims).  A sigmoid gate per head
  *                      scales the head's output.
+ *   attention          grouped queries (`heads` x dim over kv_heads keys x dim and values x vdim), RMS norm of every query and
+ *                      key, rotation of the pairs (i, i + rot_dims/2) with optionally scaled frequencies, a learned sink per
+ *                      head in the softmax's denominator, a sigmoid gate per head.  chunk > 0: a position sees the keys of its
+ *                      own chunk of that many positions.  kv_from >= 0: the keys and values cached by that earlier layer.
+ *   mlstm              matrix memory [dim, vdim] per head with exponential gates (capped at gate_cap), a normaliser vector and a
+ *                      running maximum; the cache holds this state (f32) instead of rows.
  *   dense              down(gelu_tanh(up(x)))
+ *   gated gelu         down(gelu_tanh(gate(x)) * up(x))
  *   moe                `top` of `experts` clamped-SwiGLU experts by sigmoid scores (the score scales the expert's input),
  *                      plus a shared expert (shared_ff == 0: none)
- * Sublayers read the residual itself; their outputs are RMS-normed with gain 1 + w and added.  Options of the model:
- * a bigram embedding (bigram_buckets == 0: none), and a per-layer token input after the feed-forward (side_dim == 0: none). */
+ * Norms (of the model): LUMEN_NORM_OUTPUT: sublayers read the residual itself and their outputs are RMS-normed with gain 1 + w and
+ * added.  LUMEN_NORM_BOTH: an RMS norm with gain w before every sublayer and another one of its output.  Options of the model:
+ * a factor of the embedding, the embedding as output matrix (tied_head), a bigram embedding (bigram_buckets == 0: none), and
+ * a per-layer token input after the feed-forward (side_dim == 0: none). */
+#define LUMEN_MIXER_LATENT 0
+#define LUMEN_MIXER_ATTENTION 1
+#define LUMEN_MIXER_MLSTM 2
+#define LUMEN_NORM_OUTPUT 0
+#define LUMEN_NORM_BOTH 1
 #define LUMEN_MLP_NONE 0
 #define LUMEN_MLP_DENSE 1
 #define LUMEN_MLP_MOE 2
+#define LUMEN_MLP_GATED_GELU 3
 typedef struct {
     size_t heads;
     size_t dim;
@@ -291,6 +306,15 @@ typedef struct {
     float expert_limit;
     size_t shared_ff;
     float shared_limit;
+    int mixer;
+    size_t kv_heads;      /* attention */
+    int kv_from;          /* attention: -1, or the layer whose keys and values are used */
+    size_t chunk;         /* attention: positions per chunk (0: all earlier positions are seen) */
+    double rot_factor;    /* frequency scaling (0: none): wavelengths above rot_original / rot_low are stretched by the factor, */
+    double rot_low;       /* those below rot_original / rot_high kept, those between interpolated */
+    double rot_high;
+    double rot_original;
+    float gate_cap;       /* mlstm */
 } lumen_decoder_layer;
 typedef struct {
     size_t vocab_size;
@@ -304,10 +328,13 @@ typedef struct {
     size_t bigram_mul_cur;
     size_t side_dim;
     lumen_dtype weight_dtype;
+    float embed_scale;
+    int tied_head;
+    int norms;            /* LUMEN_NORM_* */
 } lumen_decoder_config;
 /* Parameters are named as in the checkpoint (embed, bigram, side.embed, l<i>.mix.q, l<i>.mlp.e<j>.gate, final.norm, head, ...).
  * weight_dtype f32: every product in 32-bit arithmetic.  weight_dtype bf16: bf16 products with 32-bit accumulation and
- * a bf16 latent cache; positions, scores, norms, routers and the residual in 32-bit. */
+ * a bf16 cache of latents, keys and values; positions, recurrent state and gates, scores, norms, routers and the residual in 32-bit. */
 int lumen_decoder_new(lumen_ctx *ctx, const lumen_decoder_config *cfg, lumen_model **out);
 
 /* The interface every model shares; the lumen_llama_* entry points above are these under the reference's names. */

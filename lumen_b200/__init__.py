@@ -14,6 +14,7 @@ from .layers import (Embedding, KVCache, KVCacheInner, Linear, LlamaKVCache, Mod
                      gemv_repeat, matmul, reshape, sample_top_p)
 from .llama import LlamaConfig, LlamaModel  # noqa: E402
 from .fegetar import FegetarConfig, FegetarModel  # noqa: E402
+from .fekorax import FekoraxConfig, FekoraxModel  # noqa: E402
 from .loader import load_llama_weights, load_weights  # noqa: E402
 from .model import LanguageModel  # noqa: E402
 from .registry import load_model, model_config  # noqa: E402
@@ -25,6 +26,6 @@ __all__ = [
     "BF16", "F32", "LumenError", "Context", "Tensor", "default_context", "is_inference_mode", "is_no_grad",
     "no_grad", "set_inference_mode", "Module", "Linear", "Embedding", "RMSNorm", "SiLU", "RotaryEmbedding",
     "SelfAttention", "KVCache", "KVCacheInner", "LlamaKVCache", "LlamaConfig", "LlamaModel", "LlamaTokenizer", "load_llama_weights",
-    "FegetarConfig", "FegetarModel", "LanguageModel", "load_model", "load_weights", "model_config", "matmul", "reshape",
+    "FegetarConfig", "FegetarModel", "FekoraxConfig", "FekoraxModel", "LanguageModel", "load_model", "load_weights", "model_config", "matmul", "reshape",
     "fused_softmax", "gemv", "gemv_kn_static", "gemv_repeat", "attention_decode", "attention_decode_repeat", "sample_top_p",
 ]

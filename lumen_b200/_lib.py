@@ -42,7 +42,9 @@ class DecoderLayerC(C.Structure):
         ("heads", C.c_size_t), ("dim", C.c_size_t), ("rot_dim", C.c_size_t), ("vdim", C.c_size_t), ("kv_rank", C.c_size_t),
         ("rot_dims", C.c_size_t), ("rot_base", C.c_double), ("scale", C.c_float), ("mlp_kind", C.c_int), ("ff", C.c_size_t),
         ("experts", C.c_size_t), ("top", C.c_size_t), ("expert_ff", C.c_size_t), ("expert_limit", C.c_float),
-        ("shared_ff", C.c_size_t), ("shared_limit", C.c_float),
+        ("shared_ff", C.c_size_t), ("shared_limit", C.c_float), ("mixer", C.c_int), ("kv_heads", C.c_size_t), ("kv_from", C.c_int),
+        ("chunk", C.c_size_t), ("rot_factor", C.c_double), ("rot_low", C.c_double), ("rot_high", C.c_double), ("rot_original", C.c_double),
+        ("gate_cap", C.c_float),
     ]
 
 
@@ -53,10 +55,13 @@ class DecoderConfigC(C.Structure):
         ("vocab_size", C.c_size_t), ("width", C.c_size_t), ("num_layers", C.c_size_t), ("layers", C.POINTER(DecoderLayerC)),
         ("norm_eps", C.c_float), ("max_seq_len", C.c_size_t), ("bigram_buckets", C.c_size_t), ("bigram_mul_prev", C.c_size_t),
         ("bigram_mul_cur", C.c_size_t), ("side_dim", C.c_size_t), ("weight_dtype", C.c_int),
+        ("embed_scale", C.c_float), ("tied_head", C.c_int), ("norms", C.c_int),
     ]
 
 
-MLP_NONE, MLP_DENSE, MLP_MOE = 0, 1, 2
+MIXER_LATENT, MIXER_ATTENTION, MIXER_MLSTM = 0, 1, 2
+MLP_NONE, MLP_DENSE, MLP_MOE, MLP_GATED_GELU = 0, 1, 2, 3
+NORM_OUTPUT, NORM_BOTH = 0, 1
 
 _P = C.c_void_p
 _PP = C.POINTER(C.c_void_p)

@@ -1,13 +1,14 @@
 // C ABI: models given as a list of layers (lumen_decoder_new) on one GPU; the entry points they share with LlamaModel are in
 // model_base.cu.
 //
-// Memory: one device slab holds every weight (the query, latent and gate projections of a layer are stored back to back, so
-// that they are one product; gate and up rows of a gated feed-forward alternate in blocks of 64, experts follow one another),
-// one slab per set of caches holds the latent caches of all layers, one workspace the activations.  A sequence's state is
-// its layers' caches and its last token id (the bigram embedding looks back across steps).
+// Memory: one device slab holds every weight (the projections that read a layer's input are stored back to back, so that they are
+// one product; gate and up rows of a gated feed-forward alternate in blocks of 64, experts follow one another), one slab per set
+// of caches holds what all layers keep (latents, keys and values, or a recurrent state), one workspace the activations.  A
+// sequence's state is its layers' caches and its last token id (the bigram embedding looks back across steps); a recurrent
+// state counts as zeros while the sequence has no positions, so that resetting a cache resets its length alone.
 //
-// A step of one row streams the weights through vector-matrix kernels; the norm of a sublayer's output and the residual
-// sum are formed by the kernel that reads the result next.  It is captured once per split count into a CUDA graph.  Steps of
+// A step of one row streams the weights through vector-matrix kernels; the norm of a sublayer's output, the residual sum
+// and the norm before the next sublayer are formed by the kernel that reads the result next.  It is captured once per split count into a CUDA graph.  Steps of
 // several rows run every product on the tensor cores (bf16 models) with finishing kernels that write the next product's operand.
 #include <algorithm>
 #include <cmath>
@@ -28,15 +29,22 @@ struct Slot {  // where a parameter goes
 };
 
 struct LayerW {
-    char *proj = nullptr;  // [H * (dim + rot_dim) + rank + rot_dim + H, W]
+    // [proj_rows, W].  Latent attention: queries, latent and shared key part (u_kv), gates (u_gate).  Attention: queries, keys (u_k)
+    // and values (u_v) where the layer has its own, gates (u_gate).  Matrix memory: queries, keys (u_k), values (u_v), output
+    // gates (u_gate), and the 2 H rows of the input and forget gates, which are a product of their own in steps of several rows.
+    char *proj = nullptr;
     char *uk = nullptr, *uv = nullptr, *o = nullptr;
-    float *latent_gain = nullptr, *norm1 = nullptr, *norm2 = nullptr, *side_norm = nullptr;
-    char *up = nullptr, *down = nullptr;                      // dense
+    float *latent_gain = nullptr, *side_norm = nullptr;
+    float *pre1 = nullptr, *pre2 = nullptr;                   // gains of the norms before the sublayers (null: none)
+    float *norm1 = nullptr, *norm2 = nullptr;                 // gains of the norms of their outputs
+    float *q_gain = nullptr, *k_gain = nullptr, *sink = nullptr;  // attention
+    float *z_bias = nullptr, *head_gain = nullptr;            // matrix memory
+    char *up = nullptr, *down = nullptr;                      // dense (up: gate and up rows where it is gated)
     char *router = nullptr, *gate_up = nullptr, *edown = nullptr;  // experts
     char *sgate_up = nullptr, *sdown = nullptr;               // shared expert
     char *side_gate = nullptr, *side_proj = nullptr;
     float *cos_t = nullptr, *sin_t = nullptr;
-    size_t proj_rows = 0, u_kv = 0, u_gate = 0, pitch = 0;
+    size_t proj_rows = 0, main_rows = 0, u_kv = 0, u_k = 0, u_v = 0, u_gate = 0, pitch = 0;  // main_rows: without the 2 H gate rows
 };
 
 // An activation matrix as the next product reads it: f32, or bf16 hi (and lo).
@@ -49,7 +57,7 @@ struct Workspace {
     size_t M = 0;
     char *base = nullptr;
     float *x[2] = {nullptr, nullptr}, *u = nullptr, *y = nullptr, *c = nullptr, *nx = nullptr, *last_x = nullptr;
-    Act xa, att, act, side;  // xa.f unused: the residual itself
+    Act xa, att, act, side;  // xa: what the next sublayer reads (xa.f is the residual itself in models without norms before them)
     void *qf = nullptr;
     float *part_ctx = nullptr, *part_ml = nullptr;
     // experts
@@ -87,7 +95,14 @@ struct lumen_decoder : lumen_model {
     int run_forward(size_t b, size_t s, lumen_kv_cache **caches, bool last_only) override;
     size_t weight_bytes() const override { return stream_bytes; }
 
+    void cache_shape(size_t l, lumen_kv_cache *c) const;
+    int rotation_tables(size_t l, float *cos_t, float *sin_t);
+    bool norms_before() const { return cfg.norms == LUMEN_NORM_BOTH; }
     LatentArgs latent_args(size_t l, lumen_kv_cache *c, size_t B, size_t S) const;
+    GroupedArgs grouped_args(size_t l, lumen_kv_cache *c, size_t B, size_t S) const;
+    MlstmArgs mlstm_args(size_t l, lumen_kv_cache *c, size_t B, size_t S) const;
+    int pick_splits(size_t l, lumen_kv_cache *c, size_t B, size_t S) const;  // pieces of the context in the row kernels (1: no such thing)
+    int mix_rows(size_t l, lumen_kv_cache *c, size_t B, size_t S);           // projections and mixer of a step of several rows -> ws.att
     MoeArgs moe_args(size_t l, size_t M) const;
     int step_row(lumen_kv_cache **caches);
     int step_rows(size_t B, size_t S, lumen_kv_cache **caches, bool last_only);
@@ -124,7 +139,8 @@ int lumen_decoder::build() {
         return o;
     };
     struct Off {
-        size_t proj, uk, uv, o, lg, n1, n2 = 0, sn = 0, up = 0, down = 0, router = 0, gu = 0, ed = 0, sgu = 0, sd = 0, sg = 0, sp = 0, cos, sin;
+        size_t proj, uk = 0, uv = 0, o, lg = 0, n1, n2 = 0, p1 = 0, p2 = 0, qg = 0, kg = 0, sink = 0, zb = 0, hg = 0, sn = 0, up = 0, down = 0, router = 0,
+            gu = 0, ed = 0, sgu = 0, sd = 0, sg = 0, sp = 0, cos, sin;
     };
     std::vector<Off> lo(L);
     const size_t o_embed = matrix("embed", V, W);
@@ -136,28 +152,70 @@ int lumen_decoder::build() {
         LayerW &w = lw[l];
         Off &f = lo[l];
         const std::string p = "l" + std::to_string(l) + ".";
-        const size_t qn = c.heads * (c.dim + c.rot_dim), kvn = c.kv_rank + c.rot_dim;
-        w.u_kv = qn; w.u_gate = qn + kvn; w.proj_rows = qn + kvn + c.heads;
-        w.pitch = align_up(kvn, 16);
+        // projections of the layer's input, back to back: (name, rows)
+        struct Part { const char *name = ""; size_t rows = 0; };
+        Part parts[6];
+        const size_t H = c.heads;
+        if (c.mixer == LUMEN_MIXER_LATENT) {
+            const size_t qn = H * (c.dim + c.rot_dim), kvn = c.kv_rank + c.rot_dim;
+            parts[0] = {"q", qn}; parts[1] = {"dkv", kvn}; parts[2] = {"g", H};
+            w.u_kv = qn; w.u_gate = qn + kvn;
+            w.pitch = align_up(kvn, 16);
+        } else if (c.mixer == LUMEN_MIXER_ATTENTION) {
+            const size_t kn = c.kv_from < 0 ? c.kv_heads * c.dim : 0, vn = c.kv_from < 0 ? c.kv_heads * c.vdim : 0;
+            parts[0] = {"q", H * c.dim}; parts[1] = {"k", kn}; parts[2] = {"v", vn}; parts[3] = {"g", H};
+            w.u_k = H * c.dim; w.u_v = w.u_k + kn; w.u_gate = w.u_v + vn;
+        } else {
+            parts[0] = {"q", H * c.dim}; parts[1] = {"k", H * c.dim}; parts[2] = {"v", H * c.vdim}; parts[3] = {"g", H * c.vdim};
+            parts[4] = {"i", H}; parts[5] = {"f", H};
+            w.u_k = H * c.dim; w.u_v = 2 * H * c.dim; w.u_gate = w.u_v + H * c.vdim;
+        }
+        for (const Part &q : parts) w.proj_rows += q.rows;
+        w.main_rows = w.proj_rows - (c.mixer == LUMEN_MIXER_MLSTM ? 2 * H : 0);
         f.proj = take(w.proj_rows * W * esz);
-        add(p + "mix.q", f.proj, qn, W, dt);
-        add(p + "mix.dkv", f.proj + qn * W * esz, kvn, W, dt);
-        add(p + "mix.g", f.proj + (qn + kvn) * W * esz, c.heads, W, dt);
-        f.lg = vec(p + "mix.dkv.norm", c.kv_rank, false);
-        f.uk = matrix(p + "mix.uk", c.heads * c.dim, c.kv_rank);
-        f.uv = matrix(p + "mix.uv", c.heads * c.vdim, c.kv_rank);
-        f.o = matrix(p + "mix.o", W, c.heads * c.vdim);
-        f.n1 = vec(p + "norm1", W, true);
-        stream_bytes += (w.proj_rows * W + c.heads * (c.dim + c.vdim) * c.kv_rank + W * c.heads * c.vdim) * esz;
+        size_t at_row = 0;
+        for (const Part &q : parts) {
+            if (q.rows) add(p + "mix." + q.name, f.proj + at_row * W * esz, q.rows, W, dt);
+            at_row += q.rows;
+        }
+        stream_bytes += w.proj_rows * W * esz;
+        if (c.mixer == LUMEN_MIXER_LATENT) {
+            f.lg = vec(p + "mix.dkv.norm", c.kv_rank, false);
+            f.uk = matrix(p + "mix.uk", H * c.dim, c.kv_rank);
+            f.uv = matrix(p + "mix.uv", H * c.vdim, c.kv_rank);
+            stream_bytes += H * (c.dim + c.vdim) * c.kv_rank * esz;
+        } else if (c.mixer == LUMEN_MIXER_ATTENTION) {
+            f.qg = vec(p + "mix.q.norm", c.dim, false);
+            if (c.kv_from < 0) f.kg = vec(p + "mix.k.norm", c.dim, false);
+            f.sink = vec(p + "mix.sink", H, false);
+        } else {
+            f.hg = vec(p + "mix.norm", H * c.vdim, false);
+            f.zb = take(2 * H * 4);
+            add(p + "mix.i.b", f.zb, H, 0, LUMEN_F32);
+            add(p + "mix.f.b", f.zb + H * 4, H, 0, LUMEN_F32);
+        }
+        f.o = matrix(p + "mix.o", W, H * c.vdim);
+        stream_bytes += W * H * c.vdim * esz;
+        const bool both = norms_before();  // norm<i> before and norm<i>b after a sublayer, gains as they are; else norm<i> after it, around one
+        if (both) f.p1 = vec(p + "norm1", W, false);
+        f.n1 = vec(p + (both ? "norm1b" : "norm1"), W, !both);
         auto gated = [&](const std::string &name, size_t at, size_t ff) {
             add(name + ".gate", at, ff, W, dt, false, 0);
             add(name + ".up", at, ff, W, dt, false, 1);
         };
-        if (c.mlp_kind != LUMEN_MLP_NONE) f.n2 = vec(p + "norm2", W, true);
+        if (c.mlp_kind != LUMEN_MLP_NONE) {
+            if (both) f.p2 = vec(p + "norm2", W, false);
+            f.n2 = vec(p + (both ? "norm2b" : "norm2"), W, !both);
+        }
         if (c.mlp_kind == LUMEN_MLP_DENSE) {
             f.up = matrix(p + "mlp.up", c.ff, W);
             f.down = matrix(p + "mlp.down", W, c.ff);
             stream_bytes += 2 * c.ff * W * esz;
+        } else if (c.mlp_kind == LUMEN_MLP_GATED_GELU) {
+            f.up = take(gated_rows(c.ff) * W * esz);
+            gated(p + "mlp", f.up, c.ff);
+            f.down = matrix(p + "mlp.down", W, c.ff);
+            stream_bytes += 3 * c.ff * W * esz;
         } else if (c.mlp_kind == LUMEN_MLP_MOE) {
             const size_t gr = gated_rows(c.expert_ff);
             f.router = matrix(p + "mlp.router", c.experts, W);
@@ -184,13 +242,14 @@ int lumen_decoder::build() {
         // layers that turn alike share their tables
         f.cos = f.sin = 0;
         for (size_t k = 0; k < l && !f.cos; ++k)
-            if (lc[k].rot_dims == c.rot_dims && lc[k].rot_base == c.rot_base) { f.cos = lo[k].cos; f.sin = lo[k].sin; }
+            if (lc[k].rot_dims == c.rot_dims && lc[k].rot_base == c.rot_base && lc[k].rot_factor == c.rot_factor && lc[k].rot_low == c.rot_low &&
+                lc[k].rot_high == c.rot_high && lc[k].rot_original == c.rot_original) { f.cos = lo[k].cos; f.sin = lo[k].sin; }
         if (!f.cos) {
             f.cos = take(cfg.max_seq_len * (c.rot_dims / 2) * 4);
             f.sin = take(cfg.max_seq_len * (c.rot_dims / 2) * 4);
         }
     }
-    const size_t o_fn = vec("final.norm", W, true), o_head = matrix("head", V, W);
+    const size_t o_fn = vec("final.norm", W, !norms_before()), o_head = cfg.tied_head ? o_embed : matrix("head", V, W);
     stream_bytes += V * W * esz;
     LUMEN_CUDA(ctx, cudaMalloc(&wslab, std::max<size_t>(off, 256)));
     LUMEN_CUDA(ctx, cudaMemsetAsync(wslab, 0, off, ctx->stream));  // (blocks of gate and up rows are padded with zeros)
@@ -204,25 +263,43 @@ int lumen_decoder::build() {
         LayerW &w = lw[l];
         const Off &f = lo[l];
         w.proj = at(f.proj); w.uk = at(f.uk); w.uv = at(f.uv); w.o = at(f.o); w.latent_gain = atf(f.lg); w.norm1 = atf(f.n1);
+        if (norms_before()) { w.pre1 = atf(f.p1); w.pre2 = atf(f.p2); }
+        w.q_gain = atf(f.qg); w.k_gain = atf(f.kg); w.sink = atf(f.sink); w.z_bias = atf(f.zb); w.head_gain = atf(f.hg);
         w.norm2 = atf(f.n2); w.up = at(f.up); w.down = at(f.down); w.router = at(f.router); w.gate_up = at(f.gu); w.edown = at(f.ed);
         w.sgate_up = at(f.sgu); w.sdown = at(f.sd); w.side_gate = at(f.sg); w.side_proj = at(f.sp); w.side_norm = atf(f.sn);
         w.cos_t = atf(f.cos); w.sin_t = atf(f.sin);
         bool first = true;
         for (size_t k = 0; k < l; ++k) first = first && lo[k].cos != f.cos;
-        const size_t half = lc[l].rot_dims / 2;
-        if (!first || half == 0) continue;
-        std::vector<float> ch(cfg.max_seq_len * half), sh(ch.size());
-        for (size_t i = 0; i < half; ++i) {
-            const double freq = std::pow(lc[l].rot_base, -2.0 * (double)i / (double)lc[l].rot_dims);
-            for (size_t p = 0; p < cfg.max_seq_len; ++p) {
-                ch[p * half + i] = (float)std::cos((double)p * freq);
-                sh[p * half + i] = (float)std::sin((double)p * freq);
-            }
-        }
-        LUMEN_CUDA(ctx, cudaMemcpy(w.cos_t, ch.data(), ch.size() * 4, cudaMemcpyHostToDevice));
-        LUMEN_CUDA(ctx, cudaMemcpy(w.sin_t, sh.data(), sh.size() * 4, cudaMemcpyHostToDevice));
+        if (first && lc[l].rot_dims) LUMEN_TRY(rotation_tables(l, w.cos_t, w.sin_t));
     }
     n_expected = slots.size();
+    return LUMEN_OK;
+}
+
+// cos and sin of position * frequency, computed in double.  With frequency scaling, wavelengths above rot_original / rot_low are
+// stretched by rot_factor, those below rot_original / rot_high stay, and frequencies between are interpolated.
+int lumen_decoder::rotation_tables(size_t l, float *cos_t, float *sin_t) {
+    const lumen_decoder_layer &c = lc[l];
+    const size_t half = c.rot_dims / 2;
+    std::vector<float> ch(cfg.max_seq_len * half), sh(ch.size());
+    for (size_t i = 0; i < half; ++i) {
+        double freq = std::pow(c.rot_base, -2.0 * (double)i / (double)c.rot_dims);
+        if (c.rot_factor != 0.0) {
+            const double turns = c.rot_original * freq / (2.0 * M_PI);  // within the original length
+            if (turns < c.rot_low) {
+                freq /= c.rot_factor;
+            } else if (turns <= c.rot_high) {
+                const double s = (turns - c.rot_low) / (c.rot_high - c.rot_low);
+                freq = (1.0 - s) * freq / c.rot_factor + s * freq;
+            }
+        }
+        for (size_t p = 0; p < cfg.max_seq_len; ++p) {
+            ch[p * half + i] = (float)std::cos((double)p * freq);
+            sh[p * half + i] = (float)std::sin((double)p * freq);
+        }
+    }
+    LUMEN_CUDA(ctx, cudaMemcpy(cos_t, ch.data(), ch.size() * 4, cudaMemcpyHostToDevice));
+    LUMEN_CUDA(ctx, cudaMemcpy(sin_t, sh.data(), sh.size() * 4, cudaMemcpyHostToDevice));
     return LUMEN_OK;
 }
 
@@ -259,13 +336,42 @@ int lumen_decoder::set_param(const char *name, const void *host_data, const size
     return LUMEN_OK;
 }
 
+// What layer l's cache holds (see lumen_kv_cache).
+void lumen_decoder::cache_shape(size_t l, lumen_kv_cache *c) const {
+    const lumen_decoder_layer &k = lc[l];
+    c->dtype = dt;
+    if (k.mixer == LUMEN_MIXER_LATENT) {
+        c->kind = lumen_kv_cache::kLatent;
+        c->h_kv = 1; c->d = lw[l].pitch;
+    } else if (k.mixer == LUMEN_MIXER_ATTENTION) {
+        c->kind = lumen_kv_cache::kRows;
+        c->h_kv = k.kv_heads; c->d = k.dim; c->dv = k.vdim;
+    } else {
+        c->kind = lumen_kv_cache::kState;
+        c->h_kv = k.heads; c->d = k.dim; c->dv = k.vdim;
+        c->dtype = LUMEN_F32;
+    }
+}
+
 int lumen_decoder::init_kv_caches(size_t batch, lumen_kv_cache **out) {
     if (batch == 0) return set_error(ctx, LUMEN_ERR_SHAPE, "caches for an empty batch");
-    std::vector<size_t> at(L);
+    std::vector<size_t> at(L), at2(L);
     size_t off = 0;
+    auto take = [&](size_t bytes) { const size_t o = off; off += align_up(bytes, 256); return o; };
     for (size_t l = 0; l < L; ++l) {
-        at[l] = off;
-        off += align_up(batch * cfg.max_seq_len * lw[l].pitch * esz, 256);
+        const lumen_decoder_layer &k = lc[l];
+        if (k.mixer == LUMEN_MIXER_LATENT) {
+            at[l] = at2[l] = take(batch * cfg.max_seq_len * lw[l].pitch * esz);
+        } else if (k.mixer == LUMEN_MIXER_MLSTM) {
+            at[l] = take(batch * k.heads * k.dim * k.vdim * 4);
+            at2[l] = take(batch * k.heads * (k.dim + 1) * 4);
+        } else if (k.kv_from >= 0) {  // that layer's rows
+            at[l] = at[k.kv_from];
+            at2[l] = at2[k.kv_from];
+        } else {
+            at[l] = take(batch * k.kv_heads * cfg.max_seq_len * k.dim * esz);
+            at2[l] = take(batch * k.kv_heads * cfg.max_seq_len * k.vdim * esz);
+        }
     }
     const size_t lens_at = off, last_at = lens_at + align_up(L * sizeof(int), 256);
     int rc = LUMEN_OK;
@@ -274,8 +380,11 @@ int lumen_decoder::init_kv_caches(size_t batch, lumen_kv_cache **out) {
     char *base = static_cast<char *>(slab->ptr);
     for (size_t l = 0; l < L; ++l) {
         auto *c = new lumen_kv_cache();
-        c->ctx = ctx; c->b = batch; c->h_kv = 1; c->max_seq = cfg.max_seq_len; c->d = lw[l].pitch; c->dtype = dt;
+        const lumen_decoder_layer &k = lc[l];
+        c->ctx = ctx; c->b = batch; c->max_seq = cfg.max_seq_len;
+        cache_shape(l, c);
         c->k = reinterpret_cast<float *>(base + at[l]);
+        if (k.mixer != LUMEN_MIXER_LATENT) c->v = reinterpret_cast<float *>(base + at2[l]);
         c->d_len = reinterpret_cast<int *>(base + lens_at) + l;
         c->last_tok = reinterpret_cast<int *>(base + last_at);
         c->seen_abort = ctx->abort_gen;
@@ -293,7 +402,10 @@ int lumen_decoder::check_caches(size_t b, size_t s, lumen_kv_cache **caches, siz
         lumen_kv_cache *c = caches[l];
         if (!c) return set_error(ctx, LUMEN_ERR_INVALID, "null KV cache for layer %zu", l);
         LUMEN_TRY(kv_resync_len(c));
-        if (c->b != b || c->h_kv != 1 || c->d != lw[l].pitch || c->dtype != dt || c->max_seq != cfg.max_seq_len || !c->last_tok)
+        lumen_kv_cache want;
+        cache_shape(l, &want);
+        if (c->b != b || c->kind != want.kind || c->h_kv != want.h_kv || c->d != want.d || c->dv != want.dv || c->dtype != want.dtype ||
+            c->max_seq != cfg.max_seq_len || !c->last_tok)
             return set_error(ctx, LUMEN_ERR_SHAPE, "KV cache %zu [%zu,%zu,%zu,%zu] does not match batch %zu / model", l, c->b, c->h_kv, c->max_seq, c->d, b);
         if (c->slab != caches[0]->slab || c->d_len != caches[0]->d_len + l)
             return set_error(ctx, LUMEN_ERR_INVALID, "KV caches come from different sets, or are not in layer order");
@@ -319,12 +431,19 @@ int lumen_decoder::ensure_workspace(size_t M) {
         const lumen_decoder_layer &k = lc[l];
         u = std::max(u, lw[l].proj_rows);
         att = std::max(att, k.heads * k.vdim);
-        q = std::max(q, k.heads * lw[l].pitch);
-        heads = std::max(heads, k.heads);
-        rank = std::max(rank, k.kv_rank);
+        if (k.mixer == LUMEN_MIXER_MLSTM) {
+            zmax = std::max(zmax, 2 * k.heads);
+        } else {
+            q = std::max(q, k.heads * lw[l].pitch);
+            heads = std::max(heads, k.heads);
+            rank = std::max(rank, k.mixer == LUMEN_MIXER_LATENT ? k.kv_rank : k.vdim);
+        }
         if (k.mlp_kind == LUMEN_MLP_DENSE) {
             act = std::max(act, k.ff);
             c = std::max(c, k.ff);
+        } else if (k.mlp_kind == LUMEN_MLP_GATED_GELU) {
+            act = std::max(act, k.ff);
+            c = std::max(c, gated_rows(k.ff));
         } else if (k.mlp_kind == LUMEN_MLP_MOE) {
             act = std::max(act, k.shared_ff);
             c = std::max(c, gated_rows(k.shared_ff));
@@ -348,13 +467,13 @@ int lumen_decoder::ensure_workspace(size_t M) {
                  o_z = take(M * zmax * 4), o_wt = take(M * topmax * 4), o_rs = take(M * topmax * 4), o_ye = take(bf ? M * topmax * W * 2 : 0),
                  o_va = take(M * vact * 4), o_sel = take(M * topmax * 4), o_pos = take(M * topmax * 4), o_src = take(M * topmax * 4), o_nt = take(4),
                  o_tiles = take(tiles * sizeof(int4)), o_xp = take(bf ? M * permx * 2 : 0), o_ap = take(bf ? M * perma * 2 : 0),
-                 o_ids = take(M * 4), o_lg = take(M * V * 4);
+                 o_ids = take(M * 4), o_lg = take(M * V * 4), o_xn = take(norms_before() ? M * W * 4 : 0);
     LUMEN_CUDA(ctx, cudaMalloc(&ws.base, off));
     auto f = [&](size_t o) { return reinterpret_cast<float *>(ws.base + o); };
     auto h = [&](size_t o) { return reinterpret_cast<__nv_bfloat16 *>(ws.base + o); };
     auto i = [&](size_t o) { return reinterpret_cast<int *>(ws.base + o); };
     ws.x[0] = f(o_x0); ws.x[1] = f(o_x1); ws.u = f(o_u); ws.y = f(o_y); ws.c = f(o_c); ws.nx = f(o_nx); ws.last_x = f(o_last);
-    ws.xa.f = ws.x[0];
+    ws.xa.f = norms_before() ? f(o_xn) : ws.x[0];
     ws.att.f = f(o_att); ws.act.f = f(o_act); ws.side.f = f(o_sd);
     if (bf) { ws.xa.hi = h(o_xh); ws.xa.lo = h(o_xl); ws.att.hi = h(o_ah); ws.act.hi = h(o_gh); ws.side.hi = h(o_sh); }
     ws.qf = ws.base + o_q; ws.part_ctx = f(o_pc); ws.part_ml = f(o_pm);
@@ -382,6 +501,38 @@ LatentArgs lumen_decoder::latent_args(size_t l, lumen_kv_cache *c, size_t B, siz
     return a;
 }
 
+GroupedArgs lumen_decoder::grouped_args(size_t l, lumen_kv_cache *c, size_t B, size_t S) const {
+    const lumen_decoder_layer &k = lc[l];
+    const LayerW &w = lw[l];
+    GroupedArgs a;
+    a.B = B; a.S = S; a.H = k.heads; a.G = k.kv_heads; a.dim = k.dim; a.vdim = k.vdim; a.rot_dims = k.rot_dims; a.chunk = k.chunk;
+    a.max_seq = cfg.max_seq_len; a.dt = dt;
+    a.u = ws.u; a.u_ld = w.proj_rows; a.u_k = w.u_k; a.u_v = w.u_v; a.u_gate = w.u_gate; a.own_kv = k.kv_from < 0;
+    a.q_gain = w.q_gain; a.k_gain = w.k_gain; a.sink = w.sink; a.eps = cfg.norm_eps; a.scale = k.scale; a.cos_t = w.cos_t; a.sin_t = w.sin_t;
+    a.k = c->k; a.v = c->v; a.d_len = c->d_len; a.past = c->len;
+    a.part_ctx = ws.part_ctx; a.part_ml = ws.part_ml;
+    return a;
+}
+
+MlstmArgs lumen_decoder::mlstm_args(size_t l, lumen_kv_cache *c, size_t B, size_t S) const {
+    const lumen_decoder_layer &k = lc[l];
+    const LayerW &w = lw[l];
+    MlstmArgs a;
+    a.B = B; a.S = S; a.H = k.heads; a.dim = k.dim; a.vdim = k.vdim; a.cap = k.gate_cap; a.eps = cfg.norm_eps;
+    a.u = ws.u; a.u_ld = w.main_rows; a.u_k = w.u_k; a.u_v = w.u_v; a.u_g = w.u_gate;
+    a.z = ws.z; a.z_ld = 2 * k.heads; a.z_bias = w.z_bias; a.head_gain = w.head_gain;
+    a.state = c->k; a.norm = c->v; a.mx = c->v + B * k.heads * k.dim; a.d_len = c->d_len; a.past = c->len;
+    return a;
+}
+
+int lumen_decoder::pick_splits(size_t l, lumen_kv_cache *c, size_t B, size_t S) const {
+    switch (lc[l].mixer) {
+        case LUMEN_MIXER_LATENT: return latent_pick_splits(latent_args(l, c, B, S), c->len + S, ctx->num_sms);
+        case LUMEN_MIXER_ATTENTION: return grouped_pick_splits(grouped_args(l, c, B, S), ctx->num_sms);
+        default: return 1;
+    }
+}
+
 MoeArgs lumen_decoder::moe_args(size_t l, size_t M) const {
     const lumen_decoder_layer &k = lc[l];
     const LayerW &w = lw[l];
@@ -400,11 +551,11 @@ int lumen_decoder::step_row(lumen_kv_cache **caches) {
     EmbedArgs e;
     e.ids = ws.ids; e.embed = embed; e.bigram = bigram; e.dt = dt; e.vocab = V; e.dim = W;
     e.buckets = cfg.bigram_buckets; e.mul_prev = cfg.bigram_mul_prev; e.mul_cur = cfg.bigram_mul_cur;
-    e.d_len = caches[0]->d_len; e.last_tok = caches[0]->last_tok; e.x = ws.x[0];
+    e.d_len = caches[0]->d_len; e.last_tok = caches[0]->last_tok; e.x = ws.x[0]; e.scale = cfg.embed_scale;
     LUMEN_TRY(launch_embed(ctx, e, s));
     int cur = 0;
     Pending pend;
-    // y = w . x, where x is the residual after the pending output (which is thereby settled)
+    // y = w . x, where x is the residual after the pending output (which is thereby settled), normed with norm_w if given
     auto from_residual = [&](const void *w, size_t N, float *out, StepFinish::Kind act, size_t layer, const float *norm_w = nullptr) -> int {
         GemvStepArgs g;
         g.res = ws.x[cur]; g.eps = cfg.norm_eps; g.w = w; g.wdt = dt; g.K = W; g.N = N; g.out = out; g.act = act; g.norm_w = norm_w;
@@ -427,16 +578,31 @@ int lumen_decoder::step_row(lumen_kv_cache **caches) {
     for (size_t l = 0; l < L; ++l) {
         const lumen_decoder_layer &k = lc[l];
         const LayerW &w = lw[l];
-        LUMEN_TRY(from_residual(w.proj, w.proj_rows, ws.u, StepFinish::kStore, l));
-        LatentArgs a = latent_args(l, caches[l], 1, 1);
-        a.nsplit = latent_pick_splits(a, a.past + 1, ctx->num_sms);
-        a.out = ws.att.f;
-        LUMEN_TRY(launch_latent_absorb(ctx, a, true, s));
-        LUMEN_TRY(latent_mma_usable(a) ? launch_latent_mma(ctx, a, s) : launch_latent_scores(ctx, a, s));
-        LUMEN_TRY(launch_latent_value(ctx, a, s));
+        LUMEN_TRY(from_residual(w.proj, w.proj_rows, ws.u, StepFinish::kStore, l, w.pre1));
+        if (k.mixer == LUMEN_MIXER_LATENT) {
+            LatentArgs a = latent_args(l, caches[l], 1, 1);
+            a.nsplit = pick_splits(l, caches[l], 1, 1);
+            a.out = ws.att.f;
+            LUMEN_TRY(launch_latent_absorb(ctx, a, true, s));
+            LUMEN_TRY(latent_mma_usable(a) ? launch_latent_mma(ctx, a, s) : launch_latent_scores(ctx, a, s));
+            LUMEN_TRY(launch_latent_value(ctx, a, s));
+        } else if (k.mixer == LUMEN_MIXER_ATTENTION) {
+            GroupedArgs a = grouped_args(l, caches[l], 1, 1);
+            a.nsplit = pick_splits(l, caches[l], 1, 1);
+            a.out = ws.att.f;
+            LUMEN_TRY(launch_grouped_attention(ctx, a, a.own_kv, s));
+        } else {
+            MlstmArgs a = mlstm_args(l, caches[l], 1, 1);
+            a.z = ws.u + w.main_rows;  // (one row: all projections are one product)
+            a.out = ws.att.f;
+            LUMEN_TRY(launch_mlstm_step(ctx, a, s));
+        }
         LUMEN_TRY(plain(ws.att.f, w.o, k.heads * k.vdim, w.norm1));
         if (k.mlp_kind == LUMEN_MLP_DENSE) {
             LUMEN_TRY(from_residual(w.up, k.ff, ws.act.f, StepFinish::kGelu, l));
+            LUMEN_TRY(plain(ws.act.f, w.down, k.ff, w.norm2));
+        } else if (k.mlp_kind == LUMEN_MLP_GATED_GELU) {
+            LUMEN_TRY(from_residual(w.up, k.ff, ws.act.f, StepFinish::kGated, l, w.pre2));
             LUMEN_TRY(plain(ws.act.f, w.down, k.ff, w.norm2));
         } else if (k.mlp_kind == LUMEN_MLP_MOE) {
             LUMEN_TRY(from_residual(w.router, k.experts, ws.z, StepFinish::kStore, l));
@@ -473,6 +639,53 @@ int lumen_decoder::product(const Act &a, size_t lda, const void *w, size_t M, si
     return fin ? launch_step_finish(ctx, c, 1, M, N, *fin, s) : LUMEN_OK;
 }
 
+int lumen_decoder::mix_rows(size_t l, lumen_kv_cache *c, size_t B, size_t S) {
+    cudaStream_t s = ctx->stream;
+    const lumen_decoder_layer &k = lc[l];
+    const LayerW &w = lw[l];
+    const size_t M = B * S, av = k.heads * k.vdim;
+    auto output = [&](auto &a) {
+        if (on_tensor_cores(M, av)) a.out_hi = ws.att.hi;
+        else a.out = ws.att.f;
+    };
+    if (k.mixer == LUMEN_MIXER_MLSTM) {
+        MlstmArgs a = mlstm_args(l, c, B, S);
+        output(a);
+        const char *gates = w.proj + w.main_rows * W * esz;
+        LUMEN_TRY(product(ws.xa, W, gates, M, W, 2 * k.heads, ws.z, nullptr, true));
+        if (on_tensor_cores(M, W) && mlstm_chunked_usable(a)) {
+            GemmBf16Args g;
+            g.a_hi = ws.xa.hi; g.M = M; g.K = W; g.w = reinterpret_cast<const __nv_bfloat16 *>(w.proj); g.N = w.main_rows;
+            g.out16 = reinterpret_cast<__nv_bfloat16 *>(ws.u); g.ld16 = w.main_rows; g.epi = GemmBf16Args::kBf16;
+            LUMEN_TRY(launch_gemm_bf16(ctx, g, s));
+            a.u16 = g.out16;
+            return launch_mlstm_chunked(ctx, a, s);
+        }
+        LUMEN_TRY(product(ws.xa, W, w.proj, M, W, w.main_rows, ws.u, nullptr));
+        return launch_mlstm_step(ctx, a, s);
+    }
+    LUMEN_TRY(product(ws.xa, W, w.proj, M, W, w.proj_rows, ws.u, nullptr));
+    if (k.mixer == LUMEN_MIXER_ATTENTION) {
+        GroupedArgs a = grouped_args(l, c, B, S);
+        output(a);
+        if (grouped_prefill_usable(a)) return launch_grouped_prefill(ctx, a, s);
+        a.nsplit = pick_splits(l, c, B, S);
+        const bool append = a.own_kv && S == 1;
+        if (!append) LUMEN_TRY(launch_grouped_append(ctx, a, nullptr, 0, 0, s));
+        return launch_grouped_attention(ctx, a, append, s);
+    }
+    LatentArgs a = latent_args(l, c, B, S);
+    output(a);
+    if (latent_prefill_usable(a)) {
+        LUMEN_TRY(launch_latent_append(ctx, a, s));
+        return launch_latent_prefill(ctx, a, s);
+    }
+    a.nsplit = pick_splits(l, c, B, S);
+    LUMEN_TRY(launch_latent_absorb(ctx, a, true, s));
+    LUMEN_TRY(latent_mma_usable(a) ? launch_latent_mma(ctx, a, s) : launch_latent_scores(ctx, a, s));
+    return launch_latent_value(ctx, a, s);
+}
+
 // S positions of B sequences.
 int lumen_decoder::step_rows(size_t B, size_t S, lumen_kv_cache **caches, bool last_only) {
     cudaStream_t s = ctx->stream;
@@ -481,39 +694,38 @@ int lumen_decoder::step_rows(size_t B, size_t S, lumen_kv_cache **caches, bool l
     EmbedArgs e;
     e.ids = ws.ids; e.embed = embed; e.bigram = bigram; e.dt = dt; e.B = B; e.S = S; e.vocab = V; e.dim = W;
     e.buckets = cfg.bigram_buckets; e.mul_prev = cfg.bigram_mul_prev; e.mul_cur = cfg.bigram_mul_cur;
-    e.d_len = caches[0]->d_len; e.last_tok = caches[0]->last_tok; e.x = ws.x[0]; e.hi = ws.xa.hi;
+    e.d_len = caches[0]->d_len; e.last_tok = caches[0]->last_tok; e.x = ws.x[0]; e.hi = ws.xa.hi; e.scale = cfg.embed_scale;
+    if (norms_before()) {
+        e.norm_w = lw[0].pre1; e.eps = cfg.norm_eps;
+        if (!on_tensor_cores(M, W)) e.out = ws.xa.f;
+        if (lc[0].mixer == LUMEN_MIXER_MLSTM) e.lo = ws.xa.lo;  // (its gates read a pair)
+    }
     LUMEN_TRY(launch_embed(ctx, e, s));
     // What the products of this step read of an activation: bf16 on the tensor cores, f32 otherwise.
     auto target = [&](StepFinish &f, const Act &a, size_t K) {
         if (on_tensor_cores(M, K)) f.hi = a.hi;
         else f.out = a.f;
     };
-    auto norm_add = [&](const float *gain, bool pair = false) {
+    // next: gain of the norm before the next sublayer (null: it reads the residual); pair: it reads a hi/lo pair
+    auto norm_add = [&](const float *gain, bool pair = false, const float *next = nullptr) {
         StepFinish f;
-        f.kind = StepFinish::kNormAdd; f.x = ws.x[0]; f.gain = gain; f.eps = cfg.norm_eps; f.hi = ws.xa.hi;
+        f.kind = StepFinish::kNormAdd; f.x = ws.x[0]; f.gain = gain; f.eps = cfg.norm_eps; f.hi = ws.xa.hi; f.next_gain = next;
         if (pair) f.lo = ws.xa.lo;
+        if (next && !on_tensor_cores(M, W)) f.out = ws.xa.f;
         return f;
     };
+    auto is_mlstm = [&](size_t l) { return l < L && lc[l].mixer == LUMEN_MIXER_MLSTM; };
     // Products whose activation is applied in the epilogue: enough rows that K is not split.
     const bool epilogue = M > 128;
     for (size_t l = 0; l < L; ++l) {
         const lumen_decoder_layer &k = lc[l];
         const LayerW &w = lw[l];
-        LUMEN_TRY(product(ws.xa, W, w.proj, M, W, w.proj_rows, ws.u, nullptr));
-        LatentArgs a = latent_args(l, caches[l], B, S);
         const size_t av = k.heads * k.vdim;
-        if (on_tensor_cores(M, av)) a.out_hi = ws.att.hi;
-        else a.out = ws.att.f;
-        if (latent_prefill_usable(a)) {
-            LUMEN_TRY(launch_latent_append(ctx, a, s));
-            LUMEN_TRY(launch_latent_prefill(ctx, a, s));
-        } else {
-            a.nsplit = latent_pick_splits(a, a.past + S, ctx->num_sms);
-            LUMEN_TRY(launch_latent_absorb(ctx, a, true, s));
-            LUMEN_TRY(latent_mma_usable(a) ? launch_latent_mma(ctx, a, s) : launch_latent_scores(ctx, a, s));
-            LUMEN_TRY(launch_latent_value(ctx, a, s));
-        }
-        StepFinish f1 = norm_add(w.norm1, k.mlp_kind == LUMEN_MLP_MOE);  // (the router reads the pair)
+        LUMEN_TRY(mix_rows(l, caches[l], B, S));
+        // what comes next and what it reads: the router and the gates of a matrix memory read pairs
+        const bool last = k.mlp_kind == LUMEN_MLP_NONE;  // the mixer is the layer's last sublayer
+        const float *after = l + 1 < L ? lw[l + 1].pre1 : nullptr;
+        StepFinish f1 = norm_add(w.norm1, k.mlp_kind == LUMEN_MLP_MOE || (last && is_mlstm(l + 1)), last ? after : w.pre2);
         LUMEN_TRY(product(ws.att, av, w.o, M, av, W, ws.y, &f1));
         if (k.mlp_kind == LUMEN_MLP_DENSE) {
             if (epilogue && on_tensor_cores(M, W) && on_tensor_cores(M, k.ff)) {
@@ -527,11 +739,25 @@ int lumen_decoder::step_rows(size_t B, size_t S, lumen_kv_cache **caches, bool l
                 target(fa, ws.act, k.ff);
                 LUMEN_TRY(product(ws.xa, W, w.up, M, W, k.ff, ws.c, &fa));
             }
-            StepFinish f2 = norm_add(w.norm2);
+            StepFinish f2 = norm_add(w.norm2, is_mlstm(l + 1), after);
+            LUMEN_TRY(product(ws.act, k.ff, w.down, M, k.ff, W, ws.y, &f2));
+        } else if (k.mlp_kind == LUMEN_MLP_GATED_GELU) {
+            if (epilogue && on_tensor_cores(M, W) && on_tensor_cores(M, k.ff)) {
+                GemmBf16Args g;
+                g.a_hi = ws.xa.hi; g.M = M; g.K = W; g.w = reinterpret_cast<const __nv_bfloat16 *>(w.up); g.N = gated_rows(k.ff);
+                g.ff = k.ff; g.out16 = ws.act.hi; g.ld16 = k.ff; g.epi = GemmBf16Args::kGatedGelu;
+                LUMEN_TRY(launch_gemm_bf16(ctx, g, s));
+            } else {
+                StepFinish fa;
+                fa.kind = StepFinish::kGated; fa.glu = StepFinish::kGeluTanh; fa.ff = k.ff;
+                target(fa, ws.act, k.ff);
+                LUMEN_TRY(product(ws.xa, W, w.up, M, W, gated_rows(k.ff), ws.c, &fa));
+            }
+            StepFinish f2 = norm_add(w.norm2, is_mlstm(l + 1), after);
             LUMEN_TRY(product(ws.act, k.ff, w.down, M, k.ff, W, ws.y, &f2));
         } else if (k.mlp_kind == LUMEN_MLP_MOE) {
             LUMEN_TRY(product(ws.xa, W, w.router, M, W, k.experts, ws.z, nullptr, true));
-            StepFinish f2 = norm_add(w.norm2);
+            StepFinish f2 = norm_add(w.norm2, is_mlstm(l + 1), after);
             if (on_tensor_cores(M, W) && on_tensor_cores(M, k.expert_ff)) {
                 MoeGroupArgs ga;
                 ga.M = M; ga.experts = k.experts; ga.top = k.top; ga.z = ws.z; ga.sel = ws.sel; ga.pos = ws.pos; ga.src = ws.src;
@@ -581,7 +807,7 @@ int lumen_decoder::step_rows(size_t B, size_t S, lumen_kv_cache **caches, bool l
             fs.table_ld = L * cfg.side_dim; fs.table_rows = V;
             target(fs, ws.side, cfg.side_dim);
             LUMEN_TRY(product(ws.xa, W, w.side_gate, M, W, cfg.side_dim, ws.c, &fs));
-            StepFinish f3 = norm_add(w.side_norm);
+            StepFinish f3 = norm_add(w.side_norm, is_mlstm(l + 1), after);
             LUMEN_TRY(product(ws.side, cfg.side_dim, w.side_proj, M, cfg.side_dim, W, ws.y, &f3));
         }
     }
@@ -615,7 +841,7 @@ int lumen_decoder::run_forward(size_t b, size_t s, lumen_kv_cache **caches, bool
         // every launch of the step reads the position from the device; only the pieces of the context are baked in
         // (a context picks the same piece counts for all layers of one geometry, so their combination grows with the context)
         unsigned key = 0;
-        for (size_t l = 0; l < L; ++l) key = key * 7 + (unsigned)latent_pick_splits(latent_args(l, caches[l], b, 1), caches[l]->len + 1, ctx->num_sms);
+        for (size_t l = 0; l < L; ++l) key = key * 7 + (unsigned)pick_splits(l, caches[l], b, 1);
         const bool one = b == 1 && W * 4 <= 200 * 1024;
         rc = run_graphed(std::make_tuple(b, (int)key, (const void *)caches[0]->k),
                          [&] {
@@ -641,13 +867,26 @@ extern "C" int lumen_decoder_new(lumen_ctx *ctx, const lumen_decoder_config *cfg
     if (!cfg->vocab_size || !cfg->width || !cfg->max_seq_len || !cfg->num_layers) return set_error(ctx, LUMEN_ERR_SHAPE, "decoder_new: empty model");
     for (size_t l = 0; l < cfg->num_layers; ++l) {
         const lumen_decoder_layer &k = cfg->layers[l];
-        if (!k.heads || !k.dim || !k.vdim || !k.kv_rank || k.rot_dims > k.rot_dim || k.rot_dims % 2)
-            return set_error(ctx, LUMEN_ERR_SHAPE, "layer %zu: latent attention sizes", l);
+        if (!k.heads || !k.dim || !k.vdim || k.rot_dims % 2) return set_error(ctx, LUMEN_ERR_SHAPE, "layer %zu: mixer sizes", l);
+        if (k.mixer == LUMEN_MIXER_LATENT) {
+            if (!k.kv_rank || k.rot_dims > k.rot_dim) return set_error(ctx, LUMEN_ERR_SHAPE, "layer %zu: latent attention sizes", l);
+        } else if (k.mixer == LUMEN_MIXER_ATTENTION) {
+            if (!k.kv_heads || k.heads % k.kv_heads || k.rot_dims > k.dim) return set_error(ctx, LUMEN_ERR_SHAPE, "layer %zu: attention sizes", l);
+            if (std::max(k.dim, k.vdim) > kGroupedMaxDim) return set_error(ctx, LUMEN_ERR_UNSUPPORTED, "layer %zu: heads of %zu / %zu numbers (at most %zu)", l, k.dim, k.vdim, kGroupedMaxDim);
+            if (k.kv_from >= 0) {
+                const lumen_decoder_layer *j = (size_t)k.kv_from < l ? &cfg->layers[k.kv_from] : nullptr;
+                if (!j || j->mixer != LUMEN_MIXER_ATTENTION || j->kv_from >= 0 || j->kv_heads != k.kv_heads || j->dim != k.dim || j->vdim != k.vdim)
+                    return set_error(ctx, LUMEN_ERR_SHAPE, "layer %zu: keys and values of layer %d", l, k.kv_from);
+            }
+        } else if (k.mixer != LUMEN_MIXER_MLSTM || !(k.gate_cap > 0.f)) {
+            return set_error(ctx, LUMEN_ERR_SHAPE, "layer %zu: mixer %d", l, k.mixer);
+        }
         if (k.kv_rank > 1024) return set_error(ctx, LUMEN_ERR_UNSUPPORTED, "layer %zu: latent of %zu numbers (at most 1024)", l, k.kv_rank);
-        if (k.mlp_kind == LUMEN_MLP_DENSE ? !k.ff : k.mlp_kind == LUMEN_MLP_MOE ? (!k.experts || !k.top || k.top > k.experts || !k.expert_ff) : k.mlp_kind != LUMEN_MLP_NONE)
+        if (k.mlp_kind == LUMEN_MLP_DENSE || k.mlp_kind == LUMEN_MLP_GATED_GELU ? !k.ff : k.mlp_kind == LUMEN_MLP_MOE ? (!k.experts || !k.top || k.top > k.experts || !k.expert_ff) : k.mlp_kind != LUMEN_MLP_NONE)
             return set_error(ctx, LUMEN_ERR_SHAPE, "layer %zu: feed-forward sizes", l);
         if (k.mlp_kind == LUMEN_MLP_MOE && k.experts > 1536) return set_error(ctx, LUMEN_ERR_UNSUPPORTED, "layer %zu: %zu experts (at most 1536)", l, k.experts);
     }
+    if (cfg->norms != LUMEN_NORM_OUTPUT && cfg->norms != LUMEN_NORM_BOTH) return set_error(ctx, LUMEN_ERR_INVALID, "decoder_new: norms %d", cfg->norms);
     auto *m = new lumen_decoder();
     m->ctx = ctx;
     m->cfg = *cfg;

@@ -351,7 +351,7 @@ int check_caches(lumen_llama *m, size_t b, size_t s, lumen_kv_cache **caches, si
         lumen_kv_cache *c = caches[l];
         if (!c) return set_error(ctx, LUMEN_ERR_INVALID, "null KV cache for layer %zu", l);
         LUMEN_TRY(kv_resync_len(c));
-        if (c->b != b || c->h_kv != m->hkv_l || c->d != m->D || !c->v)
+        if (c->b != b || c->h_kv != m->hkv_l || c->d != m->D || c->kind != lumen_kv_cache::kLlama)
             return set_error(ctx, LUMEN_ERR_SHAPE, "KV cache %zu geometry [%zu,%zu,%zu,%zu] does not match batch %zu / model", l, c->b, c->h_kv, c->max_seq, c->d, b);
         if (c->len != caches[0]->len) return set_error(ctx, LUMEN_ERR_INVALID, "KV caches have different lengths");
         if (s == 1) {  // decode asserts overflow before touching RoPE (self_attention.rs:144-149)

@@ -362,6 +362,8 @@ int lumen_kv_free(lumen_kv_cache *c) {
 int lumen_kv_read(const lumen_kv_cache *c, float *k_out, float *v_out) {
     if (!c || !k_out || (c->v && !v_out)) return LUMEN_ERR_INVALID;
     if (c->dtype != LUMEN_F32) return set_error(c->ctx, LUMEN_ERR_DTYPE, "kv_read: the cache is not f32");
+    if (c->kind == lumen_kv_cache::kRows || c->kind == lumen_kv_cache::kState)
+        return set_error(c->ctx, LUMEN_ERR_UNSUPPORTED, "kv_read: not a cache of keys and values of one size");
     const size_t bytes = c->b * c->h_kv * c->max_seq * c->d * sizeof(float);
     LUMEN_CUDA(c->ctx, cudaMemcpyAsync(k_out, c->k, bytes, cudaMemcpyDeviceToHost, c->ctx->stream));
     if (c->v) LUMEN_CUDA(c->ctx, cudaMemcpyAsync(v_out, c->v, bytes, cudaMemcpyDeviceToHost, c->ctx->stream));
@@ -371,7 +373,7 @@ int lumen_kv_read(const lumen_kv_cache *c, float *k_out, float *v_out) {
 
 int lumen_kv_write(lumen_kv_cache *c, const float *k_in, const float *v_in, size_t len) {
     if (!c || !k_in || !v_in) return LUMEN_ERR_INVALID;
-    if (!c->v || c->dtype != LUMEN_F32) return set_error(c->ctx, LUMEN_ERR_UNSUPPORTED, "kv_write: not a cache of f32 keys and values");
+    if (!c->v || c->dtype != LUMEN_F32 || c->kind != lumen_kv_cache::kLlama) return set_error(c->ctx, LUMEN_ERR_UNSUPPORTED, "kv_write: not a cache of f32 keys and values");
     if (len > c->max_seq) return set_error(c->ctx, LUMEN_ERR_KV_OVERFLOW, "KV cache overflow: len=%zu > max_seq=%zu", len, c->max_seq);
     const size_t bytes = c->b * c->h_kv * c->max_seq * c->d * sizeof(float);
     const int ilen = (int)len;
@@ -443,7 +445,7 @@ int lumen_attention_decode(lumen_ctx *ctx, const float *q_dev, const float *k_ne
                            lumen_kv_cache *cache, lumen_rope *rope, int causal, float *out_dev) {
     if (!ctx || !q_dev || !k_new_dev || !v_new_dev || !cache || !out_dev) return set_error(ctx, LUMEN_ERR_INVALID, "attention_decode: null argument");
     (void)causal;  // with S == 1 the causal test `j > past_len` never fires (self_attention.rs:255-258)
-    if (!cache->v) return set_error(ctx, LUMEN_ERR_SHAPE, "attention_decode: a latent cache holds no values");
+    if (cache->kind != lumen_kv_cache::kLlama) return set_error(ctx, LUMEN_ERR_SHAPE, "attention_decode: the cache belongs to a model given as a list of layers");
     LUMEN_TRY(kv_resync_len(cache));
     if (cache->len + 1 > cache->max_seq)
         return set_error(ctx, LUMEN_ERR_KV_OVERFLOW, "KV cache overflow: new_len=%zu > max_seq=%zu", cache->len + 1, cache->max_seq);
@@ -526,7 +528,7 @@ int lumen_self_attention_forward(lumen_self_attention *attn, const lumen_tensor 
     if (cache->b != B || cache->h_kv != Hkv || cache->d != D) return bail(set_error(ctx, LUMEN_ERR_SHAPE, "KV cache geometry does not match the layer"));
     // Order of the reference's checks: prefill runs rope.forward (range panic) before the overflow assert;
     // decode asserts overflow first (self_attention.rs:144-149 vs :334-346).
-    if (!cache->v) return bail(set_error(ctx, LUMEN_ERR_SHAPE, "self-attention: a latent cache holds no values"));
+    if (cache->kind != lumen_kv_cache::kLlama) return bail(set_error(ctx, LUMEN_ERR_SHAPE, "self-attention: the cache belongs to a model given as a list of layers"));
     if (int rs = kv_resync_len(cache)) return bail(rs);
     const size_t past = cache->len;
     if (S == 1) {

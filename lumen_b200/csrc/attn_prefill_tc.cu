@@ -72,41 +72,15 @@ struct FaParams {
     const float *gate;     // gate logits gate[row * gate_ld + h] (null: no gate)
     size_t gate_ld;
     float scale;
+    // CHUNK: a position sees its own chunk (chunk 0: everything before it); columns of V^T start at cached row v0; sink[h] joins
+    // the denominator (null: none)
+    int chunk, v0;
+    const float *sink;
     DeviceStatus *status;
 };
 
-__device__ __forceinline__ float ex2(float x) {  // 2^x, one MUFU operation (relative error 2^-22; -inf -> 0)
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-__device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
-    const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
-    return *reinterpret_cast<const uint32_t *>(&v);
-}
-
-// A wait that also ends when another thread of the CTA has given up (nobody leaves the tile loop early, so
-// every barrier keeps its full set of participants; after a failure the remaining iterations do not wait).
-__device__ __forceinline__ bool wait_or_failed(uint64_t *bar, uint32_t parity, volatile int *failed, DeviceStatus *status, int site) {
-    if (*failed) return false;
-    if (bar_try(bar, parity)) return true;
-    const long long t0 = clock64();
-    while (!bar_try(bar, parity)) {
-        if (*failed) return false;
-        if (clock64() - t0 > kTcWaitCycles) {
-            if (status && atomicCAS(&status->code, 0, LUMEN_ERR_TIMEOUT) == 0) status->detail0 = site;
-            *failed = 1;
-            return false;
-        }
-    }
-    return true;
-}
-__device__ __forceinline__ void bar_arrive(uint64_t *bar) {
-    asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(saddr(bar)) : "memory");
-}
-
 // grid (s_pad / 128, Hq, B); 8 worker warps, warp 8 (first lane) issues the MMAs, warp 9 (first lane) the copies
-template <int KB, int DV, bool PAIR>
+template <int KB, int DV, bool PAIR, bool CHUNK>
 __global__ void __launch_bounds__(kFaThreads, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_qhi, const __grid_constant__ CUtensorMap map_qlo,
                        const __grid_constant__ CUtensorMap map_khi, const __grid_constant__ CUtensorMap map_klo,
@@ -134,7 +108,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_qhi, const __grid
     // cached rows this tile can see: up to the diagonal of its last query row
     const int i_hi = min(i0 + kBQ, p.S) - 1;
     const int visible = p.causal ? min(p.total, p.past + i_hi + 1) : p.total;
-    const int nt = (visible + kBKV - 1) / kBKV;
+    // first tile: where the chunk of the first query row starts
+    auto chunk_lo = [&](int i) { return CHUNK && p.chunk ? (p.past + i) / p.chunk * p.chunk : 0; };
+    const int jt0 = CHUNK ? chunk_lo(i0) / kBKV : 0;
+    const int nt = (visible + kBKV - 1) / kBKV - jt0;
 
     if (tid == 0) {
         bar_init(&q_bar, 1);
@@ -167,8 +144,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_qhi, const __grid
         if ((tid & 31) == 0) {
             // ---- TMA producer: Q once, then K and V^T of tile j + 2 as soon as tile j has released its half stage ----
             const int q_row0 = (b * p.Hq + h) * p.s_pad + i0;
-            const int k_row0 = b * p.k_rows_b + hk * p.k_rows_h, k_col0 = hk * p.k_cols_h, r_row0 = b * p.r_rows_b;
-            const int v_row0 = (b * p.Hkv + hk) * p.vdim;
+            const int k_row0 = b * p.k_rows_b + hk * p.k_rows_h + jt0 * kBKV, k_col0 = hk * p.k_cols_h, r_row0 = b * p.r_rows_b;
+            const int v_row0 = (b * p.Hkv + hk) * p.vdim, v_col0 = jt0 * kBKV - (CHUNK ? p.v0 : 0);
             // A stage holds K (hi, lo) and V^T (hi, lo) of one tile; the two halves are refilled separately: K as
             // soon as the tile's scores are done, V^T after its P.V.
             auto load_k = [&](int j) {
@@ -188,7 +165,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_qhi, const __grid
                 const int s = j % G::kStages;
                 unsigned char *st = ring + (size_t)s * G::kStageBytes;
                 bar_expect(&v_full[s], G::kVBytes);
-                tma_load_2d(st + G::kKBytes, &map_vhi, j * kBKV, v_row0, &v_full[s]);
+                tma_load_2d(st + G::kKBytes, &map_vhi, v_col0 + j * kBKV, v_row0, &v_full[s]);
                 if (PAIR) tma_load_2d(st + G::kKBytes + G::kVTile, &map_vlo, j * kBKV, v_row0, &v_full[s]);
             };
             bar_expect(&q_bar, G::kQBytes);
@@ -280,9 +257,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_qhi, const __grid
         const int last_min = p.causal ? min(p.total - 1, p.past + i0) : p.total - 1;  // the smallest `last` of the CTA
         // exp(s * scale - m) = 2^(s * scale * log2(e) - m'): the maximum is kept in the base-2 domain
         const float scale2 = p.scale * 1.4426950408889634f;
+        const int first = chunk_lo(i_row), first_max = chunk_lo(i_hi);  // of this row, and the largest of the CTA
 #pragma unroll
         for (int e = 0; e < kDH; ++e) ctx[e] = 0.f;
         float m = -INFINITY;
+        if (CHUNK && p.sink) {  // a weight without a value: the running maximum starts at the sink, the row sum at its weight
+            m = p.sink[h] * 1.4426950408889634f;
+            if (half == 0) l = 1.f;
+        }
         unsigned char *prow_hi = p_s + (size_t)row * 128, *prow_lo = prow_hi + G::kPTile;
 
         // ctx = ctx * factor + O of tile j (the accumulator of odd tiles sits DV columns after that of even tiles)
@@ -309,12 +291,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_qhi, const __grid
 #pragma unroll
                 for (int c = 0; c < 32; ++c) sc[c] = __uint_as_float(v[c]);
             }
-            const int key0 = j * kBKV + 32 * half;
+            const int tile0 = (jt0 + j) * kBKV, key0 = tile0 + 32 * half;
             float mx = -INFINITY;
-            if (j * kBKV + kBKV - 1 > last_min) {  // the tile crosses the diagonal or the end of the context (same for the CTA)
+            // the tile crosses the diagonal, the end of the context or the start of a chunk (same for the CTA)
+            if (tile0 + kBKV - 1 > last_min || (CHUNK && tile0 < first_max)) {
 #pragma unroll
                 for (int c = 0; c < 32; ++c) {
-                    sc[c] = key0 + c <= last ? sc[c] * scale2 : -INFINITY;
+                    sc[c] = key0 + c <= last && (!CHUNK || key0 + c >= first) ? sc[c] * scale2 : -INFINITY;
                     mx = fmaxf(mx, sc[c]);
                 }
             } else {
@@ -328,8 +311,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_qhi, const __grid
             // one after the writes, one after the reads so that the next tile's write cannot overtake a read)
             xch[half][row] = mx;
             asm volatile("bar.sync %0, 64;" ::"r"(1 + quad) : "memory");
-            const float mt = fmaxf(m, fmaxf(mx, xch[half ^ 1][row]));
+            float mt = fmaxf(m, fmaxf(mx, xch[half ^ 1][row]));
             asm volatile("bar.sync %0, 64;" ::"r"(1 + quad) : "memory");
+            if (CHUNK && mt == -INFINITY) mt = 0.f;  // (nothing of the row's chunk so far, and no sink)
             const float r = ex2(m - mt);  // 0 for the first tile (m = -inf; row 0 of the cache is visible to every query)
             m = mt;
             float lsum = 0.f;
@@ -379,7 +363,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_qhi, const __grid
         if (warp < kFaWorkers / 32) {
             const int row = tid & (kBQ - 1), half = tid >> 7;
             if (i0 + row < p.S) {
-                const float inv = __fdiv_rn(1.0f, __fadd_rn(xch[0][row] + xch[1][row], 1e-9f));
+                const float inv = __fdiv_rn(1.0f, CHUNK ? xch[0][row] + xch[1][row] : __fadd_rn(xch[0][row] + xch[1][row], 1e-9f));
                 const size_t orow = (size_t)b * p.S + (i0 + row);
                 if constexpr (PAIR) {
                     float *o = p.out + (orow * p.Hq + h) * DV + half * kDH;
@@ -505,16 +489,16 @@ __global__ void fa_pack_latent_q_kernel(const LatentArgs a, __nv_bfloat16 *__res
     reinterpret_cast<uint4 *>(q)[i] = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
 }
 
-template <int KB, int DV, bool PAIR>
+template <int KB, int DV, bool PAIR, bool CHUNK = false>
 int launch_fa(lumen_ctx *ctx, const CUtensorMap *maps, const FaParams &p, dim3 grid, cudaStream_t s) {
     using G = FaGeom<KB, DV, PAIR>;
     static bool attr_set[64] = {false};
     const int dev = ctx->device >= 0 && ctx->device < 64 ? ctx->device : 0;
     if (!attr_set[dev]) {
-        LUMEN_CUDA(ctx, cudaFuncSetAttribute(attn_prefill_tc_kernel<KB, DV, PAIR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)G::kSmem));
+        LUMEN_CUDA(ctx, cudaFuncSetAttribute(attn_prefill_tc_kernel<KB, DV, PAIR, CHUNK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)G::kSmem));
         attr_set[dev] = true;
     }
-    attn_prefill_tc_kernel<KB, DV, PAIR><<<grid, kFaThreads, G::kSmem, s>>>(maps[0], maps[1], maps[2], maps[3], maps[4], maps[5], p);
+    attn_prefill_tc_kernel<KB, DV, PAIR, CHUNK><<<grid, kFaThreads, G::kSmem, s>>>(maps[0], maps[1], maps[2], maps[3], maps[4], maps[5], p);
     LUMEN_LAUNCHED(ctx);
     return LUMEN_OK;
 }
@@ -642,6 +626,53 @@ int launch_latent_prefill(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s) {
         const dim3 grid((unsigned)(s_pad / kBQ), (unsigned)a.H, (unsigned)a.B);
         if (KB == 2) rc = wide ? launch_fa<2, 128, false>(ctx, maps, p, grid, s) : launch_fa<2, 64, false>(ctx, maps, p, grid, s);
         else rc = wide ? launch_fa<3, 128, false>(ctx, maps, p, grid, s) : launch_fa<3, 64, false>(ctx, maps, p, grid, s);
+    }
+    const int rc2 = dev_free(ctx, ws);
+    return rc != LUMEN_OK ? rc : rc2;
+}
+
+// Portions of at least 64 positions whose heads have at most 192 (keys) and 128 (values) numbers.
+bool grouped_prefill_usable(const GroupedArgs &a) {
+    static const bool off = [] {
+        const char *e = getenv("LUMEN_NO_TC_ATTN");
+        return e && e[0] == '1';
+    }();
+    if (off || a.dt != LUMEN_BF16 || a.S < 64 || a.dim > 192 || a.vdim > 128 || a.dim % 8) return false;
+    const size_t s_pad = (a.S + kBQ - 1) / kBQ * kBQ;
+    return a.B * a.H * s_pad < ((size_t)1 << 31) && a.B * a.G * a.max_seq < ((size_t)1 << 31) && a.B * a.G * a.vdim < ((size_t)1 << 31) &&
+           a.B * a.G <= 65535 && a.B <= 65535 && a.H <= 65535;
+}
+
+// Keys are read where the cache has them; the visible values are transposed into V^T.
+int launch_grouped_prefill(lumen_ctx *ctx, const GroupedArgs &a, cudaStream_t s) {
+    const size_t total = a.past + a.S, s_pad = (a.S + kBQ - 1) / kBQ * kBQ;
+    const size_t v0 = (a.chunk ? a.past / a.chunk * a.chunk : 0) / kBKV * kBKV, rows = total - v0, lp = (rows + 7) / 8 * 8;
+    const int KB = (int)((a.dim + kBK - 1) / kBK), width = KB * kBK;
+    const size_t nq = a.B * a.H * s_pad * width, nv = a.B * a.G * a.vdim * lp;
+    void *ws = nullptr;
+    LUMEN_TRY(dev_alloc(ctx, (nq + nv) * sizeof(__nv_bfloat16), &ws));
+    __nv_bfloat16 *q = static_cast<__nv_bfloat16 *>(ws), *vt = q + nq;
+    int rc = launch_grouped_append(ctx, a, q, s_pad, width, s);
+    if (rc == LUMEN_OK) rc = launch_transpose_rows(ctx, static_cast<const __nv_bfloat16 *>(a.v), a.max_seq, a.vdim, a.B * a.G, v0, rows, vt, lp, s);
+    const bool wide = a.vdim > 64;
+    CUtensorMap maps[6];
+    if (rc == LUMEN_OK) rc = make_map(ctx, &maps[0], q, a.B * a.H * s_pad, width, kBQ);
+    if (rc == LUMEN_OK) rc = make_map(ctx, &maps[2], a.k, a.B * a.G * a.max_seq, a.dim, kBKV);
+    if (rc == LUMEN_OK) rc = make_map(ctx, &maps[4], vt, a.B * a.G * a.vdim, rows, wide ? 128 : 64, lp);
+    if (rc == LUMEN_OK) {
+        maps[1] = maps[0];
+        maps[3] = maps[2];
+        maps[5] = maps[4];
+        FaParams p{};
+        p.out = a.out; p.out_hi = a.out_hi; p.out_lo = a.out_lo;
+        p.S = (int)a.S; p.Hq = (int)a.H; p.Hkv = (int)a.G; p.past = (int)a.past; p.total = (int)total; p.causal = 1; p.s_pad = (int)s_pad;
+        p.k_rows_b = (int)(a.G * a.max_seq); p.k_rows_h = (int)a.max_seq; p.kb_main = KB;
+        p.vdim = (int)a.vdim; p.gate = a.u + a.u_gate; p.gate_ld = a.u_ld; p.scale = a.scale;
+        p.chunk = (int)std::min<size_t>(a.chunk, 0x7fffffff); p.v0 = (int)v0; p.sink = a.sink; p.status = ctx->d_status;
+        const dim3 grid((unsigned)(s_pad / kBQ), (unsigned)a.H, (unsigned)a.B);
+        if (KB == 1) rc = wide ? launch_fa<1, 128, false, true>(ctx, maps, p, grid, s) : launch_fa<1, 64, false, true>(ctx, maps, p, grid, s);
+        else if (KB == 2) rc = wide ? launch_fa<2, 128, false, true>(ctx, maps, p, grid, s) : launch_fa<2, 64, false, true>(ctx, maps, p, grid, s);
+        else rc = wide ? launch_fa<3, 128, false, true>(ctx, maps, p, grid, s) : launch_fa<3, 64, false, true>(ctx, maps, p, grid, s);
     }
     const int rc2 = dev_free(ctx, ws);
     return rc != LUMEN_OK ? rc : rc2;

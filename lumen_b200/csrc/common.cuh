@@ -99,8 +99,11 @@ struct lumen_kv_cache {
     int *d_len = nullptr;  // device copy read by replayable kernels
     float *k = nullptr;    // [B,Hkv,max_seq,D]
     float *v = nullptr;
-    // Latent caches (models given as a list of layers): rows of d numbers of type dtype in k, no v.  The slab also holds the
-    // last token id of every batch row, shared by the layers.
+    // Models given as a list of layers.  kLatent: rows of d numbers of type dtype in k, no v.  kRows: keys [B,Hkv,max_seq,d] and values
+    // [B,Hkv,max_seq,dv] of type dtype.  kState: f32 matrices [B,H,d,dv] in k, vectors [B,H,d] and then numbers [B,H] in v; h_kv = H.
+    // The slab also holds the last token id of every batch row, shared by the layers.
+    enum Kind { kLlama, kLatent, kRows, kState } kind = kLlama;
+    size_t dv = 0;
     lumen_dtype dtype = LUMEN_F32;
     int *last_tok = nullptr;
     unsigned int seen_abort = 0;  // ctx->abort_gen at the last time `len` was known to equal *d_len
@@ -151,6 +154,23 @@ int launch_pdl(lumen_ctx *ctx, void (*kernel)(KA...), dim3 grid, dim3 block, siz
     attr.val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = &attr;
     cfg.numAttrs = ctx->pdl && pdl_enabled() ? 1 : 0;
+    LUMEN_CUDA(ctx, cudaLaunchKernelEx(&cfg, kernel, args...));
+    ctx->launches += 1;
+    return LUMEN_OK;
+}
+
+// The same for a kernel of thread-block clusters of (cluster, 1, 1).
+template <typename... KA, typename... A>
+int launch_pdl_cluster(lumen_ctx *ctx, void (*kernel)(KA...), unsigned cluster, dim3 grid, dim3 block, size_t smem, cudaStream_t s, A... args) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid; cfg.blockDim = block; cfg.dynamicSmemBytes = smem; cfg.stream = s;
+    cudaLaunchAttribute attr[2] = {};
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = cluster; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = ctx->pdl && pdl_enabled() ? 2 : 1;
     LUMEN_CUDA(ctx, cudaLaunchKernelEx(&cfg, kernel, args...));
     ctx->launches += 1;
     return LUMEN_OK;

@@ -1,4 +1,5 @@
-// Token inputs of the models given as a list of layers: embedding plus hashed bigram embedding, and the end of a step.
+// Token inputs of the models given as a list of layers: embedding (scaled, plus a hashed bigram embedding) with the norm that the
+// first layer reads, and the end of a step.
 #include "decoder_kernels.cuh"
 
 namespace lumen {
@@ -25,12 +26,32 @@ __global__ void __launch_bounds__(256) embed_kernel(EmbedArgs a, DeviceStatus *s
         else if (*a.d_len > 0) r = ((unsigned long long)a.last_tok[b] * a.mul_prev + tok * a.mul_cur) % a.buckets;
         brow = static_cast<const T *>(a.bigram) + r * a.dim;
     }
+    auto put = [&](float v, size_t at) {
+        if (a.out) a.out[at] = v;
+        if (a.hi) store_split(v, a.hi, a.lo, at);
+    };
+    float ss = 0.f;
     for (size_t i = threadIdx.x; i < a.dim; i += 256) {
-        float v = to_f32(row[i]);
+        float v = __fmul_rn(to_f32(row[i]), a.scale);
         if (brow) v = __fadd_rn(v, to_f32(brow[i]));
         const size_t at = m * a.dim + i;
         a.x[at] = v;
-        if (a.hi) store_split(v, a.hi, a.lo, at);
+        if (a.norm_w) ss = fmaf(v, v, ss);
+        else put(v, at);
+    }
+    if (!a.norm_w) return;
+    __shared__ float red[8];
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) ss += red[w];
+    const float inv = __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)a.dim), a.eps)));
+    for (size_t i = threadIdx.x; i < a.dim; i += 256) {  // (every thread reads back what it wrote)
+        const size_t at = m * a.dim + i;
+        put(__fmul_rn(__fmul_rn(a.x[at], inv), a.norm_w[i]), at);
     }
 }
 

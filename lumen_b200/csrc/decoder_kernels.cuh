@@ -1,5 +1,6 @@
-// Kernel launchers of the models given as a list of layers (api_decoder.cu): latent attention, routed experts, outputs
-// normed before they are added to the residual, bigram and per-layer token inputs.  Constants are parameters.
+// Kernel launchers of the models given as a list of layers (api_decoder.cu): latent attention, grouped-query attention over
+// chunks, matrix-memory layers, routed experts, outputs normed before they are added to the residual, bigram and per-layer
+// token inputs.  Constants are parameters.
 #pragma once
 
 #include "common.cuh"
@@ -7,7 +8,7 @@
 namespace lumen {
 
 // ---- embedding (decoder_embed.cu) -----------------------------------------------------------------
-// x[m] = embed[id] (+ bigram[row]), row = (previous id * mul_prev + id * mul_cur) mod buckets, `buckets` for the first
+// x[m] = embed[id] * scale (+ bigram[row]), row = (previous id * mul_prev + id * mul_cur) mod buckets, `buckets` for the first
 // token of a sequence.  Row m = b * S + s; the token before s == 0 is last_tok[b], absent when *d_len == 0.
 struct EmbedArgs {
     const float *ids = nullptr;  // [B * S]
@@ -15,8 +16,13 @@ struct EmbedArgs {
     lumen_dtype dt = LUMEN_F32;
     size_t B = 1, S = 1, vocab = 0, dim = 0, buckets = 0, mul_prev = 0, mul_cur = 0;
     const int *d_len = nullptr, *last_tok = nullptr;
+    float scale = 1.f;
     float *x = nullptr;
-    __nv_bfloat16 *hi = nullptr, *lo = nullptr;  // bf16 split of x (null: not stored)
+    // With norm_w the first layer reads RMSNorm(x) * norm_w; what it reads as f32 and/or as a bf16 split (null: not stored)
+    const float *norm_w = nullptr;
+    float eps = 0.f;
+    float *out = nullptr;
+    __nv_bfloat16 *hi = nullptr, *lo = nullptr;
 };
 int launch_embed(lumen_ctx *ctx, const EmbedArgs &a, cudaStream_t s);
 // End of a step: every layer's cache grows by S rows and last_tok[b] becomes the id of the sequence's last token.
@@ -27,13 +33,13 @@ int launch_advance(lumen_ctx *ctx, int *d_lens, size_t layers, const float *ids,
 struct StepFinish {
     enum Kind {
         kStore,     // out = sum
-        kNormAdd,   // x += RMSNorm(sum + gathered rows) * gain; (hi, lo) = split(x)
+        kNormAdd,   // x += RMSNorm(sum + gathered rows) * gain; then of x, or of RMSNorm(x) * next_gain: out, (hi, lo) = split
         kGelu,      // out = gelu_tanh(sum)
         kSideGate,  // out = gelu_tanh(sum) * table[id, col]
-        kGated,     // sum holds gate and up in blocks of 64 columns: out = clamped SwiGLU (see gated_act)
+        kGated,     // sum holds gate and up in blocks of 64 columns: out = glu(gate, up)
     } kind = kStore;
     float *x = nullptr;
-    const float *gain = nullptr;
+    const float *gain = nullptr, *next_gain = nullptr;
     float eps = 0.f;
     const __nv_bfloat16 *gather_src = nullptr;  // rows gather_idx[row, 0 .. gather_n) of this matrix are added too
     const int *gather_idx = nullptr;
@@ -42,7 +48,8 @@ struct StepFinish {
     const void *table = nullptr;
     lumen_dtype table_dt = LUMEN_F32;
     size_t table_ld = 0, table_rows = 0;
-    float limit = 0.f;                  // kGated
+    enum Glu { kClampedSwish, kGeluTanh } glu = kClampedSwish;  // kGated: see gated_act / gelu_tanh(gate) * up
+    float limit = 0.f;
     size_t ff = 0;
     float *out = nullptr;
     __nv_bfloat16 *hi = nullptr, *lo = nullptr;
@@ -61,8 +68,8 @@ struct GemmBf16Args {
     const StepFinish *fin = nullptr;
     __nv_bfloat16 *out16 = nullptr;    // instead of c: bf16 result of the epilogue
     size_t ld16 = 0;
-    enum Epi { kF32 = 0, kBf16 = 1, kGelu = 2, kGated = 3 } epi = kF32;
-    float limit = 0.f;                 // kGated: N = 2 * 64 * ceil(ff / 64) interleaved rows, ff columns stored
+    enum Epi { kF32 = 0, kBf16 = 1, kGelu = 2, kGated = 3, kGatedGelu = 4 } epi = kF32;
+    float limit = 0.f;                 // kGated, kGatedGelu: N = 2 * 64 * ceil(ff / 64) interleaved rows, ff columns stored
     size_t ff = 0;
     // Grouped: tile t covers rows tiles[t].x .. tiles[t].y - 1 of A against the N rows of W from tiles[t].z * N;
     // tiles beyond *n_tiles are empty.  row_scale multiplies a row's sums before the activation.
@@ -88,7 +95,7 @@ struct GemvStepArgs {
     lumen_dtype wdt = LUMEN_F32;
     size_t K = 0, N = 0;
     float *out = nullptr;
-    StepFinish::Kind act = StepFinish::kStore;  // kStore, kGelu or kSideGate
+    StepFinish::Kind act = StepFinish::kStore;  // kStore, kGelu, kSideGate, or kGated (gelu_tanh(gate) * up; N = ff)
     const float *ids = nullptr;
     const void *table = nullptr;
     size_t table_ld = 0, table_rows = 0;
@@ -168,6 +175,68 @@ int launch_latent_value(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s);
 // Whole portions on the tensor cores over expanded keys and values (bf16); the cache already holds the rows.
 bool latent_prefill_usable(const LatentArgs &a);
 int launch_latent_prefill(lumen_ctx *ctx, const LatentArgs &a, cudaStream_t s);
+
+// ---- matrix-memory layers (mlstm.cu, mlstm_chunk_tc.cu) ---------------------------------------------
+// Per head: S <- exp(f + m - m') S + exp(i - m') k v^T, n likewise with k alone, m' = max(f + m, i);
+// o = S^T q / (max(|n . q|, exp(-m')) + 1e-6), RMS-normed per head, times head_gain and sigmoid(g).
+struct MlstmArgs {
+    size_t B = 0, S = 0, H = 0, dim = 0, vdim = 0;
+    float cap = 0.f, eps = 0.f;
+    // Projections of row m: f32 at u + m * u_ld (queries at 0, keys at u_k, values at u_v, output gates at u_g), or bf16 at u16
+    // with the same offsets (chunked form).
+    const float *u = nullptr;
+    const __nv_bfloat16 *u16 = nullptr;
+    size_t u_ld = 0, u_k = 0, u_v = 0, u_g = 0;
+    const float *z = nullptr, *z_bias = nullptr;  // gate pre-activations z[m * z_ld + h] (input) and [.. + H + h] (forget), biases [2 H]
+    size_t z_ld = 0;
+    const float *head_gain = nullptr;             // [H * vdim]
+    float *state = nullptr, *norm = nullptr, *mx = nullptr;  // [B, H, dim, vdim], [B, H, dim], [B, H]; absent while *d_len == 0
+    const int *d_len = nullptr;
+    size_t past = 0;                              // the host's view of *d_len
+    float *out = nullptr;                         // [B * S, H * vdim] (null: not stored)
+    __nv_bfloat16 *out_hi = nullptr, *out_lo = nullptr;
+};
+// Token by token, any sizes.
+int launch_mlstm_step(lumen_ctx *ctx, const MlstmArgs &a, cudaStream_t s);
+// Portions in chunks of kMlstmChunk tokens on the tensor cores (bf16 projections).
+constexpr int kMlstmChunk = 128;
+bool mlstm_chunked_usable(const MlstmArgs &a);
+int launch_mlstm_chunked(lumen_ctx *ctx, const MlstmArgs &a, cudaStream_t s);
+
+// ---- grouped-query attention over chunks (grouped_attention.cu, attn_prefill_tc.cu) ----------------
+// u[M, u_ld] holds per row the queries (H x dim), and for layers with keys and values of their own the keys (G x dim) at u_k
+// and values (G x vdim) at u_v, and the heads' gate logits at u_gate.  T = element type of the cache: f32, or bf16 in bf16 models.
+struct GroupedArgs {
+    size_t B = 0, S = 0, H = 0, G = 0, dim = 0, vdim = 0, rot_dims = 0, chunk = 0, max_seq = 0;
+    lumen_dtype dt = LUMEN_F32;
+    const float *u = nullptr;
+    size_t u_ld = 0, u_k = 0, u_v = 0, u_gate = 0;
+    bool own_kv = true;
+    const float *q_gain = nullptr, *k_gain = nullptr, *sink = nullptr;  // [dim], [dim], [H]
+    float eps = 0.f, scale = 0.f;
+    const float *cos_t = nullptr, *sin_t = nullptr;                     // [max_seq, rot_dims / 2]
+    void *k = nullptr, *v = nullptr;                                    // [B, G, max_seq, dim], [B, G, max_seq, vdim]
+    const int *d_len = nullptr;
+    size_t past = 0;
+    float *part_ctx = nullptr, *part_ml = nullptr;  // [rows * H, nsplit, vdim], [rows * H, nsplit, 2]
+    int nsplit = 1;
+    float *out = nullptr;                           // [M, H * vdim] (null: not stored)
+    __nv_bfloat16 *out_hi = nullptr, *out_lo = nullptr;
+};
+constexpr size_t kGroupedMaxDim = 512;
+int grouped_pick_splits(const GroupedArgs &a, int num_sms);
+// Keys (normed, rotated) and values -> cache, for layers with keys and values of their own; with q also the queries
+// (normed, rotated) as bf16 [B, H, s_pad, width].
+int launch_grouped_append(lumen_ctx *ctx, const GroupedArgs &a, __nv_bfloat16 *q, size_t s_pad, size_t width, cudaStream_t s);
+// Attention of every row over the cached rows in nsplit pieces, merged with the sink and the gate.  append: the one new row of
+// every sequence (S == 1) is appended by the same launch.
+int launch_grouped_attention(lumen_ctx *ctx, const GroupedArgs &a, bool append, cudaStream_t s);
+// Whole portions on the tensor cores (bf16), append included.
+bool grouped_prefill_usable(const GroupedArgs &a);
+int launch_grouped_prefill(lumen_ctx *ctx, const GroupedArgs &a, cudaStream_t s);
+// out[(b * heads + h) * cols + c][j] = in[b][h][row0 + j][c], j < rows (zeros up to the pitch): rows of a cache as columns.
+int launch_transpose_rows(lumen_ctx *ctx, const __nv_bfloat16 *in, size_t in_rows, size_t cols, size_t mats, size_t row0, size_t rows,
+                          __nv_bfloat16 *out, size_t pitch, cudaStream_t s);
 
 // ---- shared device helpers ----------------------------------------------------------------------
 #ifdef __CUDACC__

@@ -54,7 +54,9 @@ __global__ void __launch_bounds__(256) sum_swiglu_split_kernel(const float *__re
     *reinterpret_cast<uint2 *>(lo + row * inter + col) = l;
 }
 
-// One CTA per row, any row length (the row is kept in shared memory between the two passes).
+// One CTA per row, any row length (the row is kept in shared memory between the passes).  NEXT: the next sublayer reads a norm of
+// the new residual.
+template <bool NEXT>
 __global__ void __launch_bounds__(256) norm_add_kernel(const float *__restrict__ part, int splits, size_t rows, size_t n, const StepFinish f) {
     extern __shared__ __align__(16) float row_s[];
     __shared__ float red[8];
@@ -85,14 +87,28 @@ __global__ void __launch_bounds__(256) norm_add_kernel(const float *__restrict__
             ss = fmaf(v, v, ss);
         }
     }
+    auto row_inv = [&](float s) {
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    if ((tid & 31) == 0) red[tid >> 5] = ss;
-    __syncthreads();
-    float t = 0.f;
+        for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+        if ((tid & 31) == 0) red[tid >> 5] = s;
+        __syncthreads();
+        float t = 0.f;
 #pragma unroll
-    for (int w = 0; w < 8; ++w) t += red[w];
-    const float inv = __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(t, (float)n), f.eps)));
+        for (int w = 0; w < 8; ++w) t += red[w];
+        __syncthreads();
+        return __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(t, (float)n), f.eps)));
+    };
+    const float inv = row_inv(ss);
+    auto put4 = [&](float4 v, size_t i) {
+        if (f.out) reinterpret_cast<float4 *>(f.out + base)[i] = v;
+        if (f.hi) {
+            uint2 h, l;
+            split4(v, &h, &l);
+            reinterpret_cast<uint2 *>(f.hi + base)[i] = h;
+            if (f.lo) reinterpret_cast<uint2 *>(f.lo + base)[i] = l;
+        }
+    };
+    float ss2 = 0.f;
     if (vec) {
         for (size_t i = tid; i < n / 4; i += 256) {
             const float4 v = reinterpret_cast<const float4 *>(row_s)[i], g = reinterpret_cast<const float4 *>(f.gain)[i];
@@ -100,19 +116,40 @@ __global__ void __launch_bounds__(256) norm_add_kernel(const float *__restrict__
             const float4 x = add4(*xp, make_float4(__fmul_rn(__fmul_rn(v.x, inv), g.x), __fmul_rn(__fmul_rn(v.y, inv), g.y),
                                                    __fmul_rn(__fmul_rn(v.z, inv), g.z), __fmul_rn(__fmul_rn(v.w, inv), g.w)));
             *xp = x;
-            if (f.hi) {
-                uint2 h, l;
-                split4(x, &h, &l);
-                reinterpret_cast<uint2 *>(f.hi + base)[i] = h;
-                if (f.lo) reinterpret_cast<uint2 *>(f.lo + base)[i] = l;
+            if (NEXT) {
+                reinterpret_cast<float4 *>(row_s)[i] = x;
+                ss2 = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, fmaf(x.w, x.w, ss2))));
+            } else {
+                put4(x, i);
+            }
+        }
+        if (NEXT) {
+            const float inv2 = row_inv(ss2);
+            for (size_t i = tid; i < n / 4; i += 256) {
+                const float4 x = reinterpret_cast<const float4 *>(row_s)[i], g = reinterpret_cast<const float4 *>(f.next_gain)[i];
+                put4(make_float4(__fmul_rn(__fmul_rn(x.x, inv2), g.x), __fmul_rn(__fmul_rn(x.y, inv2), g.y), __fmul_rn(__fmul_rn(x.z, inv2), g.z),
+                                 __fmul_rn(__fmul_rn(x.w, inv2), g.w)), i);
             }
         }
         return;
     }
+    auto put = [&](float v, size_t i) {
+        if (f.out) f.out[base + i] = v;
+        if (f.hi) store_split(v, f.hi, f.lo, base + i);
+    };
     for (size_t i = tid; i < n; i += 256) {
         const float x = __fadd_rn(f.x[base + i], __fmul_rn(__fmul_rn(row_s[i], inv), f.gain[i]));
         f.x[base + i] = x;
-        if (f.hi) store_split(x, f.hi, f.lo, base + i);
+        if (NEXT) {
+            row_s[i] = x;
+            ss2 = fmaf(x, x, ss2);
+        } else {
+            put(x, i);
+        }
+    }
+    if (NEXT) {
+        const float inv2 = row_inv(ss2);
+        for (size_t i = tid; i < n; i += 256) put(__fmul_rn(__fmul_rn(row_s[i], inv2), f.next_gain[i]), i);
     }
 }
 
@@ -130,7 +167,8 @@ __global__ void __launch_bounds__(256) act_finish_kernel(const float *__restrict
     float v;
     if (f.kind == StepFinish::kGated) {
         const size_t at = col / kGateBlock * (2 * kGateBlock) + col % kGateBlock;
-        v = gated_act(sum(at), sum(at + kGateBlock), f.limit);
+        const float g = sum(at), u = sum(at + kGateBlock);
+        v = f.glu == StepFinish::kGeluTanh ? gelu_tanh(g) * u : gated_act(g, u, f.limit);
     } else {
         v = sum(col);
         if (f.kind != StepFinish::kStore) v = gelu_tanh(v);
@@ -150,8 +188,9 @@ int launch_step_finish(lumen_ctx *ctx, const float *part, int splits, size_t row
     if (f.kind == StepFinish::kNormAdd) {
         const size_t smem = n * sizeof(float);
         if (smem > 200 * 1024) return set_error(ctx, LUMEN_ERR_UNSUPPORTED, "row finisher: row length %zu", n);
-        if (smem > 48 * 1024) LUMEN_CUDA(ctx, cudaFuncSetAttribute(norm_add_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-        norm_add_kernel<<<(unsigned)rows, 256, smem, s>>>(part, part ? splits : 0, rows, n, f);
+        const auto kernel = f.next_gain ? norm_add_kernel<true> : norm_add_kernel<false>;
+        if (smem > 48 * 1024) LUMEN_CUDA(ctx, cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        kernel<<<(unsigned)rows, 256, smem, s>>>(part, part ? splits : 0, rows, n, f);
     } else {
         const size_t total = rows * (f.kind == StepFinish::kGated ? f.ff : n);
         act_finish_kernel<<<(unsigned)((total + 255) / 256), 256, 0, s>>>(part, splits, rows, n, f);

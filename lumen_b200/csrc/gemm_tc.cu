@@ -175,7 +175,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid_constan
     if (have && !failed) {
         const int arow = a0 + warp * 32 + lane;  // this thread's row of the tile's 128-row side
         const bool empty_slice = nkb == 0;       // nothing was accumulated: the tile's contribution is zero
-        if constexpr (EPI == GemmBf16Args::kGated) {
+        if constexpr (EPI == GemmBf16Args::kGated || EPI == GemmBf16Args::kGatedGelu) {
             // in every 128 columns of the tile 64 are gates, and 64 the ups that go with them: 64 columns of output
             const float scale = p.row_scale && arow < a_end ? p.row_scale[arow] : 1.f;
             const bool vec = (p.ld16 & 7) == 0;
@@ -193,7 +193,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_ahi, const __grid_constan
                     for (int j = 0; j < 32; j += 8) {
                         float x[8];
 #pragma unroll
-                        for (int i = 0; i < 8; ++i) x[i] = gated_act(__uint_as_float(g[j + i]) * scale, __uint_as_float(u[j + i]) * scale, p.limit);
+                        for (int i = 0; i < 8; ++i) {
+                            const float gv = __uint_as_float(g[j + i]) * scale, uv = __uint_as_float(u[j + i]) * scale;
+                            x[i] = EPI == GemmBf16Args::kGatedGelu ? gelu_tanh(gv) * uv : gated_act(gv, uv, p.limit);
+                        }
                         if (col + j < p.ff) store8_bf16(dst + j, x, p.ff - (col + j), vec);
                     }
                 }
@@ -471,16 +474,17 @@ int launch_gemm_bf16(lumen_ctx *ctx, const GemmBf16Args &g, cudaStream_t s) {
     p.ff = (int)g.ff;
     const int kb_all = (int)((g.K + kBK - 1) / kBK);
     p.kb_per_split = kb_all;
+    const bool gated = g.epi == GemmBf16Args::kGated || g.epi == GemmBf16Args::kGatedGelu;
     const bool swap = g.M <= 64 && g.epi == GemmBf16Args::kF32 && !grouped;
     // 256-wide tiles read each activation tile half as often and keep the tensor pipe busier, unless they leave the last wave
     // of CTAs emptier than that is worth (a 256-wide tile takes about 1.5 times as long as a 128-wide one)
     const size_t row_tiles = grouped ? g.max_tiles : (g.M + kBM - 1) / kBM;
     auto waves = [&](size_t width) { return (row_tiles * ((g.N + width - 1) / width) + ctx->num_sms - 1) / ctx->num_sms; };
     const bool wide = !swap && !pair && g.M > (size_t)kBM && g.N > 128 && 3 * waves(256) <= 2 * waves(128);
-    const int bn = swap ? 64 : wide ? 256 : g.epi == GemmBf16Args::kGated || grouped ? 128 : pick_bn(g.M, g.N, ctx->num_sms);
+    const int bn = swap ? 64 : wide ? 256 : gated || grouped ? 128 : pick_bn(g.M, g.N, ctx->num_sms);
     int splits = 1;
     void *partial = nullptr;
-    if (g.epi == GemmBf16Args::kF32 && !grouped && g.M <= (size_t)kBM) {
+    if (g.epi == GemmBf16Args::kF32 && !grouped && (g.M <= (size_t)kBM || (g.N <= 64 && g.M <= 16 * (size_t)kBM))) {
         const int tiles = (int)((g.N + (swap ? kBM : bn) - 1) / (swap ? kBM : bn));
         splits = std::max(1, std::min(std::min(ctx->num_sms / std::max(tiles, 1), kb_all / 4), 16));
         p.kb_per_split = (kb_all + splits - 1) / splits;
@@ -509,11 +513,13 @@ int launch_gemm_bf16(lumen_ctx *ctx, const GemmBf16Args &g, cudaStream_t s) {
         if (grouped && wide) rc = g.epi == GemmBf16Args::kGated ? LUMEN_TC(1, 1, 256, false, 3, true) : LUMEN_TC(1, 1, 256, false, 1, true);
         else if (grouped) rc = g.epi == GemmBf16Args::kGated ? LUMEN_TC(1, 1, 128, false, 3, true) : LUMEN_TC(1, 1, 128, false, 1, true);
         else if (wide) rc = g.epi == GemmBf16Args::kGated  ? LUMEN_TC(1, 1, 256, false, 3, false)
+                            : g.epi == GemmBf16Args::kGatedGelu ? LUMEN_TC(1, 1, 256, false, 4, false)
                             : g.epi == GemmBf16Args::kGelu ? LUMEN_TC(1, 1, 256, false, 2, false)
                             : g.epi == GemmBf16Args::kBf16 ? LUMEN_TC(1, 1, 256, false, 1, false)
                                                            : LUMEN_TC(1, 1, 256, false, 0, false);
         else if (swap) rc = pair ? LUMEN_TC(1, 2, 64, true, 0, false) : LUMEN_TC(1, 1, 64, true, 0, false);
         else if (g.epi == GemmBf16Args::kGated) rc = LUMEN_TC(1, 1, 128, false, 3, false);
+        else if (gated) rc = LUMEN_TC(1, 1, 128, false, 4, false);
         else if (g.epi == GemmBf16Args::kGelu) rc = bn == 128 ? LUMEN_TC(1, 1, 128, false, 2, false) : bn == 64 ? LUMEN_TC(1, 1, 64, false, 2, false) : LUMEN_TC(1, 1, 32, false, 2, false);
         else if (g.epi == GemmBf16Args::kBf16) rc = bn == 128 ? LUMEN_TC(1, 1, 128, false, 1, false) : bn == 64 ? LUMEN_TC(1, 1, 64, false, 1, false) : LUMEN_TC(1, 1, 32, false, 1, false);
         else if (pair) rc = bn == 128 ? LUMEN_TC(2, 1, 128, false, 0, false) : bn == 64 ? LUMEN_TC(2, 1, 64, false, 0, false) : LUMEN_TC(2, 1, 32, false, 0, false);

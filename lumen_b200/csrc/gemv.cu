@@ -171,7 +171,8 @@ gemv_gate_up_kernel(const float *__restrict__ x, const WT *__restrict__ wg, cons
 // One row whose input may still owe the norm of a sublayer's output (post-norm models): x = res + RMSNorm(y) * gain is
 // formed by every CTA while it stages x, so that the norm, the residual sum and the product are one launch.  WPR warps share a
 // weight row (a slice of K each) where there are too few rows to keep enough loads in flight.
-template <typename WT, int WPR>
+// GATED: N gate rows and the N up rows that go with them (in blocks, see kGateBlock) are walked as pairs; out = gelu_tanh(gate) * up.
+template <typename WT, int WPR, bool GATED>
 __global__ void __launch_bounds__(kThreads, 4) gemv_step_kernel(const GemvStepArgs a) {
     extern __shared__ __align__(16) float smem[];
     __shared__ float red[kWarps];
@@ -179,13 +180,19 @@ __global__ void __launch_bounds__(kThreads, 4) gemv_step_kernel(const GemvStepAr
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     constexpr int VEC = 16 / sizeof(WT), kRows = kWarps / WPR;
     const int part = warp % WPR;
-    const size_t K = a.K, row0 = (size_t)blockIdx.x * kRows + warp / WPR;
+    const size_t K = a.K, n_rows = GATED ? 2 * a.N : a.N, row0 = (size_t)blockIdx.x * kRows + warp / WPR;
     const WT *w = static_cast<const WT *>(a.w);
+    // where row r of the walk is stored (GATED: r = 2 * i for gate row i, 2 * i + 1 for up row i)
+    auto stored = [&](size_t r) {
+        if (!GATED) return r;
+        const size_t i = r >> 1;
+        return i / kGateBlock * (2 * kGateBlock) + i % kGateBlock + (r & 1) * kGateBlock;
+    };
     const bool vec_ok = (K % VEC == 0) && ((reinterpret_cast<uintptr_t>(w) & 15) == 0);
     // this warp's slice of K, in whole vectors
     const int nv = (int)(K / VEC), per = (nv + WPR - 1) / WPR, v0 = min(nv, part * per), vn = min(nv - v0, per);
     uint4 pre[kAhead];
-    if (vec_ok && row0 < a.N) row_ahead(reinterpret_cast<const uint4 *>(w + row0 * K) + v0, vn, lane, pre);
+    if (vec_ok && row0 < n_rows) row_ahead(reinterpret_cast<const uint4 *>(w + stored(row0) * K) + v0, vn, lane, pre);
     pdl_launch();
     pdl_wait();
     auto inv_rms = [&](float ss) {
@@ -258,27 +265,59 @@ __global__ void __launch_bounds__(kThreads, 4) gemv_step_kernel(const GemvStepAr
     if (a.norm_w) {
         __syncthreads();
         float ss = 0.f;
+        if (k_n % 4 == 0) {
+            float4 *x4 = reinterpret_cast<float4 *>(xs);
+            const float4 *g4 = reinterpret_cast<const float4 *>(a.norm_w);
+#pragma unroll 2
+            for (int k = tid; k < k_n / 4; k += kThreads) {
+                const float4 v = x4[k];
+                ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+            }
+            const float inv = inv_rms(ss);
+#pragma unroll 2
+            for (int k = tid; k < k_n / 4; k += kThreads) {
+                const float4 v = x4[k], g = g4[k];
+                x4[k] = make_float4(__fmul_rn(__fmul_rn(v.x, inv), g.x), __fmul_rn(__fmul_rn(v.y, inv), g.y), __fmul_rn(__fmul_rn(v.z, inv), g.z),
+                                    __fmul_rn(__fmul_rn(v.w, inv), g.w));
+            }
+        } else {
 #pragma unroll 1
-        for (int k = tid; k < k_n; k += kThreads) ss = fmaf(xs[k], xs[k], ss);
-        const float inv = inv_rms(ss);
+            for (int k = tid; k < k_n; k += kThreads) ss = fmaf(xs[k], xs[k], ss);
+            const float inv = inv_rms(ss);
 #pragma unroll 1
-        for (int k = tid; k < k_n; k += kThreads) xs[k] = __fmul_rn(__fmul_rn(xs[k], inv), a.norm_w[k]);
+            for (int k = tid; k < k_n; k += kThreads) xs[k] = __fmul_rn(__fmul_rn(xs[k], inv), a.norm_w[k]);
+        }
     }
     __syncthreads();
 #pragma unroll 1
-    for (size_t base = (size_t)blockIdx.x * kRows; base < a.N; base += (size_t)gridDim.x * kRows) {
+    for (size_t base = (size_t)blockIdx.x * kRows; base < n_rows; base += (size_t)gridDim.x * kRows) {
         const size_t row = base + warp / WPR;
         float v = 0.f;
-        if (row < a.N) {
+        if (row < n_rows) {
             if (vec_ok) {
-                const uint4 *wrow = reinterpret_cast<const uint4 *>(w + row * K) + v0;
+                const uint4 *wrow = reinterpret_cast<const uint4 *>(w + stored(row) * K) + v0;
                 if (row != row0) batch_load(wrow, 0, vn, lane, pre);
                 v = row_dot_ahead<WT>(wrow, xs + v0 * VEC, vn, lane, pre);
             } else if (part == 0) {
-                v = row_dot_scalar<WT>(w + row * K, xs, (int)K, lane);
+                v = row_dot_scalar<WT>(w + stored(row) * K, xs, (int)K, lane);
             }
         }
         v = warp_sum(v);
+        if (GATED) {  // slices and the two rows of a pair meet in the pair's first warp (kRows is even, so a pair shares a CTA)
+            if (lane == 0) red[warp] = v;
+            __syncthreads();
+            if (lane == 0 && part == 0 && (row & 1) == 0 && row < n_rows) {
+                float g = 0.f, u = 0.f;
+#pragma unroll
+                for (int i = 0; i < WPR; ++i) {
+                    g += red[warp + i];
+                    u += red[warp + WPR + i];
+                }
+                a.out[row >> 1] = gelu_tanh(g) * u;
+            }
+            __syncthreads();
+            continue;
+        }
         if (WPR > 1) {  // the row's slices meet in its first warp
             if (lane == 0) red[warp] = v;
             __syncthreads();
@@ -287,7 +326,7 @@ __global__ void __launch_bounds__(kThreads, 4) gemv_step_kernel(const GemvStepAr
             for (int i = 0; i < WPR; ++i) v += red[(warp / WPR) * WPR + i];
             __syncthreads();
         }
-        if (lane == 0 && part == 0 && row < a.N) {
+        if (lane == 0 && part == 0 && row < n_rows) {
             if (a.act != StepFinish::kStore) v = gelu_tanh(v);
             if (a.act == StepFinish::kSideGate) {
                 const unsigned long long tok = id_to_index(a.ids[0]);
@@ -472,12 +511,19 @@ int launch_gemv_step(lumen_ctx *ctx, const GemvStepArgs &a, cudaStream_t s) {
     if (smem > 200 * 1024) return set_error(ctx, LUMEN_ERR_UNSUPPORTED, "gemv_step: row of %zu elements", a.K);
     // warps per row: enough warps for about three CTAs per SM, a slice of at least 1 KB each
     const size_t row_bytes = a.K * (a.wdt == LUMEN_F32 ? 4 : 2), want = (size_t)ctx->num_sms * 3 * kWarps;
-    const int wpr = a.N * 4 <= want && row_bytes >= 4096 ? 4 : a.N * 2 <= want && row_bytes >= 2048 ? 2 : row_bytes >= 8192 && a.N * 2 <= 2 * want ? 2 : 1;
-    const int grid = pick_grid(ctx, a.N * wpr, smem);
+    const bool gated = a.act == StepFinish::kGated;
+    const size_t rows = gated ? 2 * a.N : a.N;
+    const int wpr = rows * 4 <= want && row_bytes >= 4096 ? 4 : rows * 2 <= want && row_bytes >= 2048 ? 2 : row_bytes >= 8192 && rows * 2 <= 2 * want ? 2 : 1;
+    const int grid = pick_grid(ctx, rows * wpr, smem);
+#define LUMEN_STEP_G(T_, W_, G_)                                                               \
+    do {                                                                                       \
+        LUMEN_TRY(set_smem(ctx, gemv_step_kernel<T_, W_, G_>, smem));                          \
+        return launch_pdl(ctx, gemv_step_kernel<T_, W_, G_>, grid, kThreads, smem, s, a);      \
+    } while (0)
 #define LUMEN_STEP(T_, W_)                                                                     \
     do {                                                                                       \
-        LUMEN_TRY(set_smem(ctx, gemv_step_kernel<T_, W_>, smem));                              \
-        return launch_pdl(ctx, gemv_step_kernel<T_, W_>, grid, kThreads, smem, s, a);          \
+        if (gated) LUMEN_STEP_G(T_, W_, true);                                                 \
+        LUMEN_STEP_G(T_, W_, false);                                                           \
     } while (0)
     if (a.wdt == LUMEN_F32) {
         if (wpr == 4) LUMEN_STEP(float, 4);
@@ -488,6 +534,7 @@ int launch_gemv_step(lumen_ctx *ctx, const GemvStepArgs &a, cudaStream_t s) {
     if (wpr == 2) LUMEN_STEP(__nv_bfloat16, 2);
     LUMEN_STEP(__nv_bfloat16, 1);
 #undef LUMEN_STEP
+#undef LUMEN_STEP_G
 }
 
 size_t gemv_kn_scratch_bytes_for(size_t K, size_t N, lumen_dtype wdt, int num_sms) {

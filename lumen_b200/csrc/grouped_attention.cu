@@ -1,0 +1,406 @@
+// Grouped-query attention over chunks: per-head RMS norm and partial rotation of queries and keys, a cache of keys and values
+// of sizes of their own (f32, or bf16 in bf16 models), a sink per head in the denominator, a sigmoid gate per head.  A position
+// sees the keys of its own chunk up to itself; chunks are counted from position 0, so a piece of the context is found from
+// the position alone, however the sequence was cut into steps.
+//
+//   grouped_append_kernel   keys and values of the step -> cache (and queries as the tensor-core kernel reads them)
+//   grouped_rows_kernel     scores, running softmax and weighted values of one row's pieces, any sizes (decode, short portions,
+//                           f32 models); in decode steps it appends the new row itself
+//   grouped_merge_kernel    pieces and sink merged, gate applied
+// Whole portions run on the tensor cores (attn_prefill_tc.cu).
+#include <algorithm>
+
+#include "attn_decode.cuh"
+#include "decoder_kernels.cuh"
+
+namespace lumen {
+namespace {
+
+constexpr int kThreads = 256;
+constexpr int kWarps = kThreads / 32;
+constexpr int kPiece = 32;  // pieces start at multiples of this many rows from the chunk's start
+
+// One head vector by one warp: RMS norm with gains, then the pairs (i, i + rot_dims / 2) turn.  buf: shared memory [dim].
+__device__ __forceinline__ void head_norm_rotate(float *buf, const float *src, int dim, const float *gain, float eps, int rot_dims,
+                                                 const float *cos_row, const float *sin_row, int lane) {
+    float ss = 0.f;
+#pragma unroll 4
+    for (int i = lane; i < dim; i += 32) {
+        const float v = src[i];
+        buf[i] = v;
+        ss = fmaf(v, v, ss);
+    }
+    ss = attn_warp_sum(ss);
+    const float inv = __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)dim), eps)));
+    for (int i = lane; i < dim; i += 32) buf[i] = __fmul_rn(__fmul_rn(buf[i], inv), gain[i]);
+    __syncwarp();
+    const int half = rot_dims / 2;
+    for (int i = lane; i < half; i += 32) {
+        const float x = buf[i], y = buf[i + half], c = cos_row[i], s = sin_row[i];
+        buf[i] = __fsub_rn(__fmul_rn(x, c), __fmul_rn(y, s));
+        buf[i + half] = __fadd_rn(__fmul_rn(y, c), __fmul_rn(x, s));
+    }
+    __syncwarp();
+}
+
+__device__ __forceinline__ int chunk_start(int pos, size_t chunk) { return chunk ? (int)((size_t)pos / chunk * chunk) : 0; }
+__device__ __forceinline__ int piece_rows(int len, int nsplit) { return ((len + nsplit - 1) / nsplit + kPiece - 1) / kPiece * kPiece; }
+
+// One warp per (row, key head), and with q per (padded row, query head): q[B, H, s_pad, width] bf16, zeros elsewhere.
+template <typename T>
+__global__ void __launch_bounds__(kThreads) grouped_append_kernel(const GroupedArgs a, size_t kv_items, __nv_bfloat16 *q, size_t s_pad, int width) {
+    extern __shared__ __align__(16) float smem[];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, dim = (int)a.dim, vdim = (int)a.vdim;
+    float *buf = smem + warp * dim;
+    pdl_launch();
+    pdl_wait();
+    size_t i = (size_t)blockIdx.x * kWarps + warp;
+    const size_t half = a.rot_dims / 2;
+    if (i >= kv_items) {
+        i -= kv_items;
+        if (!q || i >= a.B * s_pad * a.H) return;
+        const size_t bs = i / a.H, h = i - bs * a.H, b = bs / s_pad, s = bs - b * s_pad, pos = (size_t)*a.d_len + s;
+        __nv_bfloat16 *row = q + ((b * a.H + h) * s_pad + s) * width;
+        if (s < a.S)
+            head_norm_rotate(buf, a.u + (b * a.S + s) * a.u_ld + h * dim, dim, a.q_gain, a.eps, (int)a.rot_dims, a.cos_t + pos * half,
+                             a.sin_t + pos * half, lane);
+        for (int e = lane; e < width; e += 32) row[e] = __float2bfloat16_rn(s < a.S && e < dim ? buf[e] : 0.f);
+        return;
+    }
+    const size_t m = i / a.G, g = i - m * a.G, b = m / a.S, pos = (size_t)*a.d_len + (m - b * a.S);
+    const float *u = a.u + m * a.u_ld;
+    head_norm_rotate(buf, u + a.u_k + g * dim, dim, a.k_gain, a.eps, (int)a.rot_dims, a.cos_t + pos * half, a.sin_t + pos * half, lane);
+    const size_t row = (b * a.G + g) * a.max_seq + pos;
+    T *k = static_cast<T *>(a.k) + row * dim, *v = static_cast<T *>(a.v) + row * vdim;
+    for (int e = lane; e < dim; e += 32) k[e] = from_f32<T>(buf[e]);
+    const float *vs = u + a.u_v + g * vdim;
+    for (int e = lane; e < vdim; e += 32) v[e] = from_f32<T>(vs[e]);
+}
+
+// Two neighbouring elements of a cached row as they lie there.
+template <typename T>
+struct Pair {
+    using Raw = uint32_t;
+    static __device__ __forceinline__ Raw pack(float x, float y) {
+        const __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
+        return *reinterpret_cast<const Raw *>(&v);
+    }
+    static __device__ __forceinline__ float2 get(Raw r) { return make_float2(__uint_as_float(r << 16), __uint_as_float(r & 0xffff0000u)); }
+};
+template <>
+struct Pair<float> {
+    using Raw = float2;
+    static __device__ __forceinline__ Raw pack(float x, float y) { return make_float2(x, y); }
+    static __device__ __forceinline__ float2 get(Raw r) { return r; }
+};
+
+__host__ __device__ constexpr int rows_in_flight(int ni) { return ni <= 1 ? 8 : ni == 2 ? 4 : ni <= 4 ? 2 : 1; }
+
+// grid (pieces, G * (H / G / GT), rows): GT query heads of one key head against one piece of the row's chunk.  A lane holds the
+// element pairs lane + 32 i, i < NI, of keys and values.  EVEN: dim and vdim are even (pairs are loaded as one).
+template <typename T, int GT, int NI, bool EVEN>
+__global__ void __launch_bounds__(kThreads) grouped_rows_kernel(const GroupedArgs a, int append) {
+    using P = Pair<T>;
+    using Raw = typename P::Raw;
+    extern __shared__ __align__(16) float smem[];
+    constexpr int UN = rows_in_flight(NI), NV = UN * GT;
+    const int dim = (int)a.dim, vdim = (int)a.vdim, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    float *qs = smem;                       // [GT][dim]
+    float *knew = qs + GT * dim;            // [dim]
+    float *wm = knew + dim;                 // [warps][GT]
+    float *wl = wm + kWarps * GT;           // [warps][GT]
+    float *wsoft = wl + kWarps * GT;        // [warps][NV + GT]
+    float *wctx = wsoft + kWarps * (NV + GT);  // [warps][GT][vdim]
+    const int R = (int)(a.H / a.G), groups = R / GT, hk = (int)blockIdx.y / groups, h0 = hk * R + ((int)blockIdx.y % groups) * GT;
+    pdl_launch();
+    pdl_wait();
+    for (size_t m = blockIdx.z; m < a.B * a.S; m += gridDim.z) {
+        const size_t b = m / a.S;
+        const int pos = *a.d_len + (int)(m - b * a.S), lo = chunk_start(pos, a.chunk), len = pos + 1 - lo;
+        const int per = piece_rows(len, a.nsplit), j0 = lo + (int)blockIdx.x * per, j1 = min(pos + 1, j0 + per);
+        if (j0 >= j1) continue;  // (the same for the whole CTA)
+        const T *kbase = static_cast<const T *>(a.k) + (b * a.G + hk) * a.max_seq * dim;
+        const T *vbase = static_cast<const T *>(a.v) + (b * a.G + hk) * a.max_seq * vdim;
+        const float *u = a.u + m * a.u_ld;
+        Raw kra[UN][NI], vra[UN][NI], krb[UN][NI], vrb[UN][NI];
+        auto load_pair = [&](const T *row, int n, int e, bool ok) -> Raw {
+            if constexpr (EVEN) return ok && e < n ? __ldcg(reinterpret_cast<const Raw *>(row + e)) : P::pack(0.f, 0.f);
+            else return P::pack(ok && e < n ? to_f32(row[e]) : 0.f, ok && e + 1 < n ? to_f32(row[e + 1]) : 0.f);
+        };
+        auto load_rows = [&](int jb, Raw (&kr)[UN][NI], Raw (&vr)[UN][NI]) {
+#pragma unroll
+            for (int r = 0; r < UN; ++r) {
+                const int j = jb + r;
+                const bool ok = j < j1 && !(append && j == pos);  // (an appended row comes from the projections)
+#pragma unroll
+                for (int i = 0; i < NI; ++i) {
+                    const int e = 2 * (lane + 32 * i);
+                    kr[r][i] = load_pair(kbase + (size_t)j * dim, dim, e, ok);
+                    vr[r][i] = load_pair(vbase + (size_t)j * vdim, vdim, e, ok);
+                }
+            }
+        };
+        int jb = j0 + warp * UN;
+        if (jb < j1) load_rows(jb, kra, vra);
+        const size_t half = a.rot_dims / 2;
+        const float *cos_row = a.cos_t + pos * half, *sin_row = a.sin_t + pos * half;
+        for (int g = warp; g < GT; g += kWarps)
+            head_norm_rotate(qs + g * dim, u + (size_t)(h0 + g) * dim, dim, a.q_gain, a.eps, (int)a.rot_dims, cos_row, sin_row, lane);
+        const float *vnew = u + a.u_v + (size_t)hk * vdim;
+        if (append && j1 == pos + 1 && warp == kWarps - 1) {
+            head_norm_rotate(knew, u + a.u_k + (size_t)hk * dim, dim, a.k_gain, a.eps, (int)a.rot_dims, cos_row, sin_row, lane);
+            if ((int)blockIdx.y % groups == 0) {
+                T *k_row = const_cast<T *>(kbase) + (size_t)pos * dim, *v_row = const_cast<T *>(vbase) + (size_t)pos * vdim;
+                for (int e = lane; e < dim; e += 32) k_row[e] = from_f32<T>(knew[e]);
+                for (int e = lane; e < vdim; e += 32) v_row[e] = from_f32<T>(vnew[e]);
+            }
+        }
+        __syncthreads();
+
+        // A batch of UN rows x GT heads: the NV dot products are summed across the lanes by one butterfly, after which
+        // a lane holds HELD of them; GS lanes hold the scores of one head (see attn_decode.cuh).
+        constexpr int HELD = NV >= 32 ? NV / 32 : 1, DUP = NV >= 32 ? 1 : 32 / NV, GS = 32 / GT;
+        const int idx0 = NV >= 32 ? lane * HELD : lane / DUP, g_l = idx0 / UN;
+        const bool canonical = (lane % DUP) == 0;
+        float *ws = wsoft + warp * (NV + GT);
+        float2 q[GT][NI], ctx[GT][NI];
+        float m_h = -INFINITY, l_h = 0.f;
+#pragma unroll
+        for (int g = 0; g < GT; ++g)
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                const int e = 2 * (lane + 32 * i);
+                q[g][i] = make_float2(e < dim ? qs[g * dim + e] : 0.f, e + 1 < dim ? qs[g * dim + e + 1] : 0.f);
+                ctx[g][i] = make_float2(0.f, 0.f);
+            }
+        auto do_rows = [&](int jr, Raw (&kr)[UN][NI], Raw (&vr)[UN][NI]) {
+            if (append && pos >= jr && pos < jr + UN) {
+#pragma unroll
+                for (int r = 0; r < UN; ++r)
+                    if (jr + r == pos)
+#pragma unroll
+                        for (int i = 0; i < NI; ++i) {  // (rounded as the cache holds it)
+                            const int e = 2 * (lane + 32 * i);
+                            kr[r][i] = P::pack(e < dim ? knew[e] : 0.f, e + 1 < dim ? knew[e + 1] : 0.f);
+                            vr[r][i] = P::pack(e < vdim ? vnew[e] : 0.f, e + 1 < vdim ? vnew[e + 1] : 0.f);
+                        }
+            }
+            float d[NV];
+#pragma unroll
+            for (int g = 0; g < GT; ++g)
+#pragma unroll
+                for (int r = 0; r < UN; ++r) {
+                    float s = 0.f;
+#pragma unroll
+                    for (int i = 0; i < NI; ++i) {
+                        const float2 k = P::get(kr[r][i]);
+                        s = fmaf(q[g][i].x, k.x, s);
+                        s = fmaf(q[g][i].y, k.y, s);
+                    }
+                    d[g * UN + r] = s;
+                }
+            attn_reduce_multi<NV>(d, lane);
+            float sc[HELD], cmax = -INFINITY;
+#pragma unroll
+            for (int k = 0; k < HELD; ++k) {
+                sc[k] = jr + (idx0 + k) % UN < j1 ? __fmul_rn(d[k], a.scale) : -INFINITY;
+                cmax = fmaxf(cmax, sc[k]);
+            }
+#pragma unroll
+            for (int o = 1; o < GS; o <<= 1) cmax = fmaxf(cmax, __shfl_xor_sync(0xffffffffu, cmax, o));
+            const float mn = fmaxf(m_h, cmax), r = expf(m_h - mn);  // finite: the batch's first row is inside the piece
+            float wsum = 0.f;
+#pragma unroll
+            for (int k = 0; k < HELD; ++k) {
+                const float w = expf(sc[k] - mn);
+                if (canonical) ws[idx0 + k] = w;
+                wsum += w;
+            }
+            l_h = fmaf(l_h, r, canonical ? wsum : 0.f);
+            m_h = mn;
+            if ((lane & (GS - 1)) == 0) ws[NV + g_l] = r;
+            __syncwarp();
+#pragma unroll
+            for (int g = 0; g < GT; ++g) {
+                const float rg = ws[NV + g];
+#pragma unroll
+                for (int i = 0; i < NI; ++i) {
+                    ctx[g][i].x *= rg;
+                    ctx[g][i].y *= rg;
+                }
+#pragma unroll
+                for (int rr = 0; rr < UN; ++rr) {
+                    const float w = ws[g * UN + rr];
+#pragma unroll
+                    for (int i = 0; i < NI; ++i) {
+                        const float2 v = P::get(vr[rr][i]);
+                        ctx[g][i].x = fmaf(w, v.x, ctx[g][i].x);
+                        ctx[g][i].y = fmaf(w, v.y, ctx[g][i].y);
+                    }
+                }
+            }
+            __syncwarp();  // the weights are overwritten by the next batch
+        };
+        constexpr int kStep = kWarps * UN;
+        while (jb < j1) {  // the next batch is always in flight
+            if (jb + kStep < j1) load_rows(jb + kStep, krb, vrb);
+            do_rows(jb, kra, vra);
+            jb += kStep;
+            if (jb >= j1) break;
+            if (jb + kStep < j1) load_rows(jb + kStep, kra, vra);
+            do_rows(jb, krb, vrb);
+            jb += kStep;
+        }
+#pragma unroll
+        for (int o = 1; o < GS; o <<= 1) l_h += __shfl_xor_sync(0xffffffffu, l_h, o);
+        if ((lane & (GS - 1)) == 0) {
+            wm[warp * GT + g_l] = m_h;
+            wl[warp * GT + g_l] = l_h;
+        }
+#pragma unroll
+        for (int g = 0; g < GT; ++g)
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                const int e = 2 * (lane + 32 * i);
+                if (e < vdim) wctx[(warp * GT + g) * vdim + e] = ctx[g][i].x;
+                if (e + 1 < vdim) wctx[(warp * GT + g) * vdim + e + 1] = ctx[g][i].y;
+            }
+        __syncthreads();
+        for (int i = tid; i < GT * vdim; i += kThreads) {
+            const int g = i / vdim, e = i - g * vdim;
+            float M = -INFINITY, L = 0.f, c = 0.f;
+#pragma unroll
+            for (int w = 0; w < kWarps; ++w) M = fmaxf(M, wm[w * GT + g]);
+#pragma unroll
+            for (int w = 0; w < kWarps; ++w) {
+                const float mw = wm[w * GT + g], f = mw == -INFINITY ? 0.f : expf(mw - M);
+                L = fmaf(wl[w * GT + g], f, L);
+                c = fmaf(wctx[(w * GT + g) * vdim + e], f, c);
+            }
+            const size_t o = (m * a.H + h0 + g) * a.nsplit + blockIdx.x;
+            a.part_ctx[o * vdim + e] = c;
+            if (e == 0) {
+                a.part_ml[o * 2] = M;
+                a.part_ml[o * 2 + 1] = L;
+            }
+        }
+        __syncthreads();
+    }
+}
+
+// grid (heads, rows)
+constexpr int kMergeThreads = 128;
+__global__ void __launch_bounds__(kMergeThreads) grouped_merge_kernel(const GroupedArgs a) {
+    const size_t h = blockIdx.x;
+    const int vdim = (int)a.vdim;
+    pdl_launch();
+    pdl_wait();
+    for (size_t m = blockIdx.y; m < a.B * a.S; m += gridDim.y) {
+        const size_t b = m / a.S, row = m * a.H + h;
+        const int pos = *a.d_len + (int)(m - b * a.S), len = pos + 1 - chunk_start(pos, a.chunk), per = piece_rows(len, a.nsplit);
+        const int pieces = (len + per - 1) / per;
+        const float *ml = a.part_ml + row * a.nsplit * 2;
+        const float sink = a.sink[h];
+        float M = sink;
+#pragma unroll 8
+        for (int i = 0; i < pieces; ++i) M = fmaxf(M, ml[2 * i]);
+        float L = expf(sink - M);
+#pragma unroll 8
+        for (int i = 0; i < pieces; ++i) L = fmaf(ml[2 * i + 1], expf(ml[2 * i] - M), L);
+        const float f = __fdiv_rn(sigmoid_f(a.u[m * a.u_ld + a.u_gate + h]), L);
+        for (int e = threadIdx.x; e < vdim; e += kMergeThreads) {
+            float c = 0.f;
+#pragma unroll 8
+            for (int i = 0; i < pieces; ++i) c = fmaf(a.part_ctx[(row * a.nsplit + i) * vdim + e], expf(ml[2 * i] - M), c);
+            c *= f;
+            if (a.out) a.out[row * vdim + e] = c;
+            if (a.out_hi) store_split(c, a.out_hi, a.out_lo, row * vdim + e);
+        }
+    }
+}
+
+// grid (row tiles of 64, column tiles of 64, matrices)
+__global__ void __launch_bounds__(256) transpose_rows_kernel(const __nv_bfloat16 *__restrict__ in, size_t in_rows, int cols, size_t row0, int rows,
+                                                             __nv_bfloat16 *__restrict__ out, size_t pitch) {
+    __shared__ __nv_bfloat16 tile[64][66];
+    const int r0 = blockIdx.x * 64, c0 = blockIdx.y * 64;
+    const size_t mat = blockIdx.z;
+    for (int i = threadIdx.x; i < 64 * 64; i += 256) {
+        const int r = i >> 6, c = i & 63;
+        tile[r][c] = r0 + r < rows && c0 + c < cols ? in[(mat * in_rows + row0 + r0 + r) * cols + c0 + c] : __float2bfloat16_rn(0.f);
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < 64 * 64; i += 256) {
+        const int c = i >> 6, r = i & 63;
+        if (c0 + c < cols && (size_t)(r0 + r) < pitch) out[(mat * cols + c0 + c) * pitch + r0 + r] = tile[r][c];
+    }
+}
+
+template <typename T, int GT, int NI, bool EVEN>
+int launch_rows(lumen_ctx *ctx, const GroupedArgs &a, bool append, cudaStream_t s) {
+    constexpr int NV = rows_in_flight(NI) * GT;
+    const size_t smem = ((GT + 1) * a.dim + 2 * kWarps * GT + kWarps * (NV + GT) + (size_t)kWarps * GT * a.vdim) * sizeof(float);
+    if (smem > 48 * 1024) LUMEN_CUDA(ctx, cudaFuncSetAttribute(grouped_rows_kernel<T, GT, NI, EVEN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    const dim3 grid((unsigned)a.nsplit, (unsigned)(a.H / GT), (unsigned)std::min<size_t>(a.B * a.S, 65535));
+    return launch_pdl(ctx, grouped_rows_kernel<T, GT, NI, EVEN>, grid, kThreads, smem, s, a, append ? 1 : 0);
+}
+template <typename T, int GT>
+int launch_rows_g(lumen_ctx *ctx, const GroupedArgs &a, bool append, cudaStream_t s) {
+    const size_t n = std::max(a.dim, a.vdim);
+    if (a.dim % 2 || a.vdim % 2) {
+        if (n <= 64) return launch_rows<T, GT, 1, false>(ctx, a, append, s);
+        if (n <= 256) return launch_rows<T, GT, 4, false>(ctx, a, append, s);
+        return launch_rows<T, 1, 8, false>(ctx, a, append, s);
+    }
+    if (n <= 64) return launch_rows<T, GT, 1, true>(ctx, a, append, s);
+    if (n <= 128) return launch_rows<T, GT, 2, true>(ctx, a, append, s);
+    if (n <= 256) return launch_rows<T, GT, 4, true>(ctx, a, append, s);
+    return launch_rows<T, 1, 8, true>(ctx, a, append, s);
+}
+int group_of(const GroupedArgs &a) {  // query heads a CTA takes
+    const size_t r = a.H / a.G;
+    return std::max(a.dim, a.vdim) > 256 ? 1 : r % 4 == 0 ? 4 : r % 2 == 0 ? 2 : 1;
+}
+
+}  // namespace
+
+// Two CTAs per SM, pieces of at least 64 rows, partial results within the workspace (see ensure_workspace).
+int grouped_pick_splits(const GroupedArgs &a, int num_sms) {
+    const size_t rows = a.B * a.S, items = rows * a.H / group_of(a), total = a.past + a.S;
+    const size_t len = a.chunk ? std::min(total, a.chunk) : total;
+    size_t n = std::min((2 * (size_t)num_sms + items - 1) / items, (len + 63) / 64);
+    n = std::min(n, (size_t)num_sms * 64 / (rows * a.H));
+    // few distinct counts: every one of them is a graph of its own
+    size_t p = 1;
+    while (p * 2 <= n) p *= 2;
+    return (int)p;
+}
+
+int launch_grouped_append(lumen_ctx *ctx, const GroupedArgs &a, __nv_bfloat16 *q, size_t s_pad, size_t width, cudaStream_t s) {
+    const size_t kv_items = a.own_kv ? a.B * a.S * a.G : 0, items = kv_items + (q ? a.B * s_pad * a.H : 0);
+    if (items == 0) return LUMEN_OK;
+    const auto kernel = a.dt == LUMEN_F32 ? grouped_append_kernel<float> : grouped_append_kernel<__nv_bfloat16>;
+    return launch_pdl(ctx, kernel, (unsigned)((items + kWarps - 1) / kWarps), kThreads, kWarps * a.dim * sizeof(float), s, a, kv_items, q, s_pad, (int)width);
+}
+
+int launch_grouped_attention(lumen_ctx *ctx, const GroupedArgs &a, bool append, cudaStream_t s) {
+    if (std::max(a.dim, a.vdim) > kGroupedMaxDim) return set_error(ctx, LUMEN_ERR_UNSUPPORTED, "attention: heads of %zu / %zu numbers", a.dim, a.vdim);
+    const bool f32 = a.dt == LUMEN_F32;
+    int rc;
+    switch (group_of(a)) {
+        case 4: rc = f32 ? launch_rows_g<float, 4>(ctx, a, append, s) : launch_rows_g<__nv_bfloat16, 4>(ctx, a, append, s); break;
+        case 2: rc = f32 ? launch_rows_g<float, 2>(ctx, a, append, s) : launch_rows_g<__nv_bfloat16, 2>(ctx, a, append, s); break;
+        default: rc = f32 ? launch_rows_g<float, 1>(ctx, a, append, s) : launch_rows_g<__nv_bfloat16, 1>(ctx, a, append, s); break;
+    }
+    if (rc != LUMEN_OK) return rc;
+    return launch_pdl(ctx, grouped_merge_kernel, dim3((unsigned)a.H, (unsigned)std::min<size_t>(a.B * a.S, 65535)), kMergeThreads, 0, s, a);
+}
+
+int launch_transpose_rows(lumen_ctx *ctx, const __nv_bfloat16 *in, size_t in_rows, size_t cols, size_t mats, size_t row0, size_t rows,
+                          __nv_bfloat16 *out, size_t pitch, cudaStream_t s) {
+    transpose_rows_kernel<<<dim3((unsigned)((pitch + 63) / 64), (unsigned)((cols + 63) / 64), (unsigned)mats), 256, 0, s>>>(in, in_rows, (int)cols, row0, (int)rows, out, pitch);
+    LUMEN_LAUNCHED(ctx);
+    return LUMEN_OK;
+}
+
+}  // namespace lumen

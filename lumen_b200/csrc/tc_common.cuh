@@ -42,6 +42,11 @@ __device__ __forceinline__ void tma_load_2d(void *dst, const CUtensorMap *map, i
     asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
                  ::"r"(saddr(dst)), "l"(map), "r"(x), "r"(y), "r"(saddr(bar)) : "memory");
 }
+// The same from a 3-D map: box (kBK elements, 1, rows) at (x, y, z = row).
+__device__ __forceinline__ void tma_load_3d(void *dst, const CUtensorMap *map, int x, int y, int z, uint64_t *bar) {
+    asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];"
+                 ::"r"(saddr(dst)), "l"(map), "r"(x), "r"(y), "r"(z), "r"(saddr(bar)) : "memory");
+}
 // Shared-memory matrix descriptor of a K-major bf16 tile stored as rows of 128 bytes with the 128-byte
 // swizzle (what the TMA box above produces): start address, leading offset 1 (unused with swizzle), 1024
 // bytes between groups of 8 rows, descriptor version 1, layout type 2 = 128-byte swizzle.
@@ -80,6 +85,36 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&v)[32]) {
     tmem_ld_wait();
 }
 
+__device__ __forceinline__ float ex2(float x) {  // 2^x, one MUFU operation (relative error 2^-22; -inf -> 0)
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
+    const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
+    return *reinterpret_cast<const uint32_t *>(&v);
+}
+
+// A wait that also ends when another thread of the CTA has given up (nobody leaves the tile loop early, so
+// every barrier keeps its full set of participants; after a failure the remaining iterations do not wait).
+__device__ __forceinline__ bool wait_or_failed(uint64_t *bar, uint32_t parity, volatile int *failed, DeviceStatus *status, int site) {
+    if (*failed) return false;
+    if (bar_try(bar, parity)) return true;
+    const long long t0 = clock64();
+    while (!bar_try(bar, parity)) {
+        if (*failed) return false;
+        if (clock64() - t0 > kTcWaitCycles) {
+            if (status && atomicCAS(&status->code, 0, LUMEN_ERR_TIMEOUT) == 0) status->detail0 = site;
+            *failed = 1;
+            return false;
+        }
+    }
+    return true;
+}
+__device__ __forceinline__ void bar_arrive(uint64_t *bar) {
+    asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(saddr(bar)) : "memory");
+}
+
 typedef CUresult (*EncodeTiledFn)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *, const cuuint64_t *,
                                   const cuuint32_t *, const cuuint32_t *, CUtensorMapInterleave, CUtensorMapSwizzle,
                                   CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
@@ -105,6 +140,22 @@ inline int make_map(lumen_ctx *ctx, CUtensorMap *map, const void *base, size_t r
     const cuuint32_t box[2] = {(cuuint32_t)kBK, (cuuint32_t)box_rows};
     const cuuint32_t estr[2] = {1, 1};
     CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void *>(base), dims, strides, box, estr,
+                    CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
+                    CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (r != CUDA_SUCCESS) return set_error(ctx, LUMEN_ERR_CUDA, "cuTensorMapEncodeTiled failed with %d", (int)r);
+    return LUMEN_OK;
+}
+
+// Rows of `heads` vectors of `dim` bf16 numbers, `ld` elements between rows -> map with box (kBK, 1 head, box_rows): what lies
+// beyond a head's numbers is filled with zeros, not with the next head.
+inline int make_map_heads(lumen_ctx *ctx, CUtensorMap *map, const void *base, size_t rows, size_t heads, size_t dim, size_t ld, int box_rows) {
+    EncodeTiledFn fn = encode_fn();
+    if (!fn) return set_error(ctx, LUMEN_ERR_CUDA, "cuTensorMapEncodeTiled is not available from this driver");
+    const cuuint64_t dims[3] = {(cuuint64_t)dim, (cuuint64_t)heads, (cuuint64_t)rows};
+    const cuuint64_t strides[2] = {(cuuint64_t)dim * 2, (cuuint64_t)ld * 2};
+    const cuuint32_t box[3] = {(cuuint32_t)kBK, 1, (cuuint32_t)box_rows};
+    const cuuint32_t estr[3] = {1, 1, 1};
+    CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void *>(base), dims, strides, box, estr,
                     CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
                     CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     if (r != CUDA_SUCCESS) return set_error(ctx, LUMEN_ERR_CUDA, "cuTensorMapEncodeTiled failed with %d", (int)r);

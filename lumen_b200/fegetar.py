@@ -6,12 +6,11 @@ particular model's values.
 """
 from __future__ import annotations
 
-import ctypes as C
 from dataclasses import dataclass, field
 
 from . import _lib
 from ._lib import BF16, F32, DecoderConfigC, DecoderLayerC
-from .model import LanguageModel
+from .model import DecoderModel
 
 
 @dataclass
@@ -62,7 +61,7 @@ class LayerConfig:
         kind = _lib.MLP_MOE if self.experts else _lib.MLP_DENSE if self.ff else _lib.MLP_NONE
         e, s = self.expert or ExpertConfig(0, 0.0), self.shared or ExpertConfig(0, 0.0)
         return DecoderLayerC(self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank, self.rot_dims, self.rot_base, self.scale, kind,
-                             self.ff, self.experts, self.top, e.ff, e.limit, s.ff, s.limit)
+                             self.ff, self.experts, self.top, e.ff, e.limit, s.ff, s.limit, _lib.MIXER_LATENT, 0, -1)
 
 
 @dataclass
@@ -92,7 +91,7 @@ class FegetarConfig:
     def to_c(self) -> DecoderConfigC:
         arr = (DecoderLayerC * max(len(self.layers), 1))(*[x.to_c() for x in self.layers])
         return DecoderConfigC(self.vocab_size, self.width, len(self.layers), arr, self.norm_eps, self.max_seq_len, self.bigram_buckets,
-                              self.bigram_mul_prev, self.bigram_mul_cur, self.side_dim, BF16 if self.weight_dtype == "bf16" else F32)
+                              self.bigram_mul_prev, self.bigram_mul_cur, self.side_dim, BF16 if self.weight_dtype == "bf16" else F32, 1.0, 0, _lib.NORM_OUTPUT)
 
     def param_shapes(self) -> dict:
         w, v = self.width, self.vocab_size
@@ -122,13 +121,7 @@ class FegetarConfig:
         return shapes
 
 
-class FegetarModel(LanguageModel):
-    """Parameters start unset; fill them with `set_param` / `load_state` / the loader, under their checkpoint names."""
-
-    def _new(self) -> None:
-        cfg_c = self.config.to_c()
-        self.ctx.check(self.ctx._lib.lumen_decoder_new(self.ctx.h, C.byref(cfg_c), C.byref(self.h)))
-
+class FegetarModel(DecoderModel):
     def _cache_shape(self, layer: int, batch: int) -> tuple:
         k = self.config.layers[layer]
         return batch, 1, self.config.max_seq_len, -(-(k.kv_rank + k.rot_dim) // 16) * 16

@@ -121,3 +121,12 @@ class LanguageModel:
         require_no_grad(f"{type(self).__name__}::forward")
         self.ctx.check(self._fn("forward_device")(self.h, ids_ptr, b, s, self._cache_array(caches),
                                                                 len(caches), logits_ptr))
+
+
+class DecoderModel(LanguageModel):
+    """A model given as a list of layers (`config.to_c()` is a `lumen_decoder_config`).  Parameters start unset; fill them with
+    `set_param` / `load_state` / the loader, under their checkpoint names."""
+
+    def _new(self) -> None:
+        cfg_c = self.config.to_c()
+        self.ctx.check(self.ctx._lib.lumen_decoder_new(self.ctx.h, C.byref(cfg_c), C.byref(self.h)))

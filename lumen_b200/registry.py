@@ -9,6 +9,7 @@ import json
 from pathlib import Path
 
 from .fegetar import FegetarConfig, FegetarModel
+from .fekorax import FekoraxConfig, FekoraxModel
 from .llama import LlamaConfig, LlamaModel
 from .loader import load_weights
 
@@ -27,6 +28,7 @@ MODELS = {
     "LlamaForCausalLM": (_llama_config, LlamaModel),
     "Qwen3ForCausalLM": (lambda d, n, dt: _llama_config(d, n, dt, qk_norm=True), LlamaModel),
     "Fegetar": (lambda d, n, dt: FegetarConfig.from_dict(d, int(n or 2048), dt), FegetarModel),
+    "Fekorax": (lambda d, n, dt: FekoraxConfig.from_dict(d, int(n or 2048), dt), FekoraxModel),
 }
 
 
