@@ -366,12 +366,35 @@ LAYER_CASES = {
     # routed: a token uses 6 of 64 experts and the shared one, 3 x (6 x 1408 + 2816) x 2048 parameters = LlamaModel with 11264
     "moe_2048": dict(width=2048, layers=4, heads=16, rank=512, moe=dict(experts=64, top=6, ff=1408, shared=2816),
                      llama=dict(intermediate_size=11264, num_key_value_heads=8)),
+    # Fekorax: twice (three matrix-memory layers, attention, a matrix-memory layer, attention over the former one's keys and values), the
+    # attention layers with a feed-forward; its parameters are those of 7 layers of the LlamaModel
+    "mix_2048": dict(width=2048, layers=7, heads=16, llama=dict(intermediate_size=5632, num_key_value_heads=4),
+                     matrix=dict(heads=8, dim=128, vdim=256), chunk=3072),
+    "mix_4096": dict(width=4096, layers=7, heads=32, llama=dict(intermediate_size=11008, num_key_value_heads=8),
+                     matrix=dict(heads=8, dim=256, vdim=512), chunk=6144),
 }
 
 
+def fekorax_layers(c: dict) -> list:
+    matrix = dict(type="mlstm", mixer=dict(c["matrix"], gate_cap=15.0), mlp=None)
+    out = []
+    for i in range(2):
+        mixer = dict(heads=c["heads"], kv_heads=c["llama"]["num_key_value_heads"], dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=c["chunk"]),
+                     rot=dict(base=500000.0, dims=64, scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192)))
+        mlp = dict(kind="dense", ff=c["llama"]["intermediate_size"])
+        out += [matrix] * 3 + [dict(type="attention", mixer=mixer, mlp=mlp), matrix, dict(type="attention", mixer=dict(mixer, kv_from=6 * i + 3), mlp=mlp)]
+    return out
+
+
 def layer_models(L, case: str, max_seq: int):
-    """(FegetarConfig, LlamaConfig) of a case: heads of 128 (+ 64 rotated), values of 128."""
+    """(name, configuration of the model given as a list of layers), LlamaConfig of a case.  Fegetar: heads of 128 (+ 64 rotated), values
+    of 128."""
     c = LAYER_CASES[case]
+    llama = L.LlamaConfig(vocab_size=4096, hidden_size=c["width"], num_hidden_layers=c["layers"], num_attention_heads=c["heads"], head_dim=128,
+                          max_seq_len=max_seq, weight_dtype="bf16", **c["llama"])
+    if "matrix" in c:
+        d = dict(architecture="Fekorax", vocab=4096, width=c["width"], norm=dict(eps=1e-5), embedding=dict(scale=1.0), layers=fekorax_layers(c))
+        return ("fekorax", L.FekoraxConfig.from_dict(d, max_seq, "bf16")), llama
     mixer = dict(heads=c["heads"], dim=128, rot_dim=64, vdim=128, kv_rank=c["rank"], scale=192 ** -0.5, rot=dict(base=10000.0, dims=64))
     if "moe" in c:
         m = c["moe"]
@@ -382,9 +405,28 @@ def layer_models(L, case: str, max_seq: int):
     d = dict(architecture="Fegetar", vocab=4096, width=c["width"], norm=dict(eps=1e-5), token_side=dict(dim=256),
              embedding=dict(bigram=dict(buckets=65521, mul_prev=1000003, mul_cur=101)),
              layers=[dict(type="latent_attention", mixer=mixer, mlp=mlp)] * c["layers"])
-    return L.FegetarConfig.from_dict(d, max_seq, "bf16"), L.LlamaConfig(
-        vocab_size=4096, hidden_size=c["width"], num_hidden_layers=c["layers"], num_attention_heads=c["heads"], head_dim=128,
-        max_seq_len=max_seq, weight_dtype="bf16", **c["llama"])
+    return ("fegetar", L.FegetarConfig.from_dict(d, max_seq, "bf16")), llama
+
+
+def layer_work(name: str, cfg, case: str, n: int) -> tuple:
+    """(operations of the mixers beside their projections over a prompt of n positions, bytes of cache and state that a decode step
+    at context n touches)."""
+    c = LAYER_CASES[case]
+    if name == "fekorax":
+        flops = nbytes = 0.0
+        for k in cfg.layers:
+            if k.type == "mlstm":  # the recurrence itself: update and read
+                flops += 4.0 * n * k.heads * k.dim * k.vdim
+                nbytes += 2 * 4 * k.heads * k.dim * k.vdim
+            else:
+                full, rest = divmod(n, k.chunk)
+                pairs = full * k.chunk * (k.chunk + 1) / 2 + rest * (rest + 1) / 2
+                flops += k.heads * pairs * 2 * (k.dim + k.vdim)
+                nbytes += k.kv_heads * (n % k.chunk + 1) * (k.dim + k.vdim) * 2
+        return flops, nbytes
+    qk, vd = (192, 128) if name == "fegetar" else (128, 128)
+    row_bytes = 576 * 2 if name == "fegetar" else 2 * c["llama"]["num_key_value_heads"] * 128 * 4
+    return c["layers"] * c["heads"] * n * (n + 1) / 2 * 2 * (qk + vd), c["layers"] * row_bytes * (n + 40)
 
 
 def run_layers(args):
@@ -403,7 +445,7 @@ def run_layers(args):
         tpeak = 1590.0
     cases = [args.layers_case] if args.layers_case else list(LAYER_CASES)
     phases = [args.layers_phase] if args.layers_phase else ["prefill", "decode"]
-    models = [args.layers_model] if args.layers_model else ["fegetar", "llama"]
+    models = [args.layers_model] if args.layers_model else ["fegetar", "fekorax", "llama"]
     lens = [int(x) for x in args.layers_lens.split(",")]
     rng = np.random.default_rng(0)
     base = f32_to_bf16_bits(rng.standard_normal(1 << 22, dtype=np.float32) * np.float32(0.02))
@@ -412,10 +454,11 @@ def run_layers(args):
     sampler.active = True
     for case in cases:
         max_seq = max(lens) + 96
-        for name, cfg in zip(("fegetar", "llama"), layer_models(L, case, max_seq)):
+        listed, llama_cfg = layer_models(L, case, max_seq)
+        for name, cfg in (listed, ("llama", llama_cfg)):
             if name not in models:
                 continue
-            model = (L.FegetarModel if name == "fegetar" else L.LlamaModel)(cfg, ctx)
+            model = {"fegetar": L.FegetarModel, "fekorax": L.FekoraxModel, "llama": L.LlamaModel}[name](cfg, ctx)
             for i, (n, shape) in enumerate(sorted(cfg.param_shapes().items())):
                 size = int(np.prod(shape))
                 if len(shape) == 1:
@@ -425,14 +468,12 @@ def run_layers(args):
             caches = model.init_kv_caches(1)
             ids = L.Tensor.from_array_no_grad(rng.integers(0, 4096, max_seq).astype(np.float32), ctx)
             logits = L.Tensor.from_array_no_grad(np.zeros(max(lens) * 4096, np.float32), ctx)
-            layer_params = sum(int(np.prod(s)) for n, s in cfg.param_shapes().items()
-                               if len(s) == 2 and n not in ("embed", "bigram", "side.embed", "model.embed_tokens.weight") and ".mlp.e" not in n)
+            layer_params = cfg.width * cfg.vocab_size if name == "fekorax" else 0  # (the embedding is the output matrix)
+            layer_params += sum(int(np.prod(s)) for n, s in cfg.param_shapes().items()
+                                if len(s) == 2 and n not in ("embed", "bigram", "side.embed", "model.embed_tokens.weight") and ".mlp.e" not in n)
             if "moe" in LAYER_CASES[case] and name == "fegetar":
                 m = LAYER_CASES[case]["moe"]
                 layer_params += LAYER_CASES[case]["layers"] * 3 * m["top"] * m["ff"] * cfg.width
-            heads, n_layers = LAYER_CASES[case]["heads"], LAYER_CASES[case]["layers"]
-            qk, vd = (192, 128) if name == "fegetar" else (128, 128)
-            row_bytes = 576 * 2 if name == "fegetar" else 2 * LAYER_CASES[case]["llama"]["num_key_value_heads"] * 128 * 4
             with L.no_grad():
                 for n in lens:
                     if "prefill" in phases:
@@ -440,7 +481,7 @@ def run_layers(args):
                             model.reset_kv_caches(caches)
                             model.forward_device(ids.data_ptr, 1, n, caches, logits.data_ptr)
                         ms = _event_time_ms(ctx, stream, step, iters=5 if not args.layers_once else 1, warm=3 if not args.layers_once else 1)
-                        flops = 2.0 * n * layer_params + n_layers * heads * n * (n + 1) / 2 * 2 * (qk + vd)
+                        flops = 2.0 * n * layer_params + layer_work(name, cfg, case, n)[0]
                         print(json.dumps({"micro": "layers_prefill", "case": case, "model": name, "positions": n, "ms": ms, "tokens_per_s": n / ms * 1e3,
                                           "tflops": flops / ms / 1e9, "frac_of_measured_bf16": flops / ms / 1e9 / tpeak}), flush=True)
                     if "decode" in phases:
@@ -448,7 +489,7 @@ def run_layers(args):
                         model.forward_device(ids.data_ptr, 1, n, caches, logits.data_ptr)
                         ms = _event_time_ms(ctx, stream, lambda: model.forward_device(ids.data_ptr, 1, 1, caches, logits.data_ptr),
                                             iters=64 if not args.layers_once else 2, warm=8 if not args.layers_once else 2)
-                        nbytes = model.weight_bytes_per_step + n_layers * row_bytes * (n + 40)
+                        nbytes = model.weight_bytes_per_step + layer_work(name, cfg, case, n)[1]
                         gbs = nbytes / ms / 1e6
                         print(json.dumps({"micro": "layers_decode", "case": case, "model": name, "context": n, "ms": ms, "tokens_per_s": 1e3 / ms,
                                           "weight_mb": model.weight_bytes_per_step / 1e6, "gbs": gbs, "frac_of_measured_hbm": gbs / hbm, "peak_kind": kind,
@@ -487,7 +528,7 @@ def main():
     ap.add_argument("--prefill-chunk", type=int, default=0,
                     help="prefill the prompt in slices of this many positions (0: one forward)")
     ap.add_argument("--layers-case", choices=list(LAYER_CASES), default=None, help="--micro layers: one case only")
-    ap.add_argument("--layers-model", choices=["fegetar", "llama"], default=None, help="--micro layers: one model only")
+    ap.add_argument("--layers-model", choices=["fegetar", "fekorax", "llama"], default=None, help="--micro layers: one model only")
     ap.add_argument("--layers-phase", choices=["prefill", "decode"], default=None, help="--micro layers: one phase only")
     ap.add_argument("--layers-lens", default="512,2048,8192", help="--micro layers: prompt lengths / contexts")
     ap.add_argument("--layers-once", action="store_true", help="--micro layers: very few steps (profiling aid, not a measurement)")
