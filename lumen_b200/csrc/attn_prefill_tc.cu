@@ -375,6 +375,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_qhi, const __grid
                     const float f = p.gate ? inv * sigmoid_f(p.gate[orow * p.gate_ld + h]) : inv;
                     const size_t at = (orow * p.Hq + h) * p.vdim + half * kDH;
                     const int n = min(kDH, p.vdim - half * kDH);
+                    if (!p.out && !p.out_lo && p.vdim % 8 == 0) {  // 16 bytes at a time
+#pragma unroll
+                        for (int e = 0; e < kDH; e += 8)
+                            if (e < n)
+                                *reinterpret_cast<uint4 *>(p.out_hi + at + e) =
+                                    make_uint4(pack_bf16(ctx[e] * f, ctx[e + 1] * f), pack_bf16(ctx[e + 2] * f, ctx[e + 3] * f),
+                                               pack_bf16(ctx[e + 4] * f, ctx[e + 5] * f), pack_bf16(ctx[e + 6] * f, ctx[e + 7] * f));
+                    } else
 #pragma unroll
                     for (int e = 0; e < kDH; ++e)
                         if (e < n) {

@@ -168,12 +168,13 @@ gemv_gate_up_kernel(const float *__restrict__ x, const WT *__restrict__ wg, cons
     }
 }
 
+constexpr int kStepCtas = 4;  // of gemv_step_kernel per SM
 // One row whose input may still owe the norm of a sublayer's output (post-norm models): x = res + RMSNorm(y) * gain is
 // formed by every CTA while it stages x, so that the norm, the residual sum and the product are one launch.  WPR warps share a
 // weight row (a slice of K each) where there are too few rows to keep enough loads in flight.
 // GATED: N gate rows and the N up rows that go with them (in blocks, see kGateBlock) are walked as pairs; out = gelu_tanh(gate) * up.
 template <typename WT, int WPR, bool GATED>
-__global__ void __launch_bounds__(kThreads, 4) gemv_step_kernel(const GemvStepArgs a) {
+__global__ void __launch_bounds__(kThreads, kStepCtas) gemv_step_kernel(const GemvStepArgs a) {
     extern __shared__ __align__(16) float smem[];
     __shared__ float red[kWarps];
     float *xs = smem;
@@ -295,9 +296,10 @@ __global__ void __launch_bounds__(kThreads, 4) gemv_step_kernel(const GemvStepAr
         float v = 0.f;
         if (row < n_rows) {
             if (vec_ok) {
+                const size_t after = row + (size_t)gridDim.x * kRows;
                 const uint4 *wrow = reinterpret_cast<const uint4 *>(w + stored(row) * K) + v0;
-                if (row != row0) batch_load(wrow, 0, vn, lane, pre);
-                v = row_dot_ahead<WT>(wrow, xs + v0 * VEC, vn, lane, pre);
+                const uint4 *next = after < n_rows ? reinterpret_cast<const uint4 *>(w + stored(after) * K) + v0 : nullptr;
+                v = row_dot_ahead<WT>(wrow, xs + v0 * VEC, vn, lane, pre, next);
             } else if (part == 0) {
                 v = row_dot_scalar<WT>(w + stored(row) * K, xs, (int)K, lane);
             }
@@ -514,7 +516,8 @@ int launch_gemv_step(lumen_ctx *ctx, const GemvStepArgs &a, cudaStream_t s) {
     const bool gated = a.act == StepFinish::kGated;
     const size_t rows = gated ? 2 * a.N : a.N;
     const int wpr = rows * 4 <= want && row_bytes >= 4096 ? 4 : rows * 2 <= want && row_bytes >= 2048 ? 2 : row_bytes >= 8192 && rows * 2 <= 2 * want ? 2 : 1;
-    const int grid = pick_grid(ctx, rows * wpr, smem);
+    // as many CTAs as the device holds: each stages its input once
+    const int grid = std::min(pick_grid(ctx, rows * wpr, smem), ctx->num_sms * kStepCtas);
 #define LUMEN_STEP_G(T_, W_, G_)                                                               \
     do {                                                                                       \
         LUMEN_TRY(set_smem(ctx, gemv_step_kernel<T_, W_, G_>, smem));                          \

@@ -135,13 +135,15 @@ __device__ __forceinline__ float vec_dot(uint4 w, const float *x, float acc) {
     }
 }
 template <typename WT>
-__device__ __forceinline__ float row_dot_ahead(const uint4 *__restrict__ row, const float *xs, int n, int lane, uint4 (&cur)[kAhead]) {
+__device__ __forceinline__ float row_dot_ahead(const uint4 *__restrict__ row, const float *xs, int n, int lane, uint4 (&cur)[kAhead],
+                                               const uint4 *__restrict__ next_row = nullptr) {  // its first batch is left in cur
     constexpr int VEC = 16 / sizeof(WT);
     float acc = 0.f;
 #pragma unroll 1
     for (int base = 0; base < n; base += kAhead * 32) {
         uint4 next[kAhead];
-        batch_load(row, base + kAhead * 32, n, lane, next);
+        if (next_row && base + kAhead * 32 >= n) batch_load(next_row, 0, n, lane, next);
+        else batch_load(row, base + kAhead * 32, n, lane, next);
 #pragma unroll
         for (int u = 0; u < kAhead; ++u) {
             const int i = base + u * 32 + lane;

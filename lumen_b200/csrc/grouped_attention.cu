@@ -46,34 +46,81 @@ __device__ __forceinline__ void head_norm_rotate(float *buf, const float *src, i
 __device__ __forceinline__ int chunk_start(int pos, size_t chunk) { return chunk ? (int)((size_t)pos / chunk * chunk) : 0; }
 __device__ __forceinline__ int piece_rows(int len, int nsplit) { return ((len + nsplit - 1) / nsplit + kPiece - 1) / kPiece * kPiece; }
 
-// One warp per (row, key head), and with q per (padded row, query head): q[B, H, s_pad, width] bf16, zeros elsewhere.
+// The same in registers, four neighbouring elements per lane (dim <= 128, everything a multiple of four): every load is issued
+// at once, the other half of a pair comes from another lane.
+__device__ __forceinline__ float4 head_norm_rotate4(const float *src, int dim, const float *gain, float eps, int rot_dims, const float *cos_row,
+                                                    const float *sin_row, int lane) {
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    const int e = 4 * lane, half = rot_dims / 2;
+    const bool in = e < dim, turns = e < rot_dims;
+    const float4 v = in ? *reinterpret_cast<const float4 *>(src + e) : zero, g = in ? *reinterpret_cast<const float4 *>(gain + e) : zero;
+    const int p = e < half ? e : e - half;
+    const float4 c = turns ? *reinterpret_cast<const float4 *>(cos_row + p) : zero, s = turns ? *reinterpret_cast<const float4 *>(sin_row + p) : zero;
+    const float ss = attn_warp_sum(fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w))));
+    const float inv = __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)dim), eps)));
+    float x[4] = {__fmul_rn(__fmul_rn(v.x, inv), g.x), __fmul_rn(__fmul_rn(v.y, inv), g.y), __fmul_rn(__fmul_rn(v.z, inv), g.z),
+                  __fmul_rn(__fmul_rn(v.w, inv), g.w)};
+    const float cv[4] = {c.x, c.y, c.z, c.w}, sv[4] = {s.x, s.y, s.z, s.w};
+    const int other = (e < half ? e + half : e - half) / 4 & 31;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+        const float y = __shfl_sync(0xffffffffu, x[k], other);
+        if (turns) x[k] = e < half ? __fsub_rn(__fmul_rn(x[k], cv[k]), __fmul_rn(y, sv[k])) : __fadd_rn(__fmul_rn(x[k], cv[k]), __fmul_rn(y, sv[k]));
+    }
+    return make_float4(x[0], x[1], x[2], x[3]);
+}
 template <typename T>
-__global__ void __launch_bounds__(kThreads) grouped_append_kernel(const GroupedArgs a, size_t kv_items, __nv_bfloat16 *q, size_t s_pad, int width) {
+__device__ __forceinline__ void store4(T *p, float4 v) {
+    if constexpr (sizeof(T) == 4) {
+        *reinterpret_cast<float4 *>(p) = v;
+    } else {
+        const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+        *reinterpret_cast<uint2 *>(p) = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+    }
+}
+
+// Portions: one warp per (row, key head), and with q per (padded row, query head): q[B, H, s_pad, width] bf16, zeros elsewhere.
+// VEC: head_norm_rotate4.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(kThreads) grouped_append_kernel(const GroupedArgs a, unsigned kv_items, __nv_bfloat16 *q, unsigned s_pad, int width) {
     extern __shared__ __align__(16) float smem[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, dim = (int)a.dim, vdim = (int)a.vdim;
     float *buf = smem + warp * dim;
-    pdl_launch();
-    pdl_wait();
-    size_t i = (size_t)blockIdx.x * kWarps + warp;
+    unsigned i = blockIdx.x * kWarps + warp;  // (fewer than 2^32 items, see the launcher)
+    const unsigned S = (unsigned)a.S, H = (unsigned)a.H, G = (unsigned)a.G;
     const size_t half = a.rot_dims / 2;
     if (i >= kv_items) {
         i -= kv_items;
-        if (!q || i >= a.B * s_pad * a.H) return;
-        const size_t bs = i / a.H, h = i - bs * a.H, b = bs / s_pad, s = bs - b * s_pad, pos = (size_t)*a.d_len + s;
-        __nv_bfloat16 *row = q + ((b * a.H + h) * s_pad + s) * width;
-        if (s < a.S)
-            head_norm_rotate(buf, a.u + (b * a.S + s) * a.u_ld + h * dim, dim, a.q_gain, a.eps, (int)a.rot_dims, a.cos_t + pos * half,
-                             a.sin_t + pos * half, lane);
-        for (int e = lane; e < width; e += 32) row[e] = __float2bfloat16_rn(s < a.S && e < dim ? buf[e] : 0.f);
+        const unsigned bs = i / H, h = i - bs * H, b = bs / s_pad, s = bs - b * s_pad;
+        if (!q || b >= a.B) return;
+        const size_t pos = a.past + s;
+        __nv_bfloat16 *row = q + ((size_t)(b * H + h) * s_pad + s) * width;
+        const float *src = a.u + (size_t)(b * S + s) * a.u_ld + h * dim, *cos_row = a.cos_t + pos * half, *sin_row = a.sin_t + pos * half;
+        if (VEC) {
+            const float4 v = s < S ? head_norm_rotate4(src, dim, a.q_gain, a.eps, (int)a.rot_dims, cos_row, sin_row, lane) : make_float4(0.f, 0.f, 0.f, 0.f);
+            if (4 * lane < width) store4(row + 4 * lane, v);  // (lanes beyond dim hold zeros)
+            return;
+        }
+        if (s < S) head_norm_rotate(buf, src, dim, a.q_gain, a.eps, (int)a.rot_dims, cos_row, sin_row, lane);
+        for (int e = lane; e < width; e += 32) row[e] = __float2bfloat16_rn(s < S && e < dim ? buf[e] : 0.f);
         return;
     }
-    const size_t m = i / a.G, g = i - m * a.G, b = m / a.S, pos = (size_t)*a.d_len + (m - b * a.S);
-    const float *u = a.u + m * a.u_ld;
-    head_norm_rotate(buf, u + a.u_k + g * dim, dim, a.k_gain, a.eps, (int)a.rot_dims, a.cos_t + pos * half, a.sin_t + pos * half, lane);
-    const size_t row = (b * a.G + g) * a.max_seq + pos;
+    const unsigned m = i / G, g = i - m * G, b = m / S;
+    const size_t pos = a.past + (m - b * S);
+    const float *u = a.u + m * a.u_ld, *ks = u + a.u_k + g * dim, *vs = u + a.u_v + g * vdim;
+    const float *cos_row = a.cos_t + pos * half, *sin_row = a.sin_t + pos * half;
+    const size_t row = (size_t)(b * G + g) * a.max_seq + pos;
     T *k = static_cast<T *>(a.k) + row * dim, *v = static_cast<T *>(a.v) + row * vdim;
+    if (VEC) {
+        const bool mine = 4 * lane < vdim;
+        const float4 val = mine ? *reinterpret_cast<const float4 *>(vs + 4 * lane) : make_float4(0.f, 0.f, 0.f, 0.f);
+        const float4 key = head_norm_rotate4(ks, dim, a.k_gain, a.eps, (int)a.rot_dims, cos_row, sin_row, lane);
+        if (4 * lane < dim) store4(k + 4 * lane, key);
+        if (mine) store4(v + 4 * lane, val);
+        return;
+    }
+    head_norm_rotate(buf, ks, dim, a.k_gain, a.eps, (int)a.rot_dims, cos_row, sin_row, lane);
     for (int e = lane; e < dim; e += 32) k[e] = from_f32<T>(buf[e]);
-    const float *vs = u + a.u_v + g * vdim;
     for (int e = lane; e < vdim; e += 32) v[e] = from_f32<T>(vs[e]);
 }
 
@@ -113,12 +160,19 @@ __global__ void __launch_bounds__(kThreads) grouped_rows_kernel(const GroupedArg
     float *wctx = wsoft + kWarps * (NV + GT);  // [warps][GT][vdim]
     const int R = (int)(a.H / a.G), groups = R / GT, hk = (int)blockIdx.y / groups, h0 = hk * R + ((int)blockIdx.y % groups) * GT;
     pdl_launch();
-    pdl_wait();
+    // A step's own kernels write no cached row but the appended one, and the length only at its end: a layer that appends requests its
+    // first rows while the projections still run.
+    bool ahead = append;
+    if (!ahead) pdl_wait();
     for (size_t m = blockIdx.z; m < a.B * a.S; m += gridDim.z) {
         const size_t b = m / a.S;
         const int pos = *a.d_len + (int)(m - b * a.S), lo = chunk_start(pos, a.chunk), len = pos + 1 - lo;
         const int per = piece_rows(len, a.nsplit), j0 = lo + (int)blockIdx.x * per, j1 = min(pos + 1, j0 + per);
-        if (j0 >= j1) continue;  // (the same for the whole CTA)
+        if (j0 >= j1) {  // (the same for the whole CTA)
+            if (ahead) pdl_wait();
+            ahead = false;
+            continue;
+        }
         const T *kbase = static_cast<const T *>(a.k) + (b * a.G + hk) * a.max_seq * dim;
         const T *vbase = static_cast<const T *>(a.v) + (b * a.G + hk) * a.max_seq * vdim;
         const float *u = a.u + m * a.u_ld;
@@ -142,6 +196,8 @@ __global__ void __launch_bounds__(kThreads) grouped_rows_kernel(const GroupedArg
         };
         int jb = j0 + warp * UN;
         if (jb < j1) load_rows(jb, kra, vra);
+        if (ahead) pdl_wait();
+        ahead = false;
         const size_t half = a.rot_dims / 2;
         const float *cos_row = a.cos_t + pos * half, *sin_row = a.sin_t + pos * half;
         for (int g = warp; g < GT; g += kWarps)
@@ -289,8 +345,9 @@ __global__ void __launch_bounds__(kThreads) grouped_rows_kernel(const GroupedArg
 }
 
 // grid (heads, rows)
-constexpr int kMergeThreads = 128;
+constexpr int kMergeThreads = 128, kMaxPieces = 128;
 __global__ void __launch_bounds__(kMergeThreads) grouped_merge_kernel(const GroupedArgs a) {
+    __shared__ float w_s[kMaxPieces];
     const size_t h = blockIdx.x;
     const int vdim = (int)a.vdim;
     pdl_launch();
@@ -299,23 +356,48 @@ __global__ void __launch_bounds__(kMergeThreads) grouped_merge_kernel(const Grou
         const size_t b = m / a.S, row = m * a.H + h;
         const int pos = *a.d_len + (int)(m - b * a.S), len = pos + 1 - chunk_start(pos, a.chunk), per = piece_rows(len, a.nsplit);
         const int pieces = (len + per - 1) / per;
-        const float *ml = a.part_ml + row * a.nsplit * 2;
-        const float sink = a.sink[h];
-        float M = sink;
-#pragma unroll 8
-        for (int i = 0; i < pieces; ++i) M = fmaxf(M, ml[2 * i]);
-        float L = expf(sink - M);
-#pragma unroll 8
-        for (int i = 0; i < pieces; ++i) L = fmaf(ml[2 * i + 1], expf(ml[2 * i] - M), L);
+        const float2 *ml = reinterpret_cast<const float2 *>(a.part_ml) + row * a.nsplit;
+        const float *ctx = a.part_ctx + row * a.nsplit * vdim;
+        const int e0 = threadIdx.x;
+        float first[8];  // requested before the weights are known
+#pragma unroll
+        for (int i = 0; i < 8; ++i) first[i] = i < pieces && e0 < vdim ? ctx[(size_t)i * vdim + e0] : 0.f;
+        // every warp finds the maximum and the sum for itself, a piece per lane (grouped_pick_splits: at most kMaxPieces)
+        const int lane = threadIdx.x & 31;
+        float mx[kMaxPieces / 32], sum[kMaxPieces / 32], M = a.sink[h], L = 0.f;
+#pragma unroll
+        for (int k = 0; k < kMaxPieces / 32; ++k) {
+            const float2 v = lane + 32 * k < pieces ? ml[lane + 32 * k] : make_float2(-INFINITY, 0.f);
+            mx[k] = v.x;
+            sum[k] = v.y;
+            M = fmaxf(M, v.x);
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, o));
+#pragma unroll
+        for (int k = 0; k < kMaxPieces / 32; ++k) {
+            mx[k] = expf(mx[k] - M);
+            L = fmaf(sum[k], mx[k], L);
+        }
+        L = attn_warp_sum(L) + expf(a.sink[h] - M);
+        if (threadIdx.x < 32)
+#pragma unroll
+            for (int k = 0; k < kMaxPieces / 32; ++k)
+                if (lane + 32 * k < pieces) w_s[lane + 32 * k] = mx[k];
+        __syncthreads();
         const float f = __fdiv_rn(sigmoid_f(a.u[m * a.u_ld + a.u_gate + h]), L);
-        for (int e = threadIdx.x; e < vdim; e += kMergeThreads) {
+        for (int e = e0; e < vdim; e += kMergeThreads) {
             float c = 0.f;
+#pragma unroll
+            for (int i = 0; i < 8; ++i)
+                if (i < pieces) c = fmaf(e == e0 ? first[i] : ctx[(size_t)i * vdim + e], w_s[i], c);
 #pragma unroll 8
-            for (int i = 0; i < pieces; ++i) c = fmaf(a.part_ctx[(row * a.nsplit + i) * vdim + e], expf(ml[2 * i] - M), c);
+            for (int i = 8; i < pieces; ++i) c = fmaf(ctx[(size_t)i * vdim + e], w_s[i], c);
             c *= f;
             if (a.out) a.out[row * vdim + e] = c;
             if (a.out_hi) store_split(c, a.out_hi, a.out_lo, row * vdim + e);
         }
+        __syncthreads();  // the weights are overwritten by the next row
     }
 }
 
@@ -369,7 +451,7 @@ int grouped_pick_splits(const GroupedArgs &a, int num_sms) {
     const size_t rows = a.B * a.S, items = rows * a.H / group_of(a), total = a.past + a.S;
     const size_t len = a.chunk ? std::min(total, a.chunk) : total;
     size_t n = std::min((2 * (size_t)num_sms + items - 1) / items, (len + 63) / 64);
-    n = std::min(n, (size_t)num_sms * 64 / (rows * a.H));
+    n = std::min(std::min(n, (size_t)kMaxPieces), (size_t)num_sms * 64 / (rows * a.H));
     // few distinct counts: every one of them is a graph of its own
     size_t p = 1;
     while (p * 2 <= n) p *= 2;
@@ -379,8 +461,14 @@ int grouped_pick_splits(const GroupedArgs &a, int num_sms) {
 int launch_grouped_append(lumen_ctx *ctx, const GroupedArgs &a, __nv_bfloat16 *q, size_t s_pad, size_t width, cudaStream_t s) {
     const size_t kv_items = a.own_kv ? a.B * a.S * a.G : 0, items = kv_items + (q ? a.B * s_pad * a.H : 0);
     if (items == 0) return LUMEN_OK;
-    const auto kernel = a.dt == LUMEN_F32 ? grouped_append_kernel<float> : grouped_append_kernel<__nv_bfloat16>;
-    return launch_pdl(ctx, kernel, (unsigned)((items + kWarps - 1) / kWarps), kThreads, kWarps * a.dim * sizeof(float), s, a, kv_items, q, s_pad, (int)width);
+    if (items >= ((size_t)1 << 31)) return set_error(ctx, LUMEN_ERR_UNSUPPORTED, "attention: %zu head vectors in one step", items);
+    // (width is a multiple of 64, so it is at most 128 where dim is)
+    const bool vec = a.dim <= 128 && a.vdim <= 128 && a.dim % 4 == 0 && a.vdim % 4 == 0 && a.rot_dims % 8 == 0 && a.u_ld % 4 == 0;
+    const auto kernel = a.dt == LUMEN_F32 ? (vec ? grouped_append_kernel<float, true> : grouped_append_kernel<float, false>)
+                                          : (vec ? grouped_append_kernel<__nv_bfloat16, true> : grouped_append_kernel<__nv_bfloat16, false>);
+    kernel<<<(unsigned)((items + kWarps - 1) / kWarps), kThreads, vec ? 0 : kWarps * a.dim * sizeof(float), s>>>(a, (unsigned)kv_items, q, (unsigned)s_pad, (int)width);
+    LUMEN_LAUNCHED(ctx);
+    return LUMEN_OK;
 }
 
 int launch_grouped_attention(lumen_ctx *ctx, const GroupedArgs &a, bool append, cudaStream_t s) {

@@ -50,9 +50,8 @@ __global__ void __launch_bounds__(kThreads) mlstm_step_kernel(const MlstmArgs a,
     float *ks = qs + T * dim;         // [T][dim]
     float *nq = ks + T * dim;         // [T][dim] products of n and q
     float *ns = nq + T * dim;         // [dim]
-    float *os = ns + dim;             // [T][cols]
-    float *red = os + T * cols;       // [T][ny][cols]
-    __shared__ float al[T], be[T], em[T], den[T], inv[T];
+    float *red = ns + dim;            // [T][ny][cols]
+    __shared__ float al[T], be[T], em[T];
     __shared__ float ssq[2][T];       // read by the other CTAs of the cluster
     cg::cluster_group cluster = cg::this_cluster();
     const int h = blockIdx.y, b = blockIdx.z, c0 = blockIdx.x * cols;
@@ -60,17 +59,19 @@ __global__ void __launch_bounds__(kThreads) mlstm_step_kernel(const MlstmArgs a,
     const bool active = ty < ny && col < vdim;
     const size_t bh = (size_t)b * a.H + h;
     float *st = a.state + bh * dim * vdim + col;
+    // What the cache holds does not depend on this step's projections: it is requested while they still run.  (No other kernel of a
+    // step writes it, and the length changes at the step's end.)
     Cols<VEC> pre[T == 1 ? kPre : 1];
-    if (T == 1) {  // the memory does not depend on this step's projections
+    if (T == 1) {
 #pragma unroll
         for (int i = 0; i < kPre; ++i)
             if (active && ty + i * ny < dim) pre[i] = load_cols<VEC>(st + (size_t)(ty + i * ny) * vdim);
     }
-    pdl_launch();
-    pdl_wait();
     const bool fresh = *a.d_len == 0;
     for (int i = tid; i < dim; i += kThreads) ns[i] = fresh ? 0.f : a.norm[bh * dim + i];
     float m = fresh ? 0.f : a.mx[bh];  // (kept by the first warp)
+    pdl_launch();
+    pdl_wait();
     const float qscale = rsqrtf_exact((float)dim);
     int buf = 0;
 #pragma unroll 1
@@ -104,6 +105,22 @@ __global__ void __launch_bounds__(kThreads) mlstm_step_kernel(const MlstmArgs a,
                 em[lane] = expf(-mine);
             }
         }
+        Cols<VEC> vb[T];
+        if (active)
+#pragma unroll
+            for (int t = 0; t < T; ++t)
+#pragma unroll
+                for (int k = 0; k < VEC; ++k) vb[t].v[k] = t < nt ? a.u[(row0 + t) * a.u_ld + a.u_v + (size_t)h * vdim + col + k] : 0.f;
+        // what the last stage multiplies with (a warp finishes token `warp`; the first two columns of a lane are ready by then)
+        float gain[2] = {0.f, 0.f}, gate[2] = {0.f, 0.f};
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const int c = lane + 32 * k;
+            if (warp < nt && c < cols && c0 + c < vdim) {
+                gain[k] = a.head_gain[(size_t)h * vdim + c0 + c];
+                gate[k] = a.u[(row0 + warp) * a.u_ld + a.u_g + (size_t)h * vdim + c0 + c];
+            }
+        }
         __syncthreads();
         for (int r = tid; r < dim; r += kThreads) {
             float n = ns[r];
@@ -116,12 +133,12 @@ __global__ void __launch_bounds__(kThreads) mlstm_step_kernel(const MlstmArgs a,
             ns[r] = n;
         }
         if (active) {
-            Cols<VEC> vb[T], acc[T];
+            Cols<VEC> acc[T];
 #pragma unroll
             for (int t = 0; t < T; ++t) {
 #pragma unroll
                 for (int k = 0; k < VEC; ++k) {
-                    vb[t].v[k] = t < nt ? be[t] * a.u[(row0 + t) * a.u_ld + a.u_v + (size_t)h * vdim + col + k] : 0.f;
+                    if (t < nt) vb[t].v[k] *= be[t];
                     acc[t].v[k] = 0.f;
                 }
             }
@@ -165,43 +182,39 @@ __global__ void __launch_bounds__(kThreads) mlstm_step_kernel(const MlstmArgs a,
                 for (int k = 0; k < VEC; ++k) red[(t * ny + ty) * cols + tx * VEC + k] = acc[t].v[k];
         }
         __syncthreads();
-        for (int t = warp; t < nt; t += kWarps) {
+        // warp t finishes token t (T <= 8 warps): denominator, this slice's outputs and their sum of squares
+        static_assert(T <= kWarps, "a warp per token");
+        const int t = warp;
+        float *os = red + (size_t)t * ny * cols;  // (the sums over the row groups replace the first group's)
+        if (t < nt) {
             float s = 0.f;
             for (int r = lane; r < dim; r += 32) s += nq[t * dim + r];
-            s = warp_sum(s);
-            if (lane == 0) den[t] = fmaxf(fabsf(s), em[t]) + 1e-6f;
-        }
-        __syncthreads();
-        for (int i = tid; i < nt * cols; i += kThreads) {
-            const int t = i / cols, c = i - t * cols;
-            float o = 0.f;
-            if (c0 + c < vdim) {
-                for (int y = 0; y < ny; ++y) o += red[(t * ny + y) * cols + c];
-                o = __fdiv_rn(o, den[t]);
+            const float den = fmaxf(fabsf(warp_sum(s)), em[t]) + 1e-6f;
+            float ss = 0.f;
+            for (int c = lane; c < cols; c += 32) {
+                float o = 0.f;
+                if (c0 + c < vdim) {
+#pragma unroll 8
+                    for (int y = 0; y < ny; ++y) o += os[y * cols + c];
+                    o = __fdiv_rn(o, den);
+                }
+                os[c] = o;
+                ss = fmaf(o, o, ss);
             }
-            os[i] = o;
-        }
-        __syncthreads();
-        for (int t = warp; t < nt; t += kWarps) {
-            float s = 0.f;
-            for (int c = lane; c < cols; c += 32) s = fmaf(os[t * cols + c], os[t * cols + c], s);
-            s = warp_sum(s);
-            if (lane == 0) ssq[buf][t] = s;
+            ss = warp_sum(ss);
+            if (lane == 0) ssq[buf][t] = ss;
         }
         cluster.sync();  // (the buffer is rewritten two passes later, after every CTA has been through the next barrier)
-        if (tid < nt) {
-            float s = 0.f;
-            for (unsigned r = 0; r < cluster.num_blocks(); ++r) s += *cluster.map_shared_rank(&ssq[buf][tid], r);
-            inv[tid] = __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(s, (float)vdim), a.eps)));
-        }
-        __syncthreads();
-        for (int i = tid; i < nt * cols; i += kThreads) {
-            const int t = i / cols, c = i - t * cols;
-            if (c0 + c >= vdim) continue;
-            const size_t j = (size_t)h * vdim + c0 + c, at = (row0 + t) * a.H * vdim + j;
-            const float v = os[i] * inv[t] * a.head_gain[j] * sigmoid_f(a.u[(row0 + t) * a.u_ld + a.u_g + j]);
-            if (a.out) a.out[at] = v;
-            if (a.out_hi) store_split(v, a.out_hi, a.out_lo, at);
+        if (t < nt) {
+            const float ss = warp_sum(lane < (int)cluster.num_blocks() ? *cluster.map_shared_rank(&ssq[buf][t], lane) : 0.f);
+            const float inv = __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)vdim), a.eps)));
+            for (int c = lane, k = 0; c < cols && c0 + c < vdim; c += 32, ++k) {
+                const size_t j = (size_t)h * vdim + c0 + c, at = (row0 + t) * a.H * vdim + j;
+                const float hg = k == 0 ? gain[0] : k == 1 ? gain[1] : a.head_gain[j], g = k == 0 ? gate[0] : k == 1 ? gate[1] : a.u[(row0 + t) * a.u_ld + a.u_g + j];
+                const float v = os[c] * inv * hg * sigmoid_f(g);
+                if (a.out) a.out[at] = v;
+                if (a.out_hi) store_split(v, a.out_hi, a.out_lo, at);
+            }
         }
         __syncthreads();
     }
@@ -216,7 +229,7 @@ __global__ void __launch_bounds__(kThreads) mlstm_step_kernel(const MlstmArgs a,
 template <int VEC, int T>
 int launch_step(lumen_ctx *ctx, const MlstmArgs &a, int cols, unsigned slices, cudaStream_t s) {
     const int nx = cols / VEC, ny = kThreads / nx;
-    const size_t smem = ((size_t)T * (3 * a.dim + cols + (size_t)ny * cols) + a.dim) * sizeof(float);
+    const size_t smem = ((size_t)T * (3 * a.dim + (size_t)ny * cols) + a.dim) * sizeof(float);
     if (smem > 200 * 1024) return set_error(ctx, LUMEN_ERR_UNSUPPORTED, "matrix memory: keys of %zu numbers", a.dim);
     if (smem > 48 * 1024) LUMEN_CUDA(ctx, cudaFuncSetAttribute(mlstm_step_kernel<VEC, T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     return launch_pdl_cluster(ctx, mlstm_step_kernel<VEC, T>, slices, dim3(slices, (unsigned)a.H, (unsigned)a.B), kThreads, smem, s, a, cols, nx, ny);

@@ -186,18 +186,20 @@ constexpr int kStN = 64;                             // keys of a tile
 constexpr uint32_t kStA = 128 * kBK * 2, kStB = kStN * kBK * 2;
 constexpr uint32_t kStStage = 2 * kStA + 4 * kStB;   // v^T: two blocks of 64 tokens; weighted k^T: hi and lo of each
 constexpr int kStStages = 3;
-constexpr size_t kStSmem = kStStages * kStStage + 1024;
+constexpr size_t kStSmem = kStStages * kStStage + 2 * kStA + 1024;  // + the tile on its way out, hi and lo
 
 // grid (value tiles of 128, key tiles of 64, B * H); warps 0-7 keep the tile, warp 8 issues the MMAs, warp 9 the copies
 __global__ void __launch_bounds__(kTcThreads, 1)
 mlstm_state_kernel(const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_khi,
-                   const __grid_constant__ CUtensorMap map_klo, const Seg p) {
+                   const __grid_constant__ CUtensorMap map_klo, const __grid_constant__ CUtensorMap map_shi, const __grid_constant__ CUtensorMap map_slo,
+                   const Seg p) {
     extern __shared__ unsigned char smem_raw[];
     unsigned char *ring = reinterpret_cast<unsigned char *>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
     __shared__ uint64_t full[kStStages], empty[kStStages], d_full[2], d_free[2];
     __shared__ uint32_t tmem_base_s;
     __shared__ int failed_s;
     __shared__ float decay[kSegChunks];
+    unsigned char *s_out = ring + kStStages * kStStage;
     volatile int *failed = &failed_s;
     const int tid = threadIdx.x, warp = tid >> 5, nc = p.n_chunks;
     const int m0 = blockIdx.x * 128, n0 = blockIdx.y * kStN, bh = blockIdx.z;
@@ -282,22 +284,31 @@ mlstm_state_kernel(const __grid_constant__ CUtensorMap map_v, const __grid_const
 #pragma unroll 1
         for (int c = 0; c < nc; ++c) {
             const size_t bc = (size_t)bh * nc + c;
-            if (live) {
-                const size_t at = (bc * p.vdim + val) * p.dim + key0;
+            if (!(p.fresh && c == 0)) {  // (the memory before the first token is not read)
+                if (tid == 0) tma_store_wait_read();  // the previous chunk's copies have left shared memory
+                __syncwarp();
+                asm volatile("bar.sync 1, 256;" ::: "memory");
 #pragma unroll
-                for (int q = 0; q < 4; ++q)
-                    if (key0 + 8 * q < p.dim) {
-                        uint4 hi, lo;
-                        uint32_t *hp = &hi.x, *lp = &lo.x;
+                for (int q = 0; q < 4; ++q) {
+                    uint4 hi, lo;
+                    uint32_t *hp = &hi.x, *lp = &lo.x;
 #pragma unroll
-                        for (int j = 0; j < 4; ++j) {
-                            const float x = S[8 * q + 2 * j], y = S[8 * q + 2 * j + 1];
-                            hp[j] = pack_bf16(x, y);
-                            lp[j] = pack_bf16(x - __uint_as_float(hp[j] << 16), y - __uint_as_float(hp[j] & 0xffff0000u));
-                        }
-                        *reinterpret_cast<uint4 *>(p.s_hi + at + 8 * q) = hi;
-                        *reinterpret_cast<uint4 *>(p.s_lo + at + 8 * q) = lo;
+                    for (int j = 0; j < 4; ++j) {
+                        const float x = S[8 * q + 2 * j], y = S[8 * q + 2 * j + 1];
+                        hp[j] = pack_bf16(x, y);
+                        lp[j] = pack_bf16(x - __uint_as_float(hp[j] << 16), y - __uint_as_float(hp[j] & 0xffff0000u));
                     }
+                    unsigned char *dst = s_out + (size_t)row * 128 + (((4 * half + q) ^ (row & 7)) << 4);  // 128-byte swizzle
+                    *reinterpret_cast<uint4 *>(dst) = hi;
+                    *reinterpret_cast<uint4 *>(dst + kStA) = lo;
+                }
+                asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+                asm volatile("bar.sync 1, 256;" ::: "memory");
+                if (tid == 0) {
+                    tma_store_3d(&map_shi, s_out, n0, m0, (int)bc);
+                    tma_store_3d(&map_slo, s_out + kStA, n0, m0, (int)bc);
+                    tma_store_commit();
+                }
             }
             if (nlive) {
                 p.nst[bc * p.dim + n0 + tid] = n;
@@ -319,6 +330,7 @@ mlstm_state_kernel(const __grid_constant__ CUtensorMap map_v, const __grid_const
             for (int i = 0; i < 32; ++i)
                 if (key0 + i < p.dim) st[(size_t)(key0 + i) * p.vdim] = S[i];
         if (nlive) p.norm[(size_t)bh * p.dim + n0 + tid] = n;
+        if (tid == 0) tma_store_wait();
     }
     __syncthreads();
     if (*failed && tid == kWorkers + 32) {  // copies in flight land before the CTA exits (bounded)
@@ -611,16 +623,15 @@ mlstm_out_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constan
 // One thread per 8 outputs of a row.
 __global__ void __launch_bounds__(256) mlstm_finish_kernel(const Seg p, const float *__restrict__ gain, float eps, float *__restrict__ out,
                                                            __nv_bfloat16 *__restrict__ hi, __nv_bfloat16 *__restrict__ lo) {
-    const size_t i = (size_t)blockIdx.x * 256 + threadIdx.x, per_row = (size_t)p.H * p.vdim / 8;
-    if (i >= (size_t)p.B * p.T * per_row) return;
-    const size_t row = i / per_row;
-    const unsigned j = (unsigned)(i - row * per_row) * 8, h = j / (unsigned)p.vdim;
-    const size_t b = row / p.T, m = b * p.S + p.t0 + (row - b * p.T);
-    const float *ss = p.ssq + (row * p.H + h) * 2 * p.tiles;
+    const unsigned i = blockIdx.x * 256 + threadIdx.x, per_row = (unsigned)p.H * p.vdim / 8, row = i / per_row;  // (see mlstm_chunked_usable)
+    if (row >= (unsigned)(p.B * p.T)) return;
+    const unsigned j = (i - row * per_row) * 8, h = j / (unsigned)p.vdim, b = row / (unsigned)p.T;
+    const size_t m = (size_t)b * p.S + p.t0 + (row - b * p.T);
+    const float *ss = p.ssq + ((size_t)row * p.H + h) * 2 * p.tiles;
     float s = 0.f;
     for (int k = 0; k < 2 * p.tiles; ++k) s += ss[k];
     const float inv = __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(s, (float)p.vdim), eps)));
-    const uint4 ov = *reinterpret_cast<const uint4 *>(p.o + i * 8), gv = *reinterpret_cast<const uint4 *>(p.u + m * p.u_ld + p.u_g + j);
+    const uint4 ov = *reinterpret_cast<const uint4 *>(p.o + (size_t)i * 8), gv = *reinterpret_cast<const uint4 *>(p.u + m * p.u_ld + p.u_g + j);
     const float4 n0 = *reinterpret_cast<const float4 *>(gain + j), n1 = *reinterpret_cast<const float4 *>(gain + j + 4);
     const float n[8] = {n0.x, n0.y, n0.z, n0.w, n1.x, n1.y, n1.z, n1.w};
     const uint32_t *ow = &ov.x, *gw = &gv.x;
@@ -629,7 +640,7 @@ __global__ void __launch_bounds__(256) mlstm_finish_kernel(const Seg p, const fl
 #pragma unroll
     for (int k = 0; k < 8; ++k) {
         const float o = __uint_as_float(k & 1 ? ow[k / 2] & 0xffff0000u : ow[k / 2] << 16), g = __uint_as_float(k & 1 ? gw[k / 2] & 0xffff0000u : gw[k / 2] << 16);
-        v[k] = o * inv * n[k] * sigmoid_f(g);
+        v[k] = o * inv * n[k] * __fdividef(1.0f, 1.0f + ex2(-g * kLog2e));  // (rounded to 16 bits next; 1 / inf = 0)
     }
     if (hi && !lo) {
         *reinterpret_cast<uint4 *>(hi + at) = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
@@ -660,7 +671,7 @@ bool mlstm_chunked_usable(const MlstmArgs &a) {
         return e && e[0] == '1';
     }();
     return !off && a.S >= 64 && a.dim <= 256 && a.dim % 8 == 0 && a.vdim % 8 == 0 && a.u_ld % 8 == 0 && a.B * a.H <= 65535 &&
-           a.B * a.S < ((size_t)1 << 31) && a.B * a.H * kSegChunks * std::max(a.vdim, a.dim) < ((size_t)1 << 31);
+           a.B * a.S * a.H * a.vdim / 8 < ((size_t)1 << 31) && a.B * a.S < ((size_t)1 << 31) && a.B * a.H * kSegChunks * std::max(a.vdim, a.dim) < ((size_t)1 << 31);
 }
 
 int launch_mlstm_chunked(lumen_ctx *ctx, const MlstmArgs &a, cudaStream_t s) {
@@ -691,20 +702,22 @@ int launch_mlstm_chunked(lumen_ctx *ctx, const MlstmArgs &a, cudaStream_t s) {
         mlstm_pack_kernel<<<dim3(c, kg + vg, (unsigned)BH), 256, 0, s>>>(p);
         LUMEN_LAUNCHED(ctx);
         const size_t pitch = (size_t)c * kC;
-        CUtensorMap st[3], out[5];
+        CUtensorMap st[5], out[5];
         LUMEN_TRY(make_map(ctx, &st[0], p.vt, BH * a.vdim, pitch, 128));
         LUMEN_TRY(make_map(ctx, &st[1], p.kt_hi, BH * a.dim, pitch, kStN));
         LUMEN_TRY(make_map(ctx, &st[2], p.kt_lo, BH * a.dim, pitch, kStN));
+        LUMEN_TRY(make_map_3d(ctx, &st[3], p.s_hi, a.dim, a.vdim, a.dim, BH * c, a.vdim * a.dim, 128, 1));
+        LUMEN_TRY(make_map_3d(ctx, &st[4], p.s_lo, a.dim, a.vdim, a.dim, BH * c, a.vdim * a.dim, 128, 1));
         LUMEN_CUDA(ctx, cudaFuncSetAttribute(mlstm_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kStSmem));
-        mlstm_state_kernel<<<dim3((unsigned)tiles, kg, (unsigned)BH), kTcThreads, kStSmem, s>>>(st[0], st[1], st[2], p);
+        mlstm_state_kernel<<<dim3((unsigned)tiles, kg, (unsigned)BH), kTcThreads, kStSmem, s>>>(st[0], st[1], st[2], st[3], st[4], p);
         LUMEN_LAUNCHED(ctx);
-        LUMEN_TRY(make_map_heads(ctx, &out[0], a.u16, a.B * a.S, a.H, a.dim, a.u_ld, kC));
-        LUMEN_TRY(make_map_heads(ctx, &out[1], a.u16 + a.u_k, a.B * a.S, a.H, a.dim, a.u_ld, kC));
+        LUMEN_TRY(make_map_3d(ctx, &out[0], a.u16, a.dim, a.H, a.dim, a.B * a.S, a.u_ld, 1, kC));
+        LUMEN_TRY(make_map_3d(ctx, &out[1], a.u16 + a.u_k, a.dim, a.H, a.dim, a.B * a.S, a.u_ld, 1, kC));
         LUMEN_TRY(make_map(ctx, &out[2], p.s_hi, BH * c * a.vdim, a.dim, 128));
         LUMEN_TRY(make_map(ctx, &out[3], p.s_lo, BH * c * a.vdim, a.dim, 128));
         out[4] = st[0];
-        // as many groups of value tiles as it takes to fill the device once
-        const unsigned z = (unsigned)std::min<size_t>(tiles, (ctx->num_sms + c * BH - 1) / (c * BH));
+        // as many groups of value tiles as the device holds at a time (scores are computed once per group)
+        const unsigned z = (unsigned)std::max<size_t>(1, std::min<size_t>(tiles, ctx->num_sms / (c * BH)));
         const dim3 grid(c, (unsigned)BH, z);
         switch ((a.dim + kBK - 1) / kBK) {
             case 1: LUMEN_TRY(launch_out<1>(ctx, out, p, grid, s)); break;

@@ -47,6 +47,14 @@ __device__ __forceinline__ void tma_load_3d(void *dst, const CUtensorMap *map, i
     asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];"
                  ::"r"(saddr(dst)), "l"(map), "r"(x), "r"(y), "r"(z), "r"(saddr(bar)) : "memory");
 }
+// A tile from shared memory to a 3-D map (what lies beyond the map is not written); one commit group per call of tma_store_commit.
+__device__ __forceinline__ void tma_store_3d(const CUtensorMap *map, const void *src, int x, int y, int z) {
+    asm volatile("cp.async.bulk.tensor.3d.global.shared::cta.bulk_group [%0, {%1, %2, %3}], [%4];"
+                 ::"l"(map), "r"(x), "r"(y), "r"(z), "r"(saddr(src)) : "memory");
+}
+__device__ __forceinline__ void tma_store_commit() { asm volatile("cp.async.bulk.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void tma_store_wait_read() { asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory"); }  // sources may be rewritten
+__device__ __forceinline__ void tma_store_wait() { asm volatile("cp.async.bulk.wait_group 0;" ::: "memory"); }
 // Shared-memory matrix descriptor of a K-major bf16 tile stored as rows of 128 bytes with the 128-byte
 // swizzle (what the TMA box above produces): start address, leading offset 1 (unused with swizzle), 1024
 // bytes between groups of 8 rows, descriptor version 1, layout type 2 = 128-byte swizzle.
@@ -146,14 +154,14 @@ inline int make_map(lumen_ctx *ctx, CUtensorMap *map, const void *base, size_t r
     return LUMEN_OK;
 }
 
-// Rows of `heads` vectors of `dim` bf16 numbers, `ld` elements between rows -> map with box (kBK, 1 head, box_rows): what lies
-// beyond a head's numbers is filled with zeros, not with the next head.
-inline int make_map_heads(lumen_ctx *ctx, CUtensorMap *map, const void *base, size_t rows, size_t heads, size_t dim, size_t ld, int box_rows) {
+// n2 x n1 rows of `n0` bf16 numbers, ld1 and ld2 elements apart -> map with box (kBK, box1, box2): what lies beyond one of the
+// three extents is filled with zeros on loads and left out on stores.
+inline int make_map_3d(lumen_ctx *ctx, CUtensorMap *map, const void *base, size_t n0, size_t n1, size_t ld1, size_t n2, size_t ld2, int box1, int box2) {
     EncodeTiledFn fn = encode_fn();
     if (!fn) return set_error(ctx, LUMEN_ERR_CUDA, "cuTensorMapEncodeTiled is not available from this driver");
-    const cuuint64_t dims[3] = {(cuuint64_t)dim, (cuuint64_t)heads, (cuuint64_t)rows};
-    const cuuint64_t strides[2] = {(cuuint64_t)dim * 2, (cuuint64_t)ld * 2};
-    const cuuint32_t box[3] = {(cuuint32_t)kBK, 1, (cuuint32_t)box_rows};
+    const cuuint64_t dims[3] = {(cuuint64_t)n0, (cuuint64_t)n1, (cuuint64_t)n2};
+    const cuuint64_t strides[2] = {(cuuint64_t)ld1 * 2, (cuuint64_t)ld2 * 2};
+    const cuuint32_t box[3] = {(cuuint32_t)kBK, (cuuint32_t)box1, (cuuint32_t)box2};
     const cuuint32_t estr[3] = {1, 1, 1};
     CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void *>(base), dims, strides, box, estr,
                     CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
