@@ -4,47 +4,20 @@
 // the position alone, however the sequence was cut into steps.
 //
 //   grouped_append_kernel   keys and values of the step -> cache (and queries as the tensor-core kernel reads them)
-//   grouped_rows_kernel     scores, running softmax and weighted values of one row's pieces, any sizes (decode, short portions,
-//                           f32 models); in decode steps it appends the new row itself
+//   grouped_rows_kernel     scores, running softmax and weighted values of one row's pieces in 32-bit FMAs, any sizes; f32 models, and
+//                           sizes that the MMA kernel (grouped_attn_mma.cu) does not take; in decode steps it appends the new row
 //   grouped_merge_kernel    pieces and sink merged, gate applied
 // Whole portions run on the tensor cores (attn_prefill_tc.cu).
 #include <algorithm>
 
 #include "attn_decode.cuh"
-#include "decoder_kernels.cuh"
+#include "grouped_attention.cuh"
 
 namespace lumen {
 namespace {
 
 constexpr int kThreads = 256;
 constexpr int kWarps = kThreads / 32;
-constexpr int kPiece = 32;  // pieces start at multiples of this many rows from the chunk's start
-
-// One head vector by one warp: RMS norm with gains, then the pairs (i, i + rot_dims / 2) turn.  buf: shared memory [dim].
-__device__ __forceinline__ void head_norm_rotate(float *buf, const float *src, int dim, const float *gain, float eps, int rot_dims,
-                                                 const float *cos_row, const float *sin_row, int lane) {
-    float ss = 0.f;
-#pragma unroll 4
-    for (int i = lane; i < dim; i += 32) {
-        const float v = src[i];
-        buf[i] = v;
-        ss = fmaf(v, v, ss);
-    }
-    ss = attn_warp_sum(ss);
-    const float inv = __fdiv_rn(1.0f, sqrtf(__fadd_rn(__fdiv_rn(ss, (float)dim), eps)));
-    for (int i = lane; i < dim; i += 32) buf[i] = __fmul_rn(__fmul_rn(buf[i], inv), gain[i]);
-    __syncwarp();
-    const int half = rot_dims / 2;
-    for (int i = lane; i < half; i += 32) {
-        const float x = buf[i], y = buf[i + half], c = cos_row[i], s = sin_row[i];
-        buf[i] = __fsub_rn(__fmul_rn(x, c), __fmul_rn(y, s));
-        buf[i + half] = __fadd_rn(__fmul_rn(y, c), __fmul_rn(x, s));
-    }
-    __syncwarp();
-}
-
-__device__ __forceinline__ int chunk_start(int pos, size_t chunk) { return chunk ? (int)((size_t)pos / chunk * chunk) : 0; }
-__device__ __forceinline__ int piece_rows(int len, int nsplit) { return ((len + nsplit - 1) / nsplit + kPiece - 1) / kPiece * kPiece; }
 
 // The same in registers, four neighbouring elements per lane (dim <= 128, everything a multiple of four): every load is issued
 // at once, the other half of a pair comes from another lane.
@@ -446,14 +419,17 @@ int group_of(const GroupedArgs &a) {  // query heads a CTA takes
 
 }  // namespace
 
-// Two CTAs per SM, pieces of at least 64 rows, partial results within the workspace (see ensure_workspace).
+// As many CTAs as the device holds, pieces that give every warp something, partial results within the workspace (see
+// ensure_workspace).
 int grouped_pick_splits(const GroupedArgs &a, int num_sms) {
-    const size_t rows = a.B * a.S, items = rows * a.H / group_of(a), total = a.past + a.S;
-    const size_t len = a.chunk ? std::min(total, a.chunk) : total;
-    size_t n = std::min((2 * (size_t)num_sms + items - 1) / items, (len + 63) / 64);
-    n = std::min(std::min(n, (size_t)kMaxPieces), (size_t)num_sms * 64 / (rows * a.H));
-    // few distinct counts: every one of them is a graph of its own
-    size_t p = 1;
+    const bool mma = grouped_mma_usable(a);
+    const size_t rows = a.B * a.S, r = a.H / a.G, items = rows * a.G * (mma ? (r + kMmaHeads - 1) / kMmaHeads : r / group_of(a));
+    const size_t total = a.past + a.S, len = a.chunk ? std::min(total, a.chunk) : total, piece = mma ? 128 : 64;
+    size_t most = std::max<size_t>(1, mma ? num_sms / items : (2 * (size_t)num_sms + items - 1) / items);
+    most = std::min(std::min(most, (size_t)kMaxPieces), std::max<size_t>(1, (size_t)num_sms * 64 / (rows * a.H)));
+    const size_t n = (len + piece - 1) / piece;
+    if (n >= most) return (int)most;
+    size_t p = 1;  // few distinct counts while the context grows: every one of them is a graph of its own
     while (p * 2 <= n) p *= 2;
     return (int)p;
 }
@@ -475,7 +451,8 @@ int launch_grouped_attention(lumen_ctx *ctx, const GroupedArgs &a, bool append, 
     if (std::max(a.dim, a.vdim) > kGroupedMaxDim) return set_error(ctx, LUMEN_ERR_UNSUPPORTED, "attention: heads of %zu / %zu numbers", a.dim, a.vdim);
     const bool f32 = a.dt == LUMEN_F32;
     int rc;
-    switch (group_of(a)) {
+    if (grouped_mma_usable(a)) rc = launch_grouped_mma(ctx, a, append, s);
+    else switch (group_of(a)) {
         case 4: rc = f32 ? launch_rows_g<float, 4>(ctx, a, append, s) : launch_rows_g<__nv_bfloat16, 4>(ctx, a, append, s); break;
         case 2: rc = f32 ? launch_rows_g<float, 2>(ctx, a, append, s) : launch_rows_g<__nv_bfloat16, 2>(ctx, a, append, s); break;
         default: rc = f32 ? launch_rows_g<float, 1>(ctx, a, append, s) : launch_rows_g<__nv_bfloat16, 1>(ctx, a, append, s); break;

@@ -102,10 +102,12 @@ def test_gates_far_from_their_middle(L, dtype, forget, gain):
     dict(heads=5, kv_heads=5, dim=72, vdim=40, chunk=7, rot_dims=2), dict(heads=2, kv_heads=1, dim=192, vdim=120, chunk=1000, rot_dims=48),
     dict(heads=3, kv_heads=1, dim=200, vdim=64, chunk=33, rot_dims=200), dict(heads=8, kv_heads=2, dim=40, vdim=136, chunk=65, rot_dims=8),
     dict(heads=4, kv_heads=2, dim=7, vdim=5, chunk=50, rot_dims=6), dict(heads=2, kv_heads=2, dim=300, vdim=16, chunk=128, rot_dims=10),
+    dict(heads=10, kv_heads=1, dim=64, vdim=40, chunk=90, rot_dims=24), dict(heads=18, kv_heads=2, dim=96, vdim=128, chunk=400, rot_dims=96),
     dict(heads=1, kv_heads=1, dim=16, vdim=8, chunk=1, rot_dims=4), dict(heads=3, kv_heads=3, dim=48, vdim=70, chunk=192, rot_dims=0),
 ])
 def test_attention_alone(L, dtype, a):
-    """Sizes for every kernel: tensor-core prompts with 1 to 3 key blocks and 64 or 128 values, and the row kernel of every width."""
+    """Sizes for every kernel: tensor-core prompts with 1 to 3 key blocks and 64 or 128 values, single rows on the warp-level tensor cores
+    (1 to 4 key blocks, one or two value blocks, up to two groups of heads), and the general row kernel of every width."""
     kw = dict(a, scale=0.6 * a.get("dim", 32) ** -0.5)
     cfg = K.config([(K.attn(**kw), None)])
     mistakes = ["query norm", "key norm", "sink", "head gate"]
