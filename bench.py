@@ -366,7 +366,7 @@ LAYER_CASES = {
     # routed: a token uses 6 of 64 experts and the shared one, 3 x (6 x 1408 + 2816) x 2048 parameters = LlamaModel with 11264
     "moe_2048": dict(width=2048, layers=4, heads=16, rank=512, moe=dict(experts=64, top=6, ff=1408, shared=2816),
                      llama=dict(intermediate_size=11264, num_key_value_heads=8)),
-    # Fekorax: twice (three matrix-memory layers, attention, a matrix-memory layer, attention over the former one's keys and values), the
+    # Fekorax: twice (two matrix-memory layers, attention, two matrix-memory layers, attention over the former one's keys and values), the
     # attention layers with a feed-forward; its parameters are those of 7 layers of the LlamaModel
     "mix_2048": dict(width=2048, layers=7, heads=16, llama=dict(intermediate_size=5632, num_key_value_heads=4),
                      matrix=dict(heads=8, dim=128, vdim=256), chunk=3072),
@@ -382,7 +382,7 @@ def fekorax_layers(c: dict) -> list:
         mixer = dict(heads=c["heads"], kv_heads=c["llama"]["num_key_value_heads"], dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=c["chunk"]),
                      rot=dict(base=500000.0, dims=64, scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192)))
         mlp = dict(kind="dense", ff=c["llama"]["intermediate_size"])
-        out += [matrix] * 3 + [dict(type="attention", mixer=mixer, mlp=mlp), matrix, dict(type="attention", mixer=dict(mixer, kv_from=6 * i + 3), mlp=mlp)]
+        out += [matrix] * 2 + [dict(type="attention", mixer=mixer, mlp=mlp)] + [matrix] * 2 + [dict(type="attention", mixer=dict(mixer, kv_from=6 * i + 2), mlp=mlp)]
     return out
 
 
